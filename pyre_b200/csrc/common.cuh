@@ -105,8 +105,7 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
 // this attribute a kernel lives while its predecessors still write: such a load returned stale activations
 // (seen in the fp32 tile product of tiny models, where three kernels of a chain sit on one SM at once;
 // gone with an ordinary load).  So no kernel parameter in this directory is `__restrict__`, nothing uses
-// __ldg(), and tests/test_bindings.py compiles every source to PTX and fails if an ld.global.nc appears
-// (the one in sincosf's table of 2/pi apart).
+// __ldg(), and tests/test_bindings.py fails if a source asks for such a load.
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 
