@@ -6,7 +6,8 @@ size, window, planes) form a group.  A group has its own pool ``[layers, pages, 
 page_size, head_dim]`` (two planes, keys and values, or one plane of rows that serve as both) (one page number addresses the same page in every layer of the
 group, as in the reference, pyre/paged_cache.py:107), its own allocator and its own
 block table per request.  A group with a window gives a page back as soon as every
-position in it lies before the window of any token still to come; a group without one
+position in it lies before the window of any token still to come and after the first
+positions that stay visible for ever (``PagedKVSpec.keep_first``); a group without one
 gives pages back when the request ends.  The reference has one implicit group and frees
 only at the end (pyre/paged_cache.py:163-167).  Each pool has one page more than the
 allocator hands out (``scratch_page``), and each state buffer one slot more
@@ -45,14 +46,14 @@ def pages_per_group(kv_groups: Sequence, page_size: int, full_pages: int, max_re
     """How many pages each paged group gets when a group that keeps every token gets ``full_pages``.  A group
     whose spec bounds what a request holds (``spec.tokens_held(step_tokens)``: a window) never needs more than
     ``max_requests`` times the pages of that many tokens (one more per request, because a window rarely starts
-    on a page's edge), so its pool is that small; its memory goes to the groups that keep everything."""
+    on a page's edge, and another where the kept first tokens end inside a page), so its pool is that small; its memory goes to the groups that keep everything."""
     out = []
     for g in kv_groups:
         held = g.spec.tokens_held(step_tokens) if hasattr(g.spec, "tokens_held") else None
         if held is None:
             out.append(int(full_pages))
         else:
-            out.append(max(1, min(int(full_pages), max_requests * (pages_for(held, page_size) + 1))))
+            out.append(max(1, min(int(full_pages), max_requests * (pages_for(held, page_size) + 1 + bool(getattr(g.spec, "keep_first", 0))))))
     return out
 
 
@@ -64,7 +65,7 @@ class PagedGroup:
         self.spec, self.n_layers, self.page_size, self.num_pages = spec, n_layers, page_size, num_pages
         self.allocator = PageAllocator(num_pages)
         self.tables: dict[Hashable, list[int]] = {}      # logical page -> physical page, -1 once given back
-        self.first_live: dict[Hashable, int] = {}        # first logical page not yet given back
+        self.first_live: dict[Hashable, int] = {}        # first logical page that may still be given back
         self._rows: dict[Hashable, np.ndarray] = {}      # tables as arrays, dropped whenever a table changes
         # one page beyond the allocator's range belongs to no request: the rows that pad a captured step to a
         # common size write their token there and read it back
@@ -83,7 +84,8 @@ class PagedGroup:
 
     def begin(self, req) -> None:
         self.tables[req] = []
-        self.first_live[req] = 0
+        # the pages of the kept first positions are never given back before the request ends
+        self.first_live[req] = pages_for(getattr(self.spec, "keep_first", 0), self.page_size)
 
     def pages_missing(self, req, new_len: int) -> int:
         return max(0, pages_for(new_len, self.page_size) - len(self.tables[req]))

@@ -812,3 +812,156 @@ class NipudraConfig(ModelConfig):
                 L = dataclasses.replace(L, conv=int(shape[1]))
             layers.append(L)
         return dataclasses.replace(self, layers=tuple(layers))
+
+
+@dataclass(frozen=True)
+class GadopelLayer:
+    """One layer of a Gadopel model: which mixer (``kind``: "latent_attention" or "attention") with its sizes, and the
+    intermediate size ``ff`` of its gated feed-forward (0: none)."""
+
+    kind: str
+    heads: int
+    dim: int                       # query/key entries per head (latent_attention: the unrotated ones)
+    vdim: int                      # value entries per head
+    scale: float                   # factor on q . k
+    kv_heads: int = 0              # attention: key/value heads
+    rot_dim: int = 0               # latent_attention: rotated entries per head beside ``dim``
+    kv_rank: int = 0               # latent_attention: entries of the cached latent
+    rot_dims: int = 0              # leading entries (of a head; of the rotated part) that are rotated
+    rot_base: float = 10000.0
+    rot_scaling: "tuple | None" = None      # attention: (factor, original, fast, slow) or None
+    window: int = 0                # attention: a position sees itself and window - 1 before it (0: all)
+    keep_first: int = 0            # attention: first positions that every later one sees beside its window
+    ff: int = 0
+
+
+@dataclass(frozen=True)
+class GadopelConfig(ModelConfig):
+    """A Gadopel decoder: layers whose mixer and feed-forward read two layer norms of the same stream and enter it
+    together; latent attention with a sink and a gate per head, or grouped-query attention over a window beside the
+    kept first tokens, in any order; a span of layers that runs several times in a row, its input mixed with the
+    embedding's output before every pass.  ``config.json`` keys: ``vocab``, ``width``, ``norm.eps``, ``loop {start, stop,
+    times}`` (absent: no repeated span) and ``layers``, a list of ``{"type", "mixer": {...}, "mlp": {"kind": "dense",
+    "ff"} | null}`` with the mixers ``latent_attention {heads, dim, rot_dim, vdim, kv_rank, scale, rot: {dims, base}}``
+    and ``attention {heads, kv_heads, dim, vdim, scale, mask: {size, keep_first}, rot: {dims, base, scaling: {factor,
+    original, fast, slow}}}``."""
+
+    architecture: ClassVar[str] = "Gadopel"
+    KINDS: ClassVar[tuple] = ("latent_attention", "attention")
+
+    vocab: int
+    width: int
+    norm_eps: float
+    layers: tuple
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 0            # 0: no repeated span
+
+    def __post_init__(self):
+        _positive("vocab", self.vocab)
+        _positive("width", self.width)
+        if not self.norm_eps > 0:
+            raise ConfigError(f"config.json: norm.eps must be positive, got {self.norm_eps}")
+        if not self.layers:
+            raise ConfigError("config.json: layers is empty")
+        if self.loop_times < 0 or (self.loop_times and not 0 <= self.loop_start < self.loop_stop <= len(self.layers)):
+            raise ConfigError(f"config.json: loop (start {self.loop_start}, stop {self.loop_stop}, times {self.loop_times}) must lie "
+                              f"within the {len(self.layers)} layers")
+        for i, L in enumerate(self.layers):
+            where = f"config.json: layers[{i}]"
+            if L.kind not in self.KINDS:
+                raise ConfigError(f"{where}.type {L.kind!r}: known are {', '.join(self.KINDS)}")
+            if min(L.heads, L.dim, L.vdim) <= 0 or not L.scale > 0:
+                raise ConfigError(f"{where}.mixer: heads, dim, vdim and scale must be positive")
+            rotated = L.rot_dim if L.kind == "latent_attention" else L.dim
+            if L.rot_dims < 0 or L.rot_dims % 2 or L.rot_dims > rotated or (L.rot_dims and not L.rot_base > 1):
+                raise ConfigError(f"{where}.mixer.rot: dims ({L.rot_dims}) must be even and at most {rotated}, base above 1")
+            if L.kind == "latent_attention" and (L.kv_rank <= 0 or L.rot_dim < 0):
+                raise ConfigError(f"{where}.mixer: kv_rank must be positive, rot_dim not negative")
+            if L.kind == "attention":
+                if L.kv_heads <= 0 or L.heads % L.kv_heads:
+                    raise ConfigError(f"{where}.mixer.kv_heads ({L.kv_heads}) must divide heads ({L.heads})")
+                if L.window < 0 or L.keep_first < 0:
+                    raise ConfigError(f"{where}.mixer.mask: size and keep_first must not be negative")
+            if L.ff < 0:
+                raise ConfigError(f"{where}.mlp.ff must be positive")
+
+    @classmethod
+    def from_dict(cls, raw: dict[str, Any]) -> "GadopelConfig":
+        norm = raw.get("norm")
+        if not isinstance(norm, dict):
+            raise ConfigError("config.json: required key 'norm' (with 'eps') is missing")
+        layers_raw = raw.get("layers")
+        if not isinstance(layers_raw, (list, tuple)):
+            raise ConfigError("config.json: required key 'layers' is missing")
+        layers = []
+        for i, entry in enumerate(layers_raw):
+            where = f"layers[{i}]"
+            if not isinstance(entry, dict) or not isinstance(entry.get("mixer"), dict):
+                raise ConfigError(f"config.json: {where} needs 'type' and 'mixer'")
+            m, kind = entry["mixer"], str(entry.get("type"))
+            rot = m.get("rot") or {}
+            fields = dict(kind=kind, heads=_require(m, "heads"), dim=_require(m, "dim"), vdim=_require(m, "vdim"),
+                          scale=_require(m, "scale", float), rot_base=float(rot.get("base", 10000.0)))
+            if kind == "latent_attention":
+                fields.update(rot_dim=_require(m, "rot_dim"), kv_rank=_require(m, "kv_rank"))
+                fields["rot_dims"] = int(rot.get("dims", fields["rot_dim"]))
+            elif kind == "attention":
+                sc = rot.get("scaling")
+                if sc is not None:
+                    if not isinstance(sc, dict):
+                        raise ConfigError(f"config.json: {where}.mixer.rot.scaling must be an object or null")
+                    sc = tuple(_require(sc, k, float) for k in ("factor", "original", "fast", "slow"))
+                mask = m.get("mask") or {}
+                fields.update(kv_heads=int(m.get("kv_heads") or fields["heads"]), rot_dims=int(rot.get("dims", 0)), rot_scaling=sc,
+                              window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0))
+            mlp = entry.get("mlp")
+            if mlp is not None:
+                if not isinstance(mlp, dict):
+                    raise ConfigError(f"config.json: {where}.mlp must be an object or null")
+                if mlp.get("kind", "dense") != "dense":
+                    raise ConfigError(f"config.json: {where}.mlp.kind {mlp.get('kind')!r}: known is 'dense'")
+                fields["ff"] = _require(mlp, "ff")
+                _positive(f"{where}.mlp.ff", fields["ff"])
+            layers.append(GadopelLayer(**fields))
+        loop = raw.get("loop")
+        span = {}
+        if loop is not None:
+            if not isinstance(loop, dict):
+                raise ConfigError("config.json: loop must be an object or null")
+            span = dict(loop_start=_require(loop, "start"), loop_stop=_require(loop, "stop"), loop_times=_require(loop, "times"))
+            _positive("loop.times", span["loop_times"])
+        return cls(vocab=_require(raw, "vocab"), width=_require(raw, "width"), norm_eps=_require(norm, "eps", float),
+                   layers=tuple(layers), **span)
+
+    def to_dict(self) -> dict[str, Any]:
+        layers = []
+        for L in self.layers:
+            rot = {"dims": L.rot_dims, "base": L.rot_base}
+            mixer = {"heads": L.heads, "dim": L.dim, "vdim": L.vdim, "scale": L.scale, "rot": rot}
+            if L.kind == "latent_attention":
+                mixer.update(rot_dim=L.rot_dim, kv_rank=L.kv_rank)
+            else:
+                mixer["kv_heads"] = L.kv_heads
+                if L.window:
+                    mixer["mask"] = {"size": L.window, "keep_first": L.keep_first}
+                if L.rot_scaling:
+                    rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), L.rot_scaling))
+            layers.append({"type": L.kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": L.ff} if L.ff else None})
+        out = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
+               "layers": layers}
+        if self.has_loop():
+            out["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        return out
+
+    def has_loop(self) -> bool:
+        return self.loop_times > 0
+
+    def layer_order(self) -> list:
+        """(layer index, does a pass of the repeated span begin here?) in the order the layers run."""
+        if not self.has_loop():
+            return [(i, False) for i in range(len(self.layers))]
+        order = [(i, False) for i in range(self.loop_start)]
+        for _ in range(self.loop_times):
+            order += [(i, i == self.loop_start) for i in range(self.loop_start, self.loop_stop)]
+        return order + [(i, False) for i in range(self.loop_stop, len(self.layers))]

@@ -7,7 +7,8 @@
 // window to the token's own position, with an online softmax (running maximum m, sum l
 // and an fp32 accumulator).  Prompt portions and single decoded tokens are the same
 // case: a query at absolute position p sees the cached keys lo..p, where
-// lo = max(0, p - window + 1) with a window and 0 without; the keys of the current
+// lo = max(0, p - window + 1) with a window and 0 without (and, with a window, the first
+// `keep_first` positions of the sequence, however far back); the keys of the current
 // portion were written to the pages before this kernel runs.
 //
 // The arithmetic of one (token, head) depends on nothing but its own keys: the chunks
@@ -29,7 +30,7 @@ __global__ void paged_attention_generic_kernel(
     int bt_stride,
     const int* seq_of_token,  // [n_tokens]
     const int* positions,     // [n_tokens]
-    int n_tokens, int nh, int nkv, int hd, int page_size, int window, float scale, float sink, const float* head_sinks, long long n_pages, int* err_flag) {
+    int n_tokens, int nh, int nkv, int hd, int page_size, int window, int keep_first, float scale, float sink, const float* head_sinks, long long n_pages, int* err_flag) {
     extern __shared__ float q_smem[];  // [warps][hd]
     pdl_trigger();
     pdl_wait();
@@ -55,9 +56,12 @@ __global__ void paged_attention_generic_kernel(
     for (int i = 0; i < 8; ++i) acc[i] = 0.f;
     float m = -INFINITY, l = 0.f;
 
-    for (int c = (lo / 32) * 32; c <= pos; c += 32) {
+    // the chunks of the kept first keys (if any), then those of the window
+    const int keep = window > 0 ? keep_first : 0, lo_chunk = (lo / 32) * 32;
+    for (int c = keep > 0 ? 0 : lo_chunk; c <= pos; c += 32) {
+        if (c >= keep && c < lo_chunk) c = lo_chunk;
         const int j = c + lane;
-        const bool valid = j >= lo && j <= pos;
+        const bool valid = (j >= lo || j < keep) && j <= pos;
         float score = -INFINITY;
         int vrow = -1;  // row index of this key's value vector, in units of hd elements
         if (valid) {
@@ -95,7 +99,7 @@ __global__ void paged_attention_generic_kernel(
 #pragma unroll
                 for (int u = 0; u < 4; ++u) {
                     pj[u] = __shfl_sync(0xffffffffu, p, (j0 + u) & 31);
-                    vr[u] = (j0 + u < n_keys) ? __shfl_sync(0xffffffffu, vrow, (j0 + u) & 31) : -1;   // -1: before the window, or past the chunk's keys
+                    vr[u] = (j0 + u < n_keys) ? __shfl_sync(0xffffffffu, vrow, (j0 + u) & 31) : -1;   // -1: not visible, or past the chunk's keys
                 }
 #pragma unroll
                 for (int u = 0; u < 4; ++u) {
@@ -120,7 +124,7 @@ __global__ void paged_attention_generic_kernel(
             for (int jj = 0; jj < n_keys; ++jj) {
                 const float pj = __shfl_sync(0xffffffffu, p, jj);
                 const int vr = __shfl_sync(0xffffffffu, vrow, jj);
-                if (vr < 0) continue;  // before the window: same for the whole warp
+                if (vr < 0) continue;  // not visible: same for the whole warp
                 const T* vp = cache + (size_t)vr * hd;
 #pragma unroll
                 for (int i = 0; i < 8; ++i) {
@@ -147,10 +151,10 @@ __global__ void paged_attention_generic_kernel(
 PYRE_API int pyre_paged_attention_generic(const void* q, const void* cache, void* out, const int* block_table,
                                           int bt_stride, const int* seq_of_token, const int* positions,
                                           int n_tokens, int nh, int nkv, int hd, int page_size, int window,
-                                          float scale, float sink, const float* head_sinks, int dtype, long long n_pages,
+                                          int keep_first, float scale, float sink, const float* head_sinks, int dtype, long long n_pages,
                                           int* err_flag, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (hd % 8 || hd > 256 || hd <= 0 || nkv <= 0 || nh % nkv || page_size <= 0) return PYRE_ERR_BAD_ARG;
+    if (hd % 8 || hd > 256 || hd <= 0 || nkv <= 0 || nh % nkv || page_size <= 0 || keep_first < 0) return PYRE_ERR_BAD_ARG;
     const int warps = 4;
     const long long items = (long long)n_tokens * nh;
     const int blocks = (int)ceil_div_ll(items, warps);
@@ -158,11 +162,11 @@ PYRE_API int pyre_paged_attention_generic(const void* q, const void* cache, void
     if (dtype == PYRE_F32)
         pyre_launch(paged_attention_generic_kernel<float>, dim3(blocks), dim3(warps * 32), smem, stream, 
             (const float*)q, (const float*)cache, (float*)out, block_table, bt_stride, seq_of_token, positions,
-            n_tokens, nh, nkv, hd, page_size, window, scale, sink, head_sinks, n_pages, err_flag);
+            n_tokens, nh, nkv, hd, page_size, window, keep_first, scale, sink, head_sinks, n_pages, err_flag);
     else if (dtype == PYRE_BF16)
         pyre_launch(paged_attention_generic_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, stream, 
             (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, block_table, bt_stride,
-            seq_of_token, positions, n_tokens, nh, nkv, hd, page_size, window, scale, sink, head_sinks, n_pages, err_flag);
+            seq_of_token, positions, n_tokens, nh, nkv, hd, page_size, window, keep_first, scale, sink, head_sinks, n_pages, err_flag);
     else return PYRE_ERR_BAD_ARG;
     PYRE_LAUNCH_CHECK();
     return 0;

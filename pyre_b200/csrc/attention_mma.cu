@@ -27,6 +27,9 @@
 // cp.async, zeroed in shared memory after a TMA copy), so stale or non-finite memory in
 // unowned slots cannot reach the result.
 //
+// With a window a sequence's first `keep_first` keys may stay visible: the walk is then over the tiles that hold
+// them followed by the tiles of the window (walk index -> key tile by `key_tile`), and the splits share that walk.
+//
 // Formula: pyre/model.py:104-124, pyre/kernels/paged_attn.py:43-71 (online softmax, fp32
 // scores; probabilities rounded to the activation dtype before the product with V, as
 // pyre/model.py:122 does).
@@ -114,7 +117,7 @@ struct AttnParams {
     const int* block_table;      // [B, bt_stride]
     const int* cu_seqlens;       // [B + 1]
     const int* positions;        // [T]
-    int bt_stride, n_seqs, nh, nkv, page_size, window, n_splits, tpg, hpg, head_blocks;
+    int bt_stride, n_seqs, nh, nkv, page_size, window, keep_first, n_splits, tpg, hpg, head_blocks;
     int page_shift;              // log2(page_size) if it is a power of two, else -1
     int use_tma;                 // tiles come by TMA through `map` (power-of-two pages, HD % 64 == 0): 1 = one copy per
                                  // 128-byte column box, page piece and K/V (pages under 16 tokens), 2 = one 5-d copy per tile
@@ -136,7 +139,8 @@ __device__ __forceinline__ float row_sink_l2(const float* head_sinks, float sink
 
 // CLUSTER: the n_splits CTAs of a (group, kv head) form one thread-block cluster and merge their
 // partial results through distributed shared memory; no scratch, no second kernel.
-template <int HD, bool CLUSTER>
+// KEEP: the variant for a window with kept first keys (p.keep_first > 0); without it the walk is the tiles themselves.
+template <int HD, bool CLUSTER, bool KEEP>
 __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const __grid_constant__ CUtensorMap map, const AttnParams p) {
     constexpr int KSTEPS = HD / 16;
     constexpr int NT_O = HD / 8;  // output n-tiles
@@ -216,7 +220,13 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const _
     const int pos_first = p.positions[tok0], pos_last = p.positions[tok0 + n_tok - 1];
     const int new_from = p.positions[seq_begin];   // the sequence's keys from here on are written by this step
     const int lo_g = (p.window > 0 && pos_first - p.window + 1 > 0) ? pos_first - p.window + 1 : 0;
-    const int tile_lo = lo_g / TILE, tile_hi = pos_last / TILE;
+    // the walk: the tiles of the kept first keys (none without a window), then those from the window's start on;
+    // step kt of it is key tile key_tile(kt).  A key is visible to some row of the group if it lies in [lo_g, pos_last]
+    // or among the first `keep`
+    const int keep = KEEP ? p.keep_first : 0;
+    const int kept_tiles = (keep + TILE - 1) / TILE, tiles_skipped = KEEP ? max(0, lo_g / TILE - kept_tiles) : 0;
+    auto key_tile = [&](int kt) { return !KEEP || kt < kept_tiles ? kt : kt + tiles_skipped; };
+    const int tile_lo = KEEP ? 0 : lo_g / TILE, tile_hi = pos_last / TILE - tiles_skipped;
     const int tiles_total = tile_hi - tile_lo + 1;
     const int tps = (tiles_total + p.n_splits - 1) / p.n_splits;
     const int tile_begin = tile_lo + split * tps;
@@ -237,8 +247,8 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const _
 #pragma unroll
         for (int i = lane; i < TILE * CH; i += 32) {
             const int row = i / CH, c = i % CH;
-            const int key = kt * TILE + row;
-            const bool live = key >= lo_g && key <= pos_last;
+            const int key = key_tile(kt) * TILE + row;
+            const bool live = (key >= lo_g || key < keep) && key <= pos_last;
             const int lp = p.page_shift >= 0 ? key >> p.page_shift : key / p.page_size;
             const int slot = p.page_shift >= 0 ? key & (p.page_size - 1) : key % p.page_size;
             const int page = live ? pyre_checked_page(table[lp], p.n_pages, p.err_flag) : 0;
@@ -269,14 +279,14 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const _
     auto read_pages = [&](int jb) {
         j_base = jb;
         const int kt2 = tile_begin + warp + WARPS * (jb + lane);
-        const int key = kt2 * TILE;
-        const bool live = kt2 < tile_end && key + TILE - 1 >= lo_g && key <= pos_last;
-        pg = live ? pyre_checked_page(table[key >> p.page_shift], p.n_pages, p.err_flag) : 0;   // a tile wholly outside [lo_g, pos_last] reads page 0 (masked)
+        const int key = key_tile(kt2) * TILE;
+        const bool live = kt2 < tile_end && (key + TILE - 1 >= lo_g || key < keep) && key <= pos_last;
+        pg = live ? pyre_checked_page(table[key >> p.page_shift], p.n_pages, p.err_flag) : 0;   // a tile without a visible key reads page 0 (masked)
     };
     if (p.use_tma == 2) read_pages(0);
     // bring tile number j of this warp into `stage` (the whole warp calls; lane 0 issues)
     auto tma_tile = [&](int j, int stage) {
-        const int kt2 = tile_begin + warp + WARPS * j;
+        const int kt2 = key_tile(tile_begin + warp + WARPS * j);
         const uint32_t dst = ring + stage * 2 * TILE_BYTES;
         const uint32_t bar = bar0 + 8 * stage;
         if (p.use_tma == 2) {
@@ -299,9 +309,9 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const _
         const int pieces = TILE / p.box_rows;
         for (int pc = 0; pc < pieces; ++pc) {
             const int key = kt2 * TILE + pc * p.box_rows;
-            // a piece wholly outside [lo_g, pos_last] still has to be filled: read page 0 (its scores are masked)
+            // a piece without a visible key still has to be filled: read page 0 (its scores are masked)
             const int lp = key >> p.page_shift;
-            const bool live = key + p.box_rows - 1 >= lo_g && key <= pos_last;
+            const bool live = (key + p.box_rows - 1 >= lo_g || key < keep) && key <= pos_last;
             const int page = live ? pyre_checked_page(table[lp], p.n_pages, p.err_flag) : 0;
             const int krow = ((page * 2) * p.nkv + kvh) * p.page_size + (key & (p.page_size - 1));
             const int vrow = krow + p.nkv * p.page_size;
@@ -326,7 +336,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const _
     // earlier steps even before this kernel waits for the kernels before it (their latency, and all of the
     // set-up above, then hide behind the kernel that writes this step's keys)
     const int n_mine = tile_begin + warp < tile_end ? (tile_end - tile_begin - warp + WARPS - 1) / WARPS : 0;
-    auto is_old = [&](int j) { return (tile_begin + warp + WARPS * j) * TILE + TILE - 1 < new_from; };
+    auto is_old = [&](int j) { return key_tile(tile_begin + warp + WARPS * j) * TILE + TILE - 1 < new_from; };
 #pragma unroll
     for (int j = 0; j < STAGES - 1; ++j) {
         if (j < n_mine && is_old(j)) {
@@ -371,7 +381,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const _
             else tma_tile(it + STAGES - 1, (it + STAGES - 1) % STAGES);
         }
         cp_async_commit();
-        const int key0 = kt * TILE;
+        const int key0 = key_tile(kt) * TILE;
         const uint32_t k_tile = ring + stage * 2 * TILE_BYTES, v_tile = k_tile + TILE_BYTES;
         if (!tma) {
             cp_async_wait<STAGES - 1>();
@@ -386,13 +396,13 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const _
             }
             timed_out = __any_sync(0xffffffffu, timed_out);   // the whole warp gives up together
             if (timed_out) break;
-            // the copy engine brought whole rows of the page: rows outside [lo_g, pos_last] may hold
+            // the copy engine brought whole rows of the page: rows without a visible key may hold
             // anything, so their values are zeroed here (their scores are masked below)
-            if (key0 + TILE - 1 > pos_last || key0 < lo_g) {
+            if (key0 + TILE - 1 > pos_last || (key0 < lo_g && key0 + TILE > keep)) {
                 for (int i = lane; i < TILE * CH; i += 32) {
                     const int row = i / CH, c = i % CH;
                     const int key = key0 + row;
-                    if (key > pos_last || key < lo_g)
+                    if (key > pos_last || (key < lo_g && key >= keep))
                         asm volatile("st.shared.v4.u32 [%0], {%1, %1, %1, %1};" ::"r"(chunk_addr(v_tile, row, c)), "r"(0u) : "memory");
                 }
             }
@@ -432,7 +442,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const _
                 const int r = c >> 1;
                 if (r == 1 && !upper) { s[i][c] = 0.f; continue; }
                 const int key = key0 + 8 * i + 2 * t + (c & 1);
-                const bool ok = row_ok[r] && key <= row_pos[r] && key >= row_lo[r];
+                const bool ok = row_ok[r] && key <= row_pos[r] && (key >= row_lo[r] || key < keep);
                 s[i][c] = ok ? s[i][c] * sl2 : -INFINITY;
                 tile_max[r] = fmaxf(tile_max[r], s[i][c]);
             }
@@ -711,21 +721,21 @@ bool make_cache_map_5d(CUtensorMap* map, const void* cache, long long n_pages, i
               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int HD>
+template <int HD, bool KEEP>
 int launch(const CUtensorMap& map, const AttnParams& p, int n_groups_bound, bool use_cluster, cudaStream_t stream) {
     dim3 grid(n_groups_bound, p.nkv * p.head_blocks, p.n_splits);
     constexpr int SMEM = WARPS * STAGES * 2 * TILE * HD * 2 + 1024;   // per warp: the stages of a K and a V tile; alignment slack
     static bool configured_on[PYRE_MAX_DEVICES] = {};      // the attributes are per device
     bool& configured = configured_on[pyre_current_device()];
     if (!configured) {   // more than 48 KB of dynamic shared memory and clusters of more than 8 CTAs are opt-ins
-        cudaError_t e = cudaFuncSetAttribute(paged_attention_mma_kernel<HD, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(paged_attention_mma_kernel<HD, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(paged_attention_mma_kernel<HD, true>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaError_t e = cudaFuncSetAttribute(paged_attention_mma_kernel<HD, false, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(paged_attention_mma_kernel<HD, true, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(paged_attention_mma_kernel<HD, true, KEEP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     if (!use_cluster) {
-        cudaError_t e = pyre_launch(paged_attention_mma_kernel<HD, false>, dim3(grid), dim3(WARPS * 32), (size_t)SMEM, stream, map, p);
+        cudaError_t e = pyre_launch(paged_attention_mma_kernel<HD, false, KEEP>, dim3(grid), dim3(WARPS * 32), (size_t)SMEM, stream, map, p);
         if (e != cudaSuccess) return (int)e;
         return (int)cudaGetLastError();
     }
@@ -743,7 +753,7 @@ int launch(const CUtensorMap& map, const AttnParams& p, int n_groups_bound, bool
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = pyre_pdl_enabled() ? 2 : 1;
-    cudaError_t e = cudaLaunchKernelEx(&cfg, paged_attention_mma_kernel<HD, true>, map, p);
+    cudaError_t e = cudaLaunchKernelEx(&cfg, paged_attention_mma_kernel<HD, true, KEEP>, map, p);
     if (e != cudaSuccess) return (int)e;
     return (int)cudaGetLastError();
 }
@@ -759,10 +769,10 @@ PYRE_API long long pyre_attention_mma_scratch_floats(int n_tokens, int nh, int h
 PYRE_API int pyre_paged_attention_mma(const void* q, const void* cache, void* out, float* scratch,
                                       const int* block_table, int bt_stride, const int* cu_seqlens,
                                       const int* positions, int n_tokens, int n_seqs, int nh, int nkv, int hd,
-                                      int page_size, int window, float scale, float sink, const float* head_sinks, int n_splits,
+                                      int page_size, int window, int keep_first, float scale, float sink, const float* head_sinks, int n_splits,
                                       int max_len, long long n_pages, int uniform_len, int* err_flag, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (hd % 16 || hd < 16 || hd > 128 || nkv <= 0 || nh % nkv || page_size <= 0 || n_splits < 1) return PYRE_ERR_UNSUPPORTED;
+    if (hd % 16 || hd < 16 || hd > 128 || nkv <= 0 || nh % nkv || page_size <= 0 || n_splits < 1 || keep_first < 0) return PYRE_ERR_UNSUPPORTED;
     // without scratch the splits merge through a thread-block cluster (at most 16 CTAs)
     const bool use_cluster = n_splits > 1 && !scratch;
     if (use_cluster && n_splits > 16) return PYRE_ERR_BAD_ARG;
@@ -776,7 +786,7 @@ PYRE_API int pyre_paged_attention_mma(const void* q, const void* cache, void* ou
     p.cu_seqlens = cu_seqlens;
     p.positions = positions;
     p.bt_stride = bt_stride; p.n_seqs = n_seqs; p.nh = nh; p.nkv = nkv; p.page_size = page_size;
-    p.window = window; p.n_splits = n_splits; p.scale = scale; p.max_len = max_len;
+    p.window = window; p.keep_first = window > 0 ? keep_first : 0; p.n_splits = n_splits; p.scale = scale; p.max_len = max_len;
     p.sink_l2 = sink * 1.44269504088896341f;
     p.head_sinks = head_sinks;
     p.page_shift = -1;
@@ -802,17 +812,19 @@ PYRE_API int pyre_paged_attention_mma(const void* q, const void* cache, void* ou
     p.head_blocks = (n_rep + p.hpg - 1) / p.hpg;
     const int groups_bound = n_tokens / p.tpg + n_seqs;  // sum over entries of ceil(len / tpg) is at most this
     int rc;
+#define GO(HD_) rc = p.keep_first > 0 ? launch<HD_, true>(map, p, groups_bound, use_cluster, stream) : launch<HD_, false>(map, p, groups_bound, use_cluster, stream); break;
     switch (hd) {
-        case 16: rc = launch<16>(map, p, groups_bound, use_cluster, stream); break;
-        case 32: rc = launch<32>(map, p, groups_bound, use_cluster, stream); break;
-        case 48: rc = launch<48>(map, p, groups_bound, use_cluster, stream); break;
-        case 64: rc = launch<64>(map, p, groups_bound, use_cluster, stream); break;
-        case 80: rc = launch<80>(map, p, groups_bound, use_cluster, stream); break;
-        case 96: rc = launch<96>(map, p, groups_bound, use_cluster, stream); break;
-        case 112: rc = launch<112>(map, p, groups_bound, use_cluster, stream); break;
-        case 128: rc = launch<128>(map, p, groups_bound, use_cluster, stream); break;
+        case 16: GO(16)
+        case 32: GO(32)
+        case 48: GO(48)
+        case 64: GO(64)
+        case 80: GO(80)
+        case 96: GO(96)
+        case 112: GO(112)
+        case 128: GO(128)
         default: return PYRE_ERR_UNSUPPORTED;
     }
+#undef GO
     if (rc) return rc;
     if (n_splits > 1 && !use_cluster) {
         pyre_launch(combine_splits_kernel, dim3(n_tokens * nh), dim3(COMBINE_WARPS * 32), 0, stream, p.part_acc, p.part_ml, p.out, n_splits, hd, nh, cu_seqlens, n_seqs, max_len, p.sink_l2, p.head_sinks);

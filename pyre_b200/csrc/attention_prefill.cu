@@ -4,7 +4,8 @@
 //
 // A CTA owns 64 consecutive tokens of one portion (entry of the step) and one query head;
 // its 4 warps own 16 query rows each and walk the same key tiles, from the tile that holds
-// the start of the first row's window to the tile that holds the last row's position.  A
+// the start of the first row's window (before it those of the `keep_first` first keys that a
+// windowed sequence may keep in view) to the tile that holds the last row's position.  A
 // tile is read from the paged cache row by row through the block table; rows beyond the
 // portion's last position are zero-filled, so unowned cache slots never enter the math.
 // Only entries with at least `min_len` tokens are handled here; shorter ones (decoded
@@ -56,7 +57,7 @@ struct PrefillParams {
     const int* block_table;      // [B, bt_stride]
     const int* cu_seqlens;       // [B + 1]
     const int* positions;        // [T]
-    int bt_stride, n_seqs, nh, nkv, page_size, window, min_len;
+    int bt_stride, n_seqs, nh, nkv, page_size, window, keep_first, min_len;
     float scale;
     float sink;                  // score of a sink without a value that joins every row's denominator; -inf: none
     const float* head_sinks;     // [nh] a sink score per query head instead of `sink`, or null
@@ -106,7 +107,11 @@ __global__ void __launch_bounds__(WARPS * 32, 3) attention_prefill_kernel(const 
     const int lo1 = (p.window > 0 && pos1 - p.window + 1 > 0) ? pos1 - p.window + 1 : 0;
     const int pos_first = p.positions[tok0], pos_last = p.positions[tok0 + n_tok - 1];
     const int lo_cta = (p.window > 0 && pos_first - p.window + 1 > 0) ? pos_first - p.window + 1 : 0;
-    const int tile_lo = lo_cta / BN, tile_hi = pos_last / BN;
+    // the walk: the tiles of the kept first keys (none without a window), then those from the window's start on
+    const int keep = p.window > 0 ? p.keep_first : 0;
+    const int kept_tiles = (keep + BN - 1) / BN, tiles_skipped = max(0, lo_cta / BN - kept_tiles);
+    auto key_tile = [&](int kt) { return kt < kept_tiles ? kt : kt + tiles_skipped; };
+    const int n_tiles = pos_last / BN - tiles_skipped + 1;
     // rows of this warp: positions pos_first + 16 warp .. + 15 (consecutive tokens of one entry)
     const int warp_pos_lo = pos_first + warp * 16, warp_pos_hi = min(pos_first + warp * 16 + 15, pos_last);
     const int warp_key_lo = (p.window > 0 && warp_pos_lo - p.window + 1 > 0) ? warp_pos_lo - p.window + 1 : 0;
@@ -133,8 +138,8 @@ __global__ void __launch_bounds__(WARPS * 32, 3) attention_prefill_kernel(const 
 #pragma unroll
         for (int j = 0; j < BN / ROWS_PER_PASS; ++j) {
             const int row = rr + j * ROWS_PER_PASS;
-            const int key = kt * BN + row;
-            const bool live = key >= lo_cta && key <= pos_last;
+            const int key = key_tile(kt) * BN + row;
+            const bool live = (key >= lo_cta || key < keep) && key <= pos_last;
             const int page = live ? pyre_checked_page(table[key / p.page_size], p.n_pages, p.err_flag) : 0;
             const size_t krow = ((size_t)(page * 2) * p.nkv + kvh) * p.page_size + (live ? key % p.page_size : 0);
             const __nv_bfloat16* ksrc = p.cache + krow * HD + c * 8;
@@ -151,18 +156,18 @@ __global__ void __launch_bounds__(WARPS * 32, 3) attention_prefill_kernel(const 
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
     const float sl2 = p.scale * 1.44269504088896341f;   // scores are kept in units of log2(e)
 
-    load_tile(tile_lo, 0);
+    load_tile(0, 0);
     cp_async_commit();
-    for (int kt = tile_lo; kt <= tile_hi; ++kt) {
-        const int stage = (kt - tile_lo) & 1;
-        if (kt < tile_hi) load_tile(kt + 1, stage ^ 1);
+    for (int kt = 0; kt < n_tiles; ++kt) {
+        const int stage = kt & 1;
+        if (kt + 1 < n_tiles) load_tile(kt + 1, stage ^ 1);
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
 
-        const int key0 = kt * BN;
+        const int key0 = key_tile(kt) * BN;
         // this warp needs the tile only if it holds a key that one of its rows may see
-        if (key0 <= warp_pos_hi && key0 + BN - 1 >= warp_key_lo && warp * 16 < n_tok) {
+        if (key0 <= warp_pos_hi && (key0 + BN - 1 >= warp_key_lo || key0 < keep) && warp * 16 < n_tok) {
             const uint32_t k_tile = smem_base + stage * 2 * TILE_BYTES, v_tile = k_tile + TILE_BYTES;
             // ---- S = Q K^T : 8 key n-tiles
             float s[BN / 8][4];
@@ -190,14 +195,14 @@ __global__ void __launch_bounds__(WARPS * 32, 3) attention_prefill_kernel(const 
             // on the raw scores (the scale is positive) in four independent chains; the scale and
             // the maximum enter the exponent through one fused multiply-add; the accumulator is
             // rescaled only when some row's maximum moved.
-            const bool need_mask = key0 + BN - 1 > warp_pos_lo || (p.window > 0 && key0 < warp_key_lo + 15) || !ok0 || !ok1;
+            const bool need_mask = key0 + BN - 1 > warp_pos_lo || (p.window > 0 && key0 < warp_key_lo + 15 && key0 + BN > keep) || !ok0 || !ok1;
             if (need_mask) {
 #pragma unroll
                 for (int i = 0; i < BN / 8; ++i)
 #pragma unroll
                     for (int c = 0; c < 4; ++c) {
                         const int key = key0 + 8 * i + 2 * t + (c & 1);
-                        const bool okk = (c < 2) ? (ok0 && key <= pos0 && key >= lo0) : (ok1 && key <= pos1 && key >= lo1);
+                        const bool okk = (c < 2) ? (ok0 && key <= pos0 && (key >= lo0 || key < keep)) : (ok1 && key <= pos1 && (key >= lo1 || key < keep));
                         s[i][c] = okk ? s[i][c] : -INFINITY;
                     }
             }
@@ -307,15 +312,15 @@ int launch(const PrefillParams& p, int tiles_bound, cudaStream_t stream) {
 // head sizes 64 and 128.  n_long_tokens: total tokens of those entries (bounds the grid).
 PYRE_API int pyre_attention_prefill(const void* q, const void* cache, void* out, const int* block_table, int bt_stride,
                                     const int* cu_seqlens, const int* positions, int n_long_tokens, int n_seqs, int nh,
-                                    int nkv, int hd, int page_size, int window, float scale, float sink, const float* head_sinks,
+                                    int nkv, int hd, int page_size, int window, int keep_first, float scale, float sink, const float* head_sinks,
                                     int min_len, long long n_pages, int* err_flag, cudaStream_t stream) {
     if (n_long_tokens <= 0) return 0;
-    if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv || page_size <= 0 || min_len < 1) return PYRE_ERR_UNSUPPORTED;
+    if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv || page_size <= 0 || min_len < 1 || keep_first < 0) return PYRE_ERR_UNSUPPORTED;
     PrefillParams p;
     p.q = (const __nv_bfloat16*)q; p.cache = (const __nv_bfloat16*)cache; p.out = (__nv_bfloat16*)out;
     p.block_table = block_table; p.cu_seqlens = cu_seqlens; p.positions = positions;
     p.bt_stride = bt_stride; p.n_seqs = n_seqs; p.nh = nh; p.nkv = nkv; p.page_size = page_size;
-    p.window = window; p.min_len = min_len; p.scale = scale; p.sink = sink; p.head_sinks = head_sinks; p.n_pages = n_pages; p.err_flag = err_flag;
+    p.window = window; p.keep_first = keep_first; p.min_len = min_len; p.scale = scale; p.sink = sink; p.head_sinks = head_sinks; p.n_pages = n_pages; p.err_flag = err_flag;
     const int tiles_bound = n_long_tokens / BM + n_seqs;
     return hd == 128 ? launch<128>(p, tiles_bound, stream) : launch<64>(p, tiles_bound, stream);
 }

@@ -4,7 +4,8 @@
 //
 // A CTA (224 threads) owns 128 consecutive tokens of one portion and one query head and walks
 // the keys in tiles of 64, from the tile holding the start of the first row's window to the
-// tile holding the last row's position:
+// tile holding the last row's position (with a window, the tiles of the first `keep_first` keys,
+// which may stay visible, come before them in the same walk):
 //   warps 0 and 6      : TMA producers (lane 0 issues).  Warp 0 copies the Q tile once (128 rows
 //                        of this head out of the [T, nh * hd] activation matrix) and then the K
 //                        tiles, warp 6 the V tiles: per key tile the rows of 64 / box_rows pages
@@ -176,7 +177,7 @@ struct TcParams {
     const int* block_table;      // [B, bt_stride]
     const int* cu_seqlens;       // [B + 1]
     const int* positions;        // [T]
-    int bt_stride, n_seqs, nh, nkv, page_size, page_shift, box_rows, window, min_len;
+    int bt_stride, n_seqs, nh, nkv, page_size, page_shift, box_rows, window, keep_first, min_len;
     float scale;
     float sink_l2;               // score of a sink without a value, in units of log2(e): 2^(sink_l2 - max) joins every row's
                                  // denominator once, where the row is normalised; -inf: none
@@ -206,7 +207,8 @@ struct Smem {
     static constexpr int TOTAL = OFF_BAR + N_BARS * 8 + 16;   // the dynamic window must start 1024-byte aligned (checked)
 };
 
-template <int HD>
+// KEEP: the variant for a window with kept first keys (p.keep_first > 0); without it the walk is the tiles themselves.
+template <int HD, bool KEEP>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const TcParams p) {
     using L = Smem<HD>;
@@ -251,7 +253,12 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int* table = p.block_table + (size_t)seq * p.bt_stride;
     const int pos_first = p.positions[tok0], pos_last = pos_first + n_tok - 1;   // consecutive positions
     const int lo_cta = (p.window > 0 && pos_first - p.window + 1 > 0) ? pos_first - p.window + 1 : 0;
-    int tile_lo = lo_cta / BN, tile_hi = pos_last / BN;
+    // the walk: the tiles of the kept first keys (none without a window), then those from the window's start on;
+    // step i of it is key tile key_tile(i).  [tile_lo, tile_hi] is this CTA's part of the walk
+    const int keep = KEEP ? p.keep_first : 0;
+    const int kept_tiles = (keep + BN - 1) / BN, tiles_skipped = KEEP ? max(0, lo_cta / BN - kept_tiles) : 0;
+    auto key_tile = [&](int i) { return !KEEP || i < kept_tiles ? i : i + tiles_skipped; };
+    int tile_lo = KEEP ? 0 : lo_cta / BN, tile_hi = pos_last / BN - tiles_skipped;
     if (p.key_splits > 1) {
         // this CTA's share of the key tiles; a share may be empty (few tiles): it says so and leaves
         const int per = (tile_hi - tile_lo + p.key_splits) / p.key_splits;
@@ -308,9 +315,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         // more); lane pc holds the page number of piece pc, read two tiles ahead of its use.
         const int pieces = BN / p.box_rows;   // at most 16 (pages of 4 tokens or more)
         auto read_pages = [&](int i) -> int {
-            const int key = (tile_lo + i) * BN + lane * p.box_rows;
-            const bool live = lane < pieces && i < n_tiles && key + p.box_rows - 1 >= lo_cta && key <= pos_last;
-            return live ? pyre_checked_page(table[key >> p.page_shift], p.n_pages, p.err_flag) : 0;   // pieces outside the range read page 0 (masked)
+            const int key = key_tile(tile_lo + i) * BN + lane * p.box_rows;
+            const bool live = lane < pieces && i < n_tiles && (key + p.box_rows - 1 >= lo_cta || key < keep) && key <= pos_last;
+            return live ? pyre_checked_page(table[key >> p.page_shift], p.n_pages, p.err_flag) : 0;   // pieces without a visible key read page 0 (masked)
         };
         const uint32_t bar_empty = which ? bar_o : bar_s, bar_full = which ? bar_v_full : bar_k_full;
         const uint32_t ring = base + (which ? L::OFF_V : L::OFF_K);
@@ -330,7 +337,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 const int box = b0 + lane, pc = box / HALVES, h = box - pc * HALVES;
                 const int page = __shfl_sync(0xffffffffu, pg0, pc & 31);
                 if (box < pieces * HALVES) {
-                    const int key = (tile_lo + i) * BN + pc * p.box_rows;
+                    const int key = key_tile(tile_lo + i) * BN + pc * p.box_rows;
                     const int row = page * page_rows + row_base + (key & (p.page_size - 1));
                     tma_load_2d(dst + h * (BN * 128) + pc * p.box_rows * 128, &map_kv, full, h * 64, row);
                 }
@@ -397,7 +404,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         bool alive = true;
         for (int i = 0; i < n_tiles && alive; ++i) {
             const int s = i & 1;
-            const int key0 = (tile_lo + i) * BN;
+            const int key0 = key_tile(tile_lo + i) * BN;
             bool ok = mbar_wait(bar_s + 8 * s, (i >> 1) & 1, abort_flag, p.err_flag);
             alive = __all_sync(0xffffffffu, ok);
             if (!alive) break;
@@ -418,13 +425,22 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             }
             // mask by position (only tiles that some row's causal limit or window edge cuts; rows
             // beyond the portion's end are never stored, so they need no mask); the raw maximum in four chains
-            const bool need_mask = key0 + BN - 1 > pos_first || (p.window > 0 && key0 < pos_last - p.window + 1);
+            const bool need_mask = key0 + BN - 1 > pos_first || (p.window > 0 && key0 < pos_last - p.window + 1 && key0 + BN > keep);
             if (need_mask) {
+                if constexpr (KEEP) {
+                    // the tile's visible keys of this row as bits: [.., pos] and ([lo, ..] or [.., keep))
+                    auto below = [](int n) -> uint64_t { return n <= 0 ? 0ull : n >= 64 ? ~0ull : (1ull << n) - 1; };
+                    const uint64_t vis = row_ok ? below(pos + 1 - key0) & (~below(lo - key0) | below(keep - key0)) : 0ull;
+                    const uint32_t half[2] = {(uint32_t)vis, (uint32_t)(vis >> 32)};
 #pragma unroll
-                for (int c = 0; c < BN; ++c) {
-                    const int key = key0 + c;
-                    const bool okk = row_ok && key <= pos && key >= lo;
-                    sc[c] = okk ? sc[c] : -INFINITY;
+                    for (int c = 0; c < BN; ++c) sc[c] = (half[c >> 5] >> (c & 31)) & 1u ? sc[c] : -INFINITY;
+                } else {
+#pragma unroll
+                    for (int c = 0; c < BN; ++c) {
+                        const int key = key0 + c;
+                        const bool okk = row_ok && key <= pos && key >= lo;
+                        sc[c] = okk ? sc[c] : -INFINITY;
+                    }
                 }
             }
             float tm[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -477,8 +493,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
                 }
             }
-            // rows of the V tile outside [lo_cta, pos_last] hold whatever the page holds: zero them
-            if (key0 + BN - 1 > pos_last || key0 < lo_cta) {
+            // rows of the V tile without a visible key hold whatever the page holds: zero them
+            if (key0 + BN - 1 > pos_last || (key0 < lo_cta && key0 + BN > keep)) {
                 ok = mbar_wait(bar_v_full + 8 * s, (i >> 1) & 1, abort_flag, p.err_flag);   // the tile has landed
                 alive = __all_sync(0xffffffffu, ok);
                 if (!alive) break;
@@ -486,7 +502,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 for (int idx = threadIdx.x - 64; idx < BN * HALVES * 8; idx += 128) {
                     const int k = idx / (HALVES * 8), rem = idx % (HALVES * 8);
                     const int key = key0 + k;
-                    if (key > pos_last || key < lo_cta)
+                    if (key > pos_last || (key < lo_cta && key >= keep))
                         asm volatile("st.shared.v4.u32 [%0], {%1, %1, %1, %1};" ::"r"(vd + (rem >> 3) * (BN * 128) + k * 128 + (rem & 7) * 16), "r"(0u) : "memory");
                 }
             }
@@ -635,17 +651,17 @@ bool make_map(CUtensorMap* map, const void* ptr, long long rows, long long cols,
               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int HD>
+template <int HD, bool KEEP>
 int launch(const CUtensorMap& mq, const CUtensorMap& mkv, const TcParams& p, int tiles_bound, cudaStream_t stream) {
     using L = Smem<HD>;
     static bool configured_on[PYRE_MAX_DEVICES] = {};      // the attributes are per device
     bool& configured = configured_on[pyre_current_device()];
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<HD, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    cudaError_t e = pyre_launch(attention_tc_kernel<HD>, dim3(p.nh, tiles_bound, p.key_splits), dim3(THREADS), (size_t)L::TOTAL, stream, mq, mkv, p);
+    cudaError_t e = pyre_launch(attention_tc_kernel<HD, KEEP>, dim3(p.nh, tiles_bound, p.key_splits), dim3(THREADS), (size_t)L::TOTAL, stream, mq, mkv, p);
     if (e != cudaSuccess) return (int)e;
     if (p.key_splits > 1) {
         e = pyre_launch(combine_shares_kernel<HD>, dim3(p.nh, tiles_bound), dim3(128), 0, stream, p);
@@ -664,10 +680,10 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mkv, const TcParams& p, int
 PYRE_API int pyre_attention_prefill_tc(const void* q, const void* cache, void* out, const int* block_table,
                                        int bt_stride, const int* cu_seqlens, const int* positions, int n_tokens,
                                        int n_long_tokens, int n_seqs, int nh, int nkv, int hd, int page_size,
-                                       long long n_pages, int window, float scale, float sink, const float* head_sinks, int min_len,
+                                       long long n_pages, int window, int keep_first, float scale, float sink, const float* head_sinks, int min_len,
                                        int key_splits, float* part_o, float* part_ml, int* err_flag, cudaStream_t stream) {
     if (n_long_tokens <= 0) return 0;
-    if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv || page_size < 4 || (page_size & (page_size - 1)) || min_len < 1)
+    if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv || page_size < 4 || (page_size & (page_size - 1)) || min_len < 1 || keep_first < 0)
         return PYRE_ERR_UNSUPPORTED;
     const long long kv_rows = n_pages * 2 * nkv * page_size;
     if (((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 31) || kv_rows >= (1ll << 31) || n_pages <= 0)
@@ -679,7 +695,7 @@ PYRE_API int pyre_attention_prefill_tc(const void* q, const void* cache, void* o
     p.page_shift = 0;
     while ((1 << p.page_shift) < page_size) ++p.page_shift;
     p.box_rows = page_size < BN ? page_size : BN;
-    p.window = window; p.min_len = min_len; p.scale = scale; p.sink_l2 = sink * 1.44269504088896341f; p.head_sinks = head_sinks; p.err_flag = err_flag; p.n_pages = n_pages;
+    p.window = window; p.keep_first = window > 0 ? keep_first : 0; p.min_len = min_len; p.scale = scale; p.sink_l2 = sink * 1.44269504088896341f; p.head_sinks = head_sinks; p.err_flag = err_flag; p.n_pages = n_pages;
     if (key_splits < 1 || key_splits > 32 || (key_splits > 1 && (!part_o || !part_ml || ((uintptr_t)part_o & 31)))) return PYRE_ERR_BAD_ARG;
     p.key_splits = key_splits; p.part_o = part_o; p.part_ml = part_ml;
     CUtensorMap mq, mkv;
@@ -689,5 +705,7 @@ PYRE_API int pyre_attention_prefill_tc(const void* q, const void* cache, void* o
     if (!make_map(&mkv, cache, kv_rows, hd, hd, p.box_rows)) return PYRE_ERR_UNSUPPORTED;
     const int tiles_bound = n_long_tokens / BM + n_seqs;
     if (tiles_bound > 65535) return PYRE_ERR_BAD_ARG;   // grid.y
-    return hd == 128 ? launch<128>(mq, mkv, p, tiles_bound, stream) : launch<64>(mq, mkv, p, tiles_bound, stream);
+    if (p.keep_first > 0)
+        return hd == 128 ? launch<128, true>(mq, mkv, p, tiles_bound, stream) : launch<64, true>(mq, mkv, p, tiles_bound, stream);
+    return hd == 128 ? launch<128, false>(mq, mkv, p, tiles_bound, stream) : launch<64, false>(mq, mkv, p, tiles_bound, stream);
 }

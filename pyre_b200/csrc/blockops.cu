@@ -227,6 +227,8 @@ PYRE_API int pyre_activation(const void* in, void* out, long long n, int kind, i
 //         n = (v * (1 / sqrt(mean(v^2) + eps))) * w; null: no norm
 //   rotation (pairs (j, j + rot / 2), j < rot / 2, after the norm):
 //         out[j] = n[j] cos[j] - n[j + rot/2] sin[j];  out[j + rot/2] = n[j + rot/2] cos[j] + n[j] sin[j]
+//         neighbours: the pairs are (2j, 2j + 1) instead
+//   post_norm: after the rotation a head's query or key is divided by its root mean square over the dk dims (same eps)
 //   vcos_t, vsin_t [T, dv / 2] or null: the VALUES are turned too, over all their dv dims (pairs (m, m + dv / 2)),
 //         by tables of their own, and cached so; whoever reads them turns the weighted sum back (head_gate below)
 //   q_out [T, nh, D]; cache: one layer [page][2][nkv][page_size][D]; slot_mapping[t] < 0: store nothing
@@ -237,7 +239,7 @@ __global__ void qk_norm_rope_write_kernel(const T* proj, long long row_stride, i
                                           const float* q_w, const float* k_w, float eps, const float* cos_t,
                                           const float* sin_t, const float* vcos_t, const float* vsin_t, T* q_out, T* cache,
                                           const int* slot_mapping, int n_tokens, int nh, int nkv, int dk, int dv, int D,
-                                          int rot, int page_size, long long n_pages, int* err_flag) {
+                                          int rot, int neighbours, int post_norm, int page_size, long long n_pages, int* err_flag) {
     extern __shared__ float head_smem[];   // [warps][D]
     pdl_trigger();
     pdl_wait();
@@ -294,19 +296,38 @@ __global__ void qk_norm_rope_write_kernel(const T* proj, long long row_stride, i
     const int half = rot / 2;
     const float* ct = cos_t ? cos_t + (size_t)t * half : nullptr;
     const float* st = sin_t ? sin_t + (size_t)t * half : nullptr;
-    for (int d = lane; d < D; d += 32) {
-        float o = 0.f;
-        if (d < half) o = __fadd_rn(__fmul_rn(n[d], ct[d]), __fmul_rn(-n[d + half], st[d]));
-        else if (d < rot) o = __fadd_rn(__fmul_rn(n[d], ct[d - half]), __fmul_rn(n[d - half], st[d - half]));
-        else if (d < dk) o = n[d];
-        dst[d] = from_f32<T>(o);
+    if (!neighbours && !post_norm) {
+        for (int d = lane; d < D; d += 32) {
+            float o = 0.f;
+            if (d < half) o = __fadd_rn(__fmul_rn(n[d], ct[d]), __fmul_rn(-n[d + half], st[d]));
+            else if (d < rot) o = __fadd_rn(__fmul_rn(n[d], ct[d - half]), __fmul_rn(n[d - half], st[d - half]));
+            else if (d < dk) o = n[d];
+            dst[d] = from_f32<T>(o);
+        }
+        return;
     }
+    // a lane owns the pairs lane, lane + 32, ... and turns them in place
+    for (int i = lane; i < half; i += 32) {
+        const int a = neighbours ? 2 * i : i, b = neighbours ? 2 * i + 1 : i + half;
+        const float u = n[a], v = n[b];
+        n[a] = __fadd_rn(__fmul_rn(u, ct[i]), __fmul_rn(-v, st[i]));
+        n[b] = __fadd_rn(__fmul_rn(v, ct[i]), __fmul_rn(u, st[i]));
+    }
+    __syncwarp();
+    float rstd = 1.f;
+    if (post_norm) {
+        ss = 0.f;
+        for (int d = lane; d < dk; d += 32) ss = fmaf(n[d], n[d], ss);
+        ss = warp_sum(ss);
+        rstd = 1.0f / sqrtf(ss / (float)dk + eps);
+    }
+    for (int d = lane; d < D; d += 32) dst[d] = from_f32<T>(d < dk ? __fmul_rn(n[d], rstd) : 0.f);
 }
 
 PYRE_API int pyre_qk_norm_rope_write(const void* proj, long long row_stride, int q_col, int k_col, int v_col,
                                      const float* q_w, const float* k_w, float eps, const float* cos_t, const float* sin_t,
                                      const float* vcos_t, const float* vsin_t, void* q_out, void* cache, const int* slot_mapping, int n_tokens, int nh, int nkv,
-                                     int dk, int dv, int D, int rot, int page_size, int dtype, long long n_pages,
+                                     int dk, int dv, int D, int rot, int neighbours, int post_norm, int page_size, int dtype, long long n_pages,
                                      int* err_flag, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (dk <= 0 || dv <= 0 || D < dk || D < dv || rot < 0 || rot > dk || rot % 2 || page_size <= 0 || nh <= 0 || nkv <= 0)
@@ -319,9 +340,9 @@ PYRE_API int pyre_qk_norm_rope_write(const void* proj, long long row_stride, int
     const int blocks = (int)ceil_div_ll(items, warps);
     const size_t smem = (size_t)warps * D * sizeof(float);
     if (dtype == PYRE_BF16)
-        pyre_launch(qk_norm_rope_write_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, stream, (const __nv_bfloat16*)proj, row_stride, q_col, k_col, v_col, q_w, k_w, eps, cos_t, sin_t, vcos_t, vsin_t, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, page_size, n_pages, err_flag);
+        pyre_launch(qk_norm_rope_write_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, stream, (const __nv_bfloat16*)proj, row_stride, q_col, k_col, v_col, q_w, k_w, eps, cos_t, sin_t, vcos_t, vsin_t, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, neighbours, post_norm, page_size, n_pages, err_flag);
     else if (dtype == PYRE_F32)
-        pyre_launch(qk_norm_rope_write_kernel<float>, dim3(blocks), dim3(warps * 32), smem, stream, (const float*)proj, row_stride, q_col, k_col, v_col, q_w, k_w, eps, cos_t, sin_t, vcos_t, vsin_t, (float*)q_out, (float*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, page_size, n_pages, err_flag);
+        pyre_launch(qk_norm_rope_write_kernel<float>, dim3(blocks), dim3(warps * 32), smem, stream, (const float*)proj, row_stride, q_col, k_col, v_col, q_w, k_w, eps, cos_t, sin_t, vcos_t, vsin_t, (float*)q_out, (float*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, neighbours, post_norm, page_size, n_pages, err_flag);
     else return PYRE_ERR_BAD_ARG;
     PYRE_LAUNCH_CHECK();
     return 0;

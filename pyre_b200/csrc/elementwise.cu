@@ -455,10 +455,10 @@ PYRE_API int pyre_qkv_rope_write(const void* qkv, const float* partials, int n_p
 }
 
 // ---------------------------------------------------------------------------
-// out[t, i] = silu(gu[t, i]) * gu[t, I + i],  silu(z) = z / (1 + exp(-z))  in fp32.
+// out[t, i] = act(gu[t, i]) * gu[t, I + i] in fp32; act: silu, z / (1 + exp(-z)), or (relu) max(z, 0).
 // ---------------------------------------------------------------------------
 template <typename T, int VEC>
-__global__ void silu_mul_kernel(const T* gu, T* out, int n_tokens, int I, int block) {
+__global__ void silu_mul_kernel(const T* gu, T* out, int n_tokens, int I, int block, int relu) {
     pdl_trigger();
     pdl_wait();
     const size_t per_row = (size_t)(I / VEC);
@@ -476,7 +476,7 @@ __global__ void silu_mul_kernel(const T* gu, T* out, int n_tokens, int I, int bl
 #pragma unroll
         for (int k = 0; k < VEC; ++k) {
             const float z = to_f32<T>(g.v[k]);
-            const float s = z / (1.0f + expf(-z));
+            const float s = relu ? fmaxf(z, 0.f) : z / (1.0f + expf(-z));
             o.v[k] = from_f32<T>(__fmul_rn(s, to_f32<T>(u.v[k])));
         }
         store_vec<T, VEC>(out + t * (size_t)I + i, o);
@@ -485,7 +485,7 @@ __global__ void silu_mul_kernel(const T* gu, T* out, int n_tokens, int I, int bl
 
 // block: 0 for gate_up = [gates | ups]; n > 0 for gates and ups interleaved in blocks of n features
 // (n a multiple of 8 that divides I).
-PYRE_API int pyre_silu_mul(const void* gu, void* out, int n_tokens, int I, int block, int dtype, cudaStream_t stream) {
+PYRE_API int pyre_silu_mul(const void* gu, void* out, int n_tokens, int I, int block, int relu, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || I <= 0) return 0;
     if (block < 0 || (block > 0 && (block % 8 || I % block))) return PYRE_ERR_BAD_ARG;
     const int threads = 256;
@@ -493,7 +493,7 @@ PYRE_API int pyre_silu_mul(const void* gu, void* out, int n_tokens, int I, int b
     do {                                                                                                   \
         long long total = (long long)n_tokens * (I / V);                                                   \
         int blocks = (int)min((long long)pyre_sm_count() * 16, ceil_div_ll(total, threads));                           \
-        pyre_launch(silu_mul_kernel<TT, V>, dim3(blocks), dim3(threads), 0, stream, (const TT*)gu, (TT*)out, n_tokens, I, block);      \
+        pyre_launch(silu_mul_kernel<TT, V>, dim3(blocks), dim3(threads), 0, stream, (const TT*)gu, (TT*)out, n_tokens, I, block, relu);      \
     } while (0)
     if (dtype == PYRE_F32) { if (I % 4 == 0) LAUNCH(float, 4); else LAUNCH(float, 1); }
     else if (dtype == PYRE_BF16) { if (I % 8 == 0) LAUNCH(__nv_bfloat16, 8); else if (I % 4 == 0) LAUNCH(__nv_bfloat16, 4); else LAUNCH(__nv_bfloat16, 1); }

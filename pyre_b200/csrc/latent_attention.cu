@@ -9,8 +9,12 @@
 //   latent_rotate_q  rotation of the queries' rotated part into the absorbed query rows
 //   latent_attention_exact   fp32 arithmetic, any sizes, bit-identical under cutting and batching
 //
-// Rotation (neighbouring pairs): (u, v) = (x[2i], x[2i + 1]) -> (u cos a - v sin a, v cos a + u sin a), i < rot / 2,
-// with cos/sin of the token's angles from a table [T, rot / 2]; entries from `rot` on pass unchanged.
+// Rotation: (u, v) -> (u cos a - v sin a, v cos a + u sin a) for the pairs (x[2i], x[2i + 1]) (`halves` 0) or
+// (x[i], x[i + rot / 2]) (`halves` 1), i < rot / 2, with cos/sin of the token's angles from a table [T, rot / 2];
+// entries from `rot` on pass unchanged.
+// A sink per head (`head_sinks`, null: none) adds exp(sink) to a row's denominator, with no value; a gate per head
+// (`gates`: activation-dtype logits at gates[t * gate_stride + h], null: none) multiplies a head's normalised sum by
+// its sigmoid, which commutes with the head's value map.
 // `dtype`: type of activations and cache (0 = float32, 1 = bfloat16); all arithmetic is fp32.
 #include "common.cuh"
 
@@ -24,11 +28,30 @@ __device__ __forceinline__ float proj_at(const T* proj, const float* parts, int 
     return to_f32<T>(proj[at]);
 }
 
+// Entry i of a rotated vector whose entries at(j) gives; c, s: the token's cos and sin
+template <typename At>
+__device__ __forceinline__ float turned(At at, int i, int rot, int halves, const float* c, const float* s) {
+    const float v = at(i);
+    if (i >= rot) return v;
+    const int half = rot >> 1;
+    const bool second = halves ? i >= half : (i & 1);
+    const int pair = halves ? (second ? i - half : i) : i >> 1;
+    const float other = at(halves ? (second ? i - half : i + half) : i ^ 1);
+    return second ? fmaf(v, c[pair], __fmul_rn(other, s[pair])) : fmaf(v, c[pair], -__fmul_rn(other, s[pair]));
+}
+
+template <typename T>
+__device__ __forceinline__ float head_gate_of(const T* gates, long long gate_stride, size_t t, int h) {
+    return gates ? 1.0f / (1.0f + expf(-to_f32<T>(gates[t * gate_stride + h]))) : 1.0f;
+}
+
 // ---------------------------------------------------------------------------
 // proj [T, W] (activation dtype, or fp32 partial sums): columns [q_col, q_col + q_rank) the query latent,
 // [c_col, c_col + rank) the key/value latent, [c_col + rank, c_col + rank + rope) the shared key part.
 //   cq_out[t]      = rmsnorm(query latent) * wq            [T, q_rank]   (q_rank = 0: none)
 //   cache[slot[t]] = [ rmsnorm(latent) * wc | rotate(key part) ]          rows of `row` >= rank + rope entries
+//   qa[t, h, rank ..] = [ rotate(rotated part of head h's query) | 0 ]    (qa null: the queries are handled elsewhere);
+//                       head h's query lies at column qh_col + h (dq + rope), its rotated part last
 // One block per token.
 // ---------------------------------------------------------------------------
 template <typename T>
@@ -36,7 +59,7 @@ __global__ void latent_prepare_kernel(const T* proj, const float* parts, int n_p
                                       int q_col, int q_rank, int c_col, int rank, int rope, int rot, const float* wq,
                                       const float* wc, float eps, const float* cos_t, const float* sin_t, T* cq_out,
                                       T* cache, const int* slot_mapping, int row, long long n_pages, int page_size,
-                                      int* err_flag) {
+                                      int halves, T* qa, int qh_col, int nh, int dq, int* err_flag) {
     __shared__ float scratch[33];
     pdl_trigger();
     pdl_wait();
@@ -54,6 +77,20 @@ __global__ void latent_prepare_kernel(const T* proj, const float* parts, int n_p
             cq_out[(size_t)t * q_rank + i] = from_f32<T>(__fmul_rn(__fmul_rn(v, rstd), wq[i]));
         }
     }
+    const float* ct = cos_t + (size_t)t * (rot / 2);
+    const float* st = sin_t + (size_t)t * (rot / 2);
+    if (qa) {
+        const int tail = row - rank;
+        for (int idx = threadIdx.x; idx < nh * tail; idx += blockDim.x) {
+            const int h = idx / tail, i = idx - h * tail;
+            float o = 0.f;
+            if (i < rope) {
+                const size_t at0 = base + qh_col + (size_t)h * (dq + rope) + dq;
+                o = turned([&](int j) { return proj_at<T>(proj, parts, n_parts, part_stride, at0 + j); }, i, rot, halves, ct, st);
+            }
+            qa[((size_t)t * nh + h) * row + rank + i] = from_f32<T>(o);
+        }
+    }
     const int slot = cache ? pyre_checked_slot(slot_mapping[t], n_pages, page_size, err_flag) : -1;
     if (slot < 0) return;   // the whole block
     T* dst = cache + (size_t)slot * row;
@@ -67,16 +104,9 @@ __global__ void latent_prepare_kernel(const T* proj, const float* parts, int n_p
         const float v = proj_at<T>(proj, parts, n_parts, part_stride, base + c_col + i);
         dst[i] = from_f32<T>(__fmul_rn(__fmul_rn(v, rstd), wc[i]));
     }
-    const int half = rot / 2;
     for (int i = threadIdx.x; i < rope; i += blockDim.x) {
-        const float v = proj_at<T>(proj, parts, n_parts, part_stride, base + c_col + rank + i);
-        float o = v;
-        if (i < rot) {
-            const float other = proj_at<T>(proj, parts, n_parts, part_stride, base + c_col + rank + (i ^ 1));
-            const float c = cos_t[(size_t)t * half + (i >> 1)], s = sin_t[(size_t)t * half + (i >> 1)];
-            o = (i & 1) ? fmaf(v, c, __fmul_rn(other, s)) : fmaf(v, c, -__fmul_rn(other, s));
-        }
-        dst[rank + i] = from_f32<T>(o);
+        const size_t at0 = base + c_col + rank;
+        dst[rank + i] = from_f32<T>(turned([&](int j) { return proj_at<T>(proj, parts, n_parts, part_stride, at0 + j); }, i, rot, halves, ct, st));
     }
     for (int i = rank + rope + threadIdx.x; i < row; i += blockDim.x) dst[i] = from_f32<T>(0.f);
 }
@@ -85,21 +115,21 @@ PYRE_API int pyre_latent_prepare(const void* proj, const float* parts, int n_par
                                  int q_rank, int c_col, int rank, int rope, int rot, const float* wq, const float* wc,
                                  float eps, const float* cos_t, const float* sin_t, void* cq_out, void* cache,
                                  const int* slot_mapping, int n_tokens, int row, long long n_pages, int page_size,
-                                 int dtype, int* err_flag, cudaStream_t stream) {
+                                 int halves, void* qa, int qh_col, int nh, int dq, int dtype, int* err_flag, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if ((proj == nullptr) == (parts == nullptr) || rank <= 0 || rope < 0 || rot < 0 || rot > rope || rot % 2 ||
         row < rank + rope || (q_rank > 0 && (!wq || !cq_out)) || !wc || (cache && !slot_mapping) ||
-        (rot > 0 && (!cos_t || !sin_t)))
+        (rot > 0 && (!cos_t || !sin_t)) || (qa && (nh <= 0 || dq <= 0 || qh_col < 0 || (long long)qh_col + (long long)nh * (dq + rope) > W)))
         return PYRE_ERR_BAD_ARG;
-    const int threads = 128;
+    const int threads = qa && nh * (row - rank) >= 1024 ? 256 : 128;
     if (dtype == PYRE_BF16)
         pyre_launch(latent_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream, (const __nv_bfloat16*)proj, parts,
                     n_parts, part_stride, W, q_col, q_rank, c_col, rank, rope, rot, wq, wc, eps, cos_t, sin_t,
-                    (__nv_bfloat16*)cq_out, (__nv_bfloat16*)cache, slot_mapping, row, n_pages, page_size, err_flag);
+                    (__nv_bfloat16*)cq_out, (__nv_bfloat16*)cache, slot_mapping, row, n_pages, page_size, halves, (__nv_bfloat16*)qa, qh_col, nh, dq, err_flag);
     else if (dtype == PYRE_F32)
         pyre_launch(latent_prepare_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, (const float*)proj, parts, n_parts,
                     part_stride, W, q_col, q_rank, c_col, rank, rope, rot, wq, wc, eps, cos_t, sin_t, (float*)cq_out,
-                    (float*)cache, slot_mapping, row, n_pages, page_size, err_flag);
+                    (float*)cache, slot_mapping, row, n_pages, page_size, halves, (float*)qa, qh_col, nh, dq, err_flag);
     else return PYRE_ERR_BAD_ARG;
     PYRE_LAUNCH_CHECK();
     return 0;
@@ -112,7 +142,7 @@ PYRE_API int pyre_latent_prepare(const void* proj, const float* parts, int n_par
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void latent_rotate_q_kernel(const T* q, T* qa, const float* cos_t, const float* sin_t, int n_tokens, int nh,
-                                       int dq, int rope, int rot, int rank, int row) {
+                                       int dq, int rope, int rot, int rank, int row, int halves) {
     pdl_trigger();
     pdl_wait();
     const int tail = row - rank;
@@ -126,30 +156,24 @@ __global__ void latent_rotate_q_kernel(const T* q, T* qa, const float* cos_t, co
         float o = 0.f;
         if (i < rope) {
             const T* src = q + th * (size_t)(dq + rope) + dq;
-            const float v = to_f32<T>(src[i]);
-            o = v;
-            if (i < rot) {
-                const float other = to_f32<T>(src[i ^ 1]);
-                const float c = cos_t[(size_t)t * half + (i >> 1)], s = sin_t[(size_t)t * half + (i >> 1)];
-                o = (i & 1) ? fmaf(v, c, __fmul_rn(other, s)) : fmaf(v, c, -__fmul_rn(other, s));
-            }
+            o = turned([&](int j) { return to_f32<T>(src[j]); }, i, rot, halves, cos_t + (size_t)t * half, sin_t + (size_t)t * half);
         }
         qa[th * (size_t)row + rank + i] = from_f32<T>(o);
     }
 }
 
 PYRE_API int pyre_latent_rotate_q(const void* q, void* qa, const float* cos_t, const float* sin_t, int n_tokens, int nh, int dq,
-                                  int rope, int rot, int rank, int row, int dtype, cudaStream_t stream) {
+                                  int rope, int rot, int rank, int row, int halves, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || nh <= 0 || row <= rank) return 0;
     if (rot < 0 || rot > rope || rot % 2 || row < rank + rope || (rot > 0 && (!cos_t || !sin_t))) return PYRE_ERR_BAD_ARG;
     const long long total = (long long)n_tokens * nh * (row - rank);
     const int blocks = (int)min((long long)pyre_sm_count() * 8, ceil_div_ll(total, 256));
     if (dtype == PYRE_BF16)
         pyre_launch(latent_rotate_q_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)q, (__nv_bfloat16*)qa,
-                    cos_t, sin_t, n_tokens, nh, dq, rope, rot, rank, row);
+                    cos_t, sin_t, n_tokens, nh, dq, rope, rot, rank, row, halves);
     else if (dtype == PYRE_F32)
         pyre_launch(latent_rotate_q_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)q, (float*)qa, cos_t, sin_t,
-                    n_tokens, nh, dq, rope, rot, rank, row);
+                    n_tokens, nh, dq, rope, rot, rank, row, halves);
     else return PYRE_ERR_BAD_ARG;
     PYRE_LAUNCH_CHECK();
     return 0;
@@ -168,8 +192,8 @@ constexpr int LATENT_MAX_RANK = 512;
 template <typename T>
 __global__ void latent_attention_exact_kernel(const T* qa, const T* cache, T* out, const int* block_table, int bt_stride,
                                               const int* seq_of_token, const int* positions, int n_tokens, int nh, int rank,
-                                              int kd, int row, int page_size, int window, float scale, long long n_pages,
-                                              int* err_flag) {
+                                              int kd, int row, int page_size, int window, float scale, const float* head_sinks,
+                                              const T* gates, long long gate_stride, long long n_pages, int* err_flag) {
     extern __shared__ float q_smem[];   // [warps][kd]
     pdl_trigger();
     pdl_wait();
@@ -177,7 +201,7 @@ __global__ void latent_attention_exact_kernel(const T* qa, const T* cache, T* ou
     const int warps = blockDim.x >> 5;
     const long long item = (long long)blockIdx.x * warps + warp;
     if (item >= (long long)n_tokens * nh) return;
-    const int t = (int)(item / nh);
+    const int t = (int)(item / nh), head = (int)(item - (long long)t * nh);
     const int seq = seq_of_token[t];
     const int pos = positions[t];
     const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
@@ -239,7 +263,8 @@ __global__ void latent_attention_exact_kernel(const T* qa, const T* cache, T* ou
         for (int i = 0; i < OWN; ++i) acc[i] = fmaf(acc[i], alpha, part[i]);
         m = m_new;
     }
-    const float inv_l = 1.0f / l;
+    const float denom = head_sinks ? l + expf(head_sinks[head] - m) : l;
+    const float inv_l = head_gate_of<T>(gates, gate_stride, t, head) / denom;
     T* orow = out + (size_t)item * rank;
 #pragma unroll
     for (int i = 0; i < OWN; ++i) {
@@ -250,8 +275,8 @@ __global__ void latent_attention_exact_kernel(const T* qa, const T* cache, T* ou
 
 PYRE_API int pyre_latent_attention_exact(const void* qa, const void* cache, void* out, const int* block_table, int bt_stride,
                                          const int* seq_of_token, const int* positions, int n_tokens, int nh, int rank,
-                                         int rope, int row, int page_size, int window, float scale, int dtype,
-                                         long long n_pages, int* err_flag, cudaStream_t stream) {
+                                         int rope, int row, int page_size, int window, float scale, const float* head_sinks,
+                                         const void* gates, long long gate_stride, int dtype, long long n_pages, int* err_flag, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (rank <= 0 || rope < 0 || row < rank + rope || nh <= 0 || page_size <= 0) return PYRE_ERR_BAD_ARG;
     if (rank > LATENT_MAX_RANK) return PYRE_ERR_UNSUPPORTED;
@@ -264,11 +289,11 @@ PYRE_API int pyre_latent_attention_exact(const void* qa, const void* cache, void
     if (dtype == PYRE_F32)
         pyre_launch(latent_attention_exact_kernel<float>, dim3(blocks), dim3(warps * 32), smem, stream, (const float*)qa,
                     (const float*)cache, (float*)out, block_table, bt_stride, seq_of_token, positions, n_tokens, nh, rank, kd,
-                    row, page_size, window, scale, n_pages, err_flag);
+                    row, page_size, window, scale, head_sinks, (const float*)gates, gate_stride, n_pages, err_flag);
     else if (dtype == PYRE_BF16)
         pyre_launch(latent_attention_exact_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, stream, (const __nv_bfloat16*)qa,
                     (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, block_table, bt_stride, seq_of_token, positions, n_tokens,
-                    nh, rank, kd, row, page_size, window, scale, n_pages, err_flag);
+                    nh, rank, kd, row, page_size, window, scale, head_sinks, (const __nv_bfloat16*)gates, gate_stride, n_pages, err_flag);
     else return PYRE_ERR_BAD_ARG;
     PYRE_LAUNCH_CHECK();
     return 0;
@@ -314,7 +339,8 @@ __device__ __forceinline__ uint32_t lm_pack(float lo, float hi) {
 __global__ void __launch_bounds__(512) latent_attention_mma_kernel(
     const __nv_bfloat16* qa, const __nv_bfloat16* cache, __nv_bfloat16* out, float* part_o, float* part_ml,
     const int* block_table, int bt_stride, const int* cu_seqlens, const int* positions, int n_seqs, int nh, int hg, int rank,
-    int row, int page_size, int window, float scale_log2, int n_splits, int max_len, long long n_pages, int* err_flag) {
+    int row, int page_size, int window, float scale_log2, const float* head_sinks, const __nv_bfloat16* gates, long long gate_stride,
+    int n_splits, int max_len, long long n_pages, int* err_flag) {
     extern __shared__ __align__(16) unsigned char lm_smem[];
     __shared__ int item[3];
     pdl_trigger();
@@ -539,7 +565,8 @@ __global__ void __launch_bounds__(512) latent_attention_mma_kernel(
         const int tt = r / hg, hh = r - tt * hg;
         const size_t th = (size_t)(tok0 + tt) * nh + h0 + hh;
         if (n_splits == 1) {
-            const float inv = 1.0f / l[u];
+            const float sink = head_sinks ? exp2f(head_sinks[h0 + hh] * 1.4426950408889634f - m[u]) : 0.f;
+            const float inv = head_gate_of<__nv_bfloat16>(gates, gate_stride, tok0 + tt, h0 + hh) / (l[u] + sink);
 #pragma unroll
             for (int i = 0; i < LM_DV / 8; ++i)
 #pragma unroll
@@ -565,7 +592,8 @@ __global__ void __launch_bounds__(512) latent_attention_mma_kernel(
 }
 
 // out[t, h] = sum_s O_s 2^(m_s - m) / sum_s l_s 2^(m_s - m): the shares of one (token, head); maxima are base-2 exponents
-__global__ void latent_combine_kernel(const float* part_o, const float* part_ml, __nv_bfloat16* out, int n_splits, int rank) {
+__global__ void latent_combine_kernel(const float* part_o, const float* part_ml, __nv_bfloat16* out, int n_splits, int rank,
+                                      int nh, const float* head_sinks, const __nv_bfloat16* gates, long long gate_stride) {
     pdl_trigger();
     pdl_wait();
     const size_t th = blockIdx.x;
@@ -574,7 +602,9 @@ __global__ void latent_combine_kernel(const float* part_o, const float* part_ml,
     for (int s = 0; s < n_splits; ++s) mx = fmaxf(mx, ml[2 * s]);
     float denom = 0.f;
     for (int s = 0; s < n_splits; ++s) denom += ml[2 * s] == -INFINITY ? 0.f : ml[2 * s + 1] * exp2f(ml[2 * s] - mx);
-    const float inv = 1.0f / denom;
+    const int t = (int)(th / nh), head = (int)(th - (size_t)t * nh);
+    if (head_sinks) denom += exp2f(head_sinks[head] * 1.4426950408889634f - mx);
+    const float inv = head_gate_of<__nv_bfloat16>(gates, gate_stride, t, head) / denom;
     for (int c = threadIdx.x; c < rank; c += blockDim.x) {
         float acc = 0.f;
         for (int s = 0; s < n_splits; ++s)
@@ -588,8 +618,8 @@ __global__ void latent_combine_kernel(const float* part_o, const float* part_ml,
 PYRE_API int pyre_latent_attention_mma(const void* qa, const void* cache, void* out, float* part_o, float* part_ml,
                                        const int* block_table, int bt_stride, const int* cu_seqlens, const int* positions,
                                        int n_tokens, int n_seqs, int n_tiles, int nh, int rank, int row, int page_size, int window,
-                                       float scale, int n_splits, int max_len, long long n_pages, int* err_flag,
-                                       cudaStream_t stream) {
+                                       float scale, const float* head_sinks, const void* gates, long long gate_stride, int n_splits,
+                                       int max_len, long long n_pages, int* err_flag, cudaStream_t stream) {
     if (n_tokens <= 0 || n_tiles <= 0) return 0;
     if (rank <= 0 || row < rank || row % 16 || nh <= 0 || page_size <= 0 || n_splits < 1) return PYRE_ERR_BAD_ARG;
     if (n_splits > 1 && (!part_o || !part_ml)) return PYRE_ERR_BAD_ARG;
@@ -608,12 +638,12 @@ PYRE_API int pyre_latent_attention_mma(const void* qa, const void* cache, void* 
     const float scale_log2 = scale * 1.4426950408889634f;
     pyre_launch(latent_attention_mma_kernel, dim3(n_tiles, ceil_div(nh, hg), n_splits), dim3(128 * chunks), smem, stream,
                 (const __nv_bfloat16*)qa, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, part_o, part_ml, block_table, bt_stride,
-                cu_seqlens, positions, n_seqs, nh, hg, rank, row, page_size, window, scale_log2, n_splits, max_len, n_pages,
-                err_flag);
+                cu_seqlens, positions, n_seqs, nh, hg, rank, row, page_size, window, scale_log2, head_sinks, (const __nv_bfloat16*)gates,
+                gate_stride, n_splits, max_len, n_pages, err_flag);
     PYRE_LAUNCH_CHECK();
     if (n_splits > 1) {
         pyre_launch(latent_combine_kernel, dim3(n_tokens * nh), dim3(128), 0, stream, (const float*)part_o, (const float*)part_ml,
-                    (__nv_bfloat16*)out, n_splits, rank);
+                    (__nv_bfloat16*)out, n_splits, rank, nh, head_sinks, (const __nv_bfloat16*)gates, gate_stride);
         PYRE_LAUNCH_CHECK();
     }
     return 0;

@@ -310,8 +310,8 @@ def qkv_rope_write(qkv: torch.Tensor, bias: "torch.Tensor | None", cos: torch.Te
     return q_out
 
 
-def silu_mul(gate_up: torch.Tensor, out: "torch.Tensor | None" = None, block: int = 0) -> torch.Tensor:
-    """out[t, i] = silu(gate[t, i]) * up[t, i].  ``block == 0``: gate_up = [all gates | all ups];
+def silu_mul(gate_up: torch.Tensor, out: "torch.Tensor | None" = None, block: int = 0, kind: str = "silu") -> torch.Tensor:
+    """out[t, i] = act(gate[t, i]) * up[t, i], act ``silu`` or ``relu`` (``kind``).  ``block == 0``: gate_up = [all gates | all ups];
     ``block == n``: gates and ups alternate in blocks of n features (n gates, their n ups, ...)."""
     _check(gate_up, "gate_up", dim=2)
     T, two_i = gate_up.shape
@@ -322,7 +322,9 @@ def silu_mul(gate_up: torch.Tensor, out: "torch.Tensor | None" = None, block: in
         raise UnsupportedSize(f"silu_mul: blocks of {block} features do not tile {inter} features in steps of 8")
     if out is None:
         out = torch.empty((T, inter), dtype=gate_up.dtype, device=gate_up.device)
-    lib.call("pyre_silu_mul", gate_up.data_ptr(), out.data_ptr(), T, inter, int(block), _dt(gate_up.dtype), _stream())
+    if kind not in GATE_KINDS:
+        raise UnsupportedSize(f"gate activation {kind!r}: this kernel knows {sorted(GATE_KINDS)}")
+    lib.call("pyre_silu_mul", gate_up.data_ptr(), out.data_ptr(), T, inter, int(block), int(kind == "relu"), _dt(gate_up.dtype), _stream())
     return out
 
 
@@ -368,10 +370,11 @@ def sample(logits: torch.Tensor, temperature: "torch.Tensor | None" = None, seed
 def paged_attention_generic(q: torch.Tensor, cache_layer: torch.Tensor, block_table: torch.Tensor,
                             seq_of_token: torch.Tensor, positions: torch.Tensor, n_heads: int, n_kv_heads: int,
                             head_dim: int, scale: float, window: "int | None" = None,
-                            out: "torch.Tensor | None" = None, sink: "float | None" = None) -> torch.Tensor:
+                            out: "torch.Tensor | None" = None, sink: "float | None" = None, keep_first: int = 0) -> torch.Tensor:
     """Exact fp32-arithmetic attention of every query token over its sequence's pages.  ``sink``: the score of a
     sink that has no value: exp(sink) joins every softmax denominator (None: no sink; a float32 tensor [n_heads]: a
-    score per query head)."""
+    score per query head).  ``keep_first``: with a window, the sequence's first positions that stay visible however
+    far back they lie (here and in the other attention wrappers)."""
     _check(q, "q", dim=2)
     _check(cache_layer, "cache_layer", q.dtype, 5)
     _check(block_table, "block_table", torch.int32, 2)
@@ -391,7 +394,7 @@ def paged_attention_generic(q: torch.Tensor, cache_layer: torch.Tensor, block_ta
         out = torch.empty_like(q)
     lib.call("pyre_paged_attention_generic", q.data_ptr(), cache_layer.data_ptr(), out.data_ptr(),
              block_table.data_ptr(), block_table.stride(0), seq_of_token.data_ptr(), positions.data_ptr(), T,
-             n_heads, n_kv_heads, head_dim, page_size, int(window or 0), float(scale), _sink_args(sink, n_heads)[0], _sink_args(sink, n_heads)[1], _dt(q.dtype), cache_layer.shape[0],
+             n_heads, n_kv_heads, head_dim, page_size, int(window or 0), int(keep_first), float(scale), _sink_args(sink, n_heads)[0], _sink_args(sink, n_heads)[1], _dt(q.dtype), cache_layer.shape[0],
              device_error_flag(q.device).data_ptr(), _stream())
     return out
 
@@ -479,7 +482,7 @@ def paged_attention_mma(q: torch.Tensor, cache_layer: torch.Tensor, block_table:
                         n_kv_heads: int, head_dim: int, scale: float, window: "int | None" = None,
                         n_splits: int = 1, out: "torch.Tensor | None" = None,
                         scratch: "torch.Tensor | None" = None, max_len: int = 0, uniform_len: int = 0,
-                        sink: "float | None" = None) -> torch.Tensor:
+                        sink: "float | None" = None, keep_first: int = 0) -> torch.Tensor:
     """bfloat16 attention on the tensor cores over the block table (decode tokens and
     prompt portions alike); ``n_splits`` > 1 splits each sequence's keys over CTAs and needs
     ``T * nh * n_splits * (hd + 2)`` floats of scratch (allocated here if not given)."""
@@ -511,7 +514,7 @@ def paged_attention_mma(q: torch.Tensor, cache_layer: torch.Tensor, block_table:
             raise ValueError(f"scratch must be {need} contiguous floats")
     lib.call("pyre_paged_attention_mma", q.data_ptr(), cache_layer.data_ptr(), out.data_ptr(), _ptr(scratch),
              block_table.data_ptr(), block_table.stride(0), cu_seqlens.data_ptr(), positions.data_ptr(), T, n_seqs,
-             n_heads, n_kv_heads, head_dim, page_size, int(window or 0), float(scale), _sink_args(sink, n_heads)[0], _sink_args(sink, n_heads)[1], n_splits, int(max_len),
+             n_heads, n_kv_heads, head_dim, page_size, int(window or 0), int(keep_first), float(scale), _sink_args(sink, n_heads)[0], _sink_args(sink, n_heads)[1], n_splits, int(max_len),
              cache_layer.shape[0], int(uniform_len), device_error_flag(q.device).data_ptr(), _stream())
     return out
 
@@ -523,7 +526,7 @@ PREFILL_MIN_LEN = 32     # entries with at least this many tokens go to the prom
 def attention_prefill(q: torch.Tensor, cache_layer: torch.Tensor, block_table: torch.Tensor, cu_seqlens: torch.Tensor,
                       positions: torch.Tensor, n_seqs: int, n_long_tokens: int, n_heads: int, n_kv_heads: int,
                       head_dim: int, scale: float, window: "int | None", out: torch.Tensor,
-                      min_len: int = PREFILL_MIN_LEN, sink: "float | None" = None) -> torch.Tensor:
+                      min_len: int = PREFILL_MIN_LEN, sink: "float | None" = None, keep_first: int = 0) -> torch.Tensor:
     """bfloat16 attention of the entries with at least ``min_len`` tokens (64 queries of a head
     per CTA, keys and values tiled through shared memory); writes only those entries' rows of ``out``."""
     _check(q, "q", torch.bfloat16, 2)
@@ -543,7 +546,7 @@ def attention_prefill(q: torch.Tensor, cache_layer: torch.Tensor, block_table: t
         raise ValueError("out, cu_seqlens and positions do not match the batch")
     lib.call("pyre_attention_prefill", q.data_ptr(), cache_layer.data_ptr(), out.data_ptr(), block_table.data_ptr(),
              block_table.stride(0), cu_seqlens.data_ptr(), positions.data_ptr(), int(n_long_tokens), n_seqs, n_heads,
-             n_kv_heads, head_dim, page_size, int(window or 0), float(scale), _sink_args(sink, n_heads)[0], _sink_args(sink, n_heads)[1], int(min_len), cache_layer.shape[0],
+             n_kv_heads, head_dim, page_size, int(window or 0), int(keep_first), float(scale), _sink_args(sink, n_heads)[0], _sink_args(sink, n_heads)[1], int(min_len), cache_layer.shape[0],
              device_error_flag(q.device).data_ptr(), _stream())
     return out
 
@@ -580,7 +583,7 @@ def prefill_key_splits(n_items: int, mean_tiles: float, n_tokens: int, n_heads: 
 def attention_prefill_tc(q: torch.Tensor, cache_layer: torch.Tensor, block_table: torch.Tensor, cu_seqlens: torch.Tensor,
                          positions: torch.Tensor, n_seqs: int, n_long_tokens: int, n_heads: int, n_kv_heads: int,
                          head_dim: int, scale: float, window: "int | None", out: torch.Tensor, min_len: int,
-                         key_splits: int = 1, sink: "float | None" = None) -> torch.Tensor:
+                         key_splits: int = 1, sink: "float | None" = None, keep_first: int = 0) -> torch.Tensor:
     """bfloat16 attention of the entries with at least ``min_len`` tokens on the tcgen05 tensor
     cores (scores and output in tensor memory, Q/K/V tiles by TMA); writes only those entries' rows.
     ``key_splits`` > 1: that many CTAs share the keys of every (query tile, head); a second kernel combines them."""
@@ -606,14 +609,14 @@ def attention_prefill_tc(q: torch.Tensor, cache_layer: torch.Tensor, block_table
         part_ml = torch.empty((q.shape[0], n_heads, key_splits, 2), dtype=torch.float32, device=q.device)
     lib.call("pyre_attention_prefill_tc", q.data_ptr(), cache_layer.data_ptr(), out.data_ptr(), block_table.data_ptr(),
              block_table.stride(0), cu_seqlens.data_ptr(), positions.data_ptr(), q.shape[0], int(n_long_tokens), n_seqs,
-             n_heads, n_kv_heads, head_dim, page_size, cache_layer.shape[0], int(window or 0), float(scale), _sink_args(sink, n_heads)[0], _sink_args(sink, n_heads)[1], int(min_len),
+             n_heads, n_kv_heads, head_dim, page_size, cache_layer.shape[0], int(window or 0), int(keep_first), float(scale), _sink_args(sink, n_heads)[0], _sink_args(sink, n_heads)[1], int(min_len),
              key_splits, _ptr(part_o), _ptr(part_ml), device_error_flag(q.device).data_ptr(), _stream())
     return out
 
 
 def paged_attention_bf16(ctx, q: torch.Tensor, cache_layer: torch.Tensor, block_table: torch.Tensor, n_heads: int,
                          n_kv_heads: int, head_dim: int, scale: float, window: "int | None",
-                         sink: "float | None" = None) -> torch.Tensor:
+                         sink: "float | None" = None, keep_first: int = 0) -> torch.Tensor:
     """Attention of a whole step in bfloat16: entries with many tokens go to the
     prompt-portion kernel, the others (decoded tokens, short portions) to the split-KV kernel."""
     lens = ctx.cu_seqlens_host[1:] - ctx.cu_seqlens_host[:-1]
@@ -631,24 +634,24 @@ def paged_attention_bf16(ctx, q: torch.Tensor, cache_layer: torch.Tensor, block_
         # to the tile's last row
         keys = long_starts + long_lens / 2.0 + 64.0
         if window:
-            keys = keys.clip(max=window + 192.0)
+            keys = keys.clip(max=window + keep_first + 192.0)
         mean_tiles = float((keys / 64.0 * q_tiles).sum() / q_tiles.sum())
         key_splits = prefill_key_splits(int(q_tiles.sum()) * n_heads, mean_tiles, q.shape[0], n_heads, head_dim)
         attention_prefill_tc(q, cache_layer, block_table, ctx.cu_seqlens, ctx.positions, ctx.num_seqs, n_long, n_heads,
-                             n_kv_heads, head_dim, scale, window, out, min_len, key_splits, sink=sink)
+                             n_kv_heads, head_dim, scale, window, out, min_len, key_splits, sink=sink, keep_first=keep_first)
     elif n_long:
         attention_prefill(q, cache_layer, block_table, ctx.cu_seqlens, ctx.positions, ctx.num_seqs, n_long, n_heads,
-                          n_kv_heads, head_dim, scale, window, out, sink=sink)
+                          n_kv_heads, head_dim, scale, window, out, sink=sink, keep_first=keep_first)
     if n_short_seqs:
         n_short = ctx.num_tokens - n_long
         short_ctx = int((ctx.start_pos_host + lens)[~long_mask].max())
         tpg = max(1, 16 // min(n_heads // n_kv_heads, 16))
         groups = int((-(-lens[~long_mask] // tpg)).sum())
-        splits = attention_splits(n_short, n_short_seqs, n_heads, n_kv_heads, short_ctx, window, groups)
+        splits = attention_splits(n_short, n_short_seqs, n_heads, n_kv_heads, short_ctx, window and window + keep_first, groups)
         uniform = int(lens[0]) if not n_long and bool((lens == lens[0]).all()) else 0
         paged_attention_mma(q, cache_layer, block_table, ctx.cu_seqlens, ctx.positions, ctx.num_seqs, n_heads,
                             n_kv_heads, head_dim, scale, window, splits, out=out,
-                            max_len=min_len - 1 if n_long else 0, uniform_len=uniform, sink=sink)
+                            max_len=min_len - 1 if n_long else 0, uniform_len=uniform, sink=sink, keep_first=keep_first)
     return out
 
 
@@ -783,6 +786,7 @@ def tc_gemm_plan(M: int, N: int, K: int) -> tuple[bool, int, int]:
     return False, whole[1], whole[2]
 
 
+GATE_KINDS = {"silu": 1, "relu": 3}     # gates that a gated product applies in its epilogue: the kernel's argument
 GATED_BLOCK = 64     # gate and up rows of a fused feed-forward weight alternate in blocks of this many features
 
 
@@ -805,7 +809,7 @@ def _scale_fields(fx: "lib.GemmFix", x: "ScaledRows") -> None:
 
 
 def gemm_tc(x: "torch.Tensor | ScaledRows", w: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16,
-            plan: "tuple[bool, int, int] | None" = None, reduce: bool = True, gated: bool = False,
+            plan: "tuple[bool, int, int] | None" = None, reduce: bool = True, gated: "bool | str" = False,
             pair: "bool | None" = None, checked: bool = False) -> torch.Tensor:
     """y = x w^T on the tensor cores (tcgen05, TMEM accumulators, TMA-fed), bf16 in, fp32 accumulate.
 
@@ -814,7 +818,7 @@ def gemm_tc(x: "torch.Tensor | ScaledRows", w: torch.Tensor, out_dtype: torch.dt
     as ``PartialSums`` for a consumer kernel that adds them itself.
 
     ``gated``: w holds gate and up rows alternating in blocks of ``GATED_BLOCK`` features; the
-    result is silu(x gate^T) * (x up^T), [M, N / 2] bf16.  The activation runs in the product's
+    result is silu(x gate^T) * (x up^T), [M, N / 2] bf16 (``gated="relu"``: relu instead).  The activation runs in the product's
     epilogue (whole tiles, one split: the usual case in both orientations), otherwise after it.
 
     ``x`` may be ``ScaledRows``: the result rows are scaled by the tokens' 1/rms in the epilogue, before the
@@ -829,6 +833,9 @@ def gemm_tc(x: "torch.Tensor | ScaledRows", w: torch.Tensor, out_dtype: torch.dt
     if K != K2:
         raise ValueError(f"inner sizes differ: x is [{M}, {K}], w is [{N}, {K2}]")
     weights_as_rows, bn, splits = plan or tc_gemm_plan(M, N, K)
+    gate = "silu" if gated is True else gated
+    if gated and gate not in GATE_KINDS:
+        raise UnsupportedSize(f"gate activation {gate!r}: the product's epilogue knows {sorted(GATE_KINDS)}")
     if gated and plan is None and M == 128 and N % 256 == 0:
         # exactly 128 tokens: 58.6 us with the weights on the rows, 52.4 so; with 72-120 tokens (a tile of token rows
         # that is not full) this orientation takes 66 us and the other 54-58
@@ -854,15 +861,15 @@ def gemm_tc(x: "torch.Tensor | ScaledRows", w: torch.Tensor, out_dtype: torch.dt
         if not weights_as_rows and bn == 256 and splits == 1 and N % 256 == 0:
             out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
             lib.call("pyre_gemm_tc", x.data_ptr(), M, x.stride(0), w.data_ptr(), N, w.stride(0), K, out.data_ptr(), 0,
-                     N // 2, 1, 0, 1, bn, 0, 1, pair, err.data_ptr(), fx, _stream())
+                     N // 2, 1, 0, 1, bn, 0, GATE_KINDS[gate], pair, err.data_ptr(), fx, _stream())
             return out
         if weights_as_rows and bn <= 128 and splits == 1 and N % 128 == 0:
             out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
             lib.call("pyre_gemm_tc", w.data_ptr(), N, w.stride(0), x.data_ptr(), M, x.stride(0), K, out.data_ptr(), 0,
-                     1, N // 2, 0, 1, bn, 1, 1, 0, err.data_ptr(), fx, _stream())
+                     1, N // 2, 0, 1, bn, 1, GATE_KINDS[gate], 0, err.data_ptr(), fx, _stream())
             return out
         return silu_mul(gemm_tc(scaled if scaled is not None else x, w, torch.bfloat16, (weights_as_rows, bn, splits), pair=bool(pair)),
-                        block=GATED_BLOCK)
+                        block=GATED_BLOCK, kind=gate)
     if splits == 1 and reduce:
         out = torch.empty((M, N), dtype=out_dtype, device=x.device)
         target, split_stride = out, 0
@@ -1061,14 +1068,14 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor, block: int = GATED_
     return torch.stack([gate.view(inter // block, block, K), up.view(inter // block, block, K)], dim=1).reshape(2 * inter, K).contiguous()
 
 
-def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, interleaved: bool) -> torch.Tensor:
-    """silu(x gate^T) * (x up^T) for the stacked weight of a gated feed-forward: [gates | ups] rows, or
+def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, interleaved: bool, kind: str = "silu") -> torch.Tensor:
+    """act(x gate^T) * (x up^T), act silu or relu (``kind``), for the stacked weight of a gated feed-forward: [gates | ups] rows, or
     (``interleaved``) blocks of ``GATED_BLOCK`` gate rows and up rows in turn, which lets the bfloat16
     tensor-core product apply the activation in its epilogue."""
     rows = x.rows if isinstance(x, ScaledRows) else x
     if interleaved and x.dtype == torch.bfloat16 and USE_TC_GEMM and tc_gemm_supported(rows, w_gate_up):
-        return gemm_tc(x, w_gate_up, torch.bfloat16, gated=True, checked=True)
-    return silu_mul(linear(x, w_gate_up), block=GATED_BLOCK if interleaved else 0)
+        return gemm_tc(x, w_gate_up, torch.bfloat16, gated=kind, checked=True)
+    return silu_mul(linear(x, w_gate_up), block=GATED_BLOCK if interleaved else 0, kind=kind)
 
 
 # ---------------------------------------------------------------------------------- layers that are no pre-norm block
@@ -1153,7 +1160,8 @@ def qk_norm_rope_write(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
                        k_weight: "torch.Tensor | None", eps: float, cos: "torch.Tensor | None", sin: "torch.Tensor | None",
                        cache_layer: "torch.Tensor | None", slot_mapping: "torch.Tensor | None", n_heads: int,
                        n_kv_heads: int, qk_dim: int, v_dim: int, row_dim: int, rotary_dim: int, page_size: int,
-                       v_cos: "torch.Tensor | None" = None, v_sin: "torch.Tensor | None" = None) -> torch.Tensor:
+                       v_cos: "torch.Tensor | None" = None, v_sin: "torch.Tensor | None" = None, neighbours: bool = False,
+                       post_norm: bool = False) -> torch.Tensor:
     """Per-head RMS norm of queries and keys (weights [qk_dim], shared by the heads; None: no norm), rotation of
     the first ``rotary_dim`` dims of each head, and the paged write, for heads whose query/key size ``qk_dim`` and
     value size ``v_dim`` differ from the cache's row size ``row_dim`` (the rest of a row is zero).
@@ -1161,6 +1169,8 @@ def qk_norm_rope_write(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
     ``cache_layer`` None: nothing is stored and no keys or values are read from ``proj`` (a layer that reads another
     layer's cache).  ``v_cos`` / ``v_sin`` [T, v_dim / 2]: the values are turned too, over all their dims in
     half-split pairs, by these tables, and cached so (``head_gate`` turns a head's weighted sum back).
+    ``neighbours``: the rotation's pairs are (2i, 2i + 1) instead of (i, i + rotary_dim / 2).  ``post_norm``: after the
+    rotation every query and key head is divided by its root mean square over ``qk_dim`` (with ``eps``, no weight).
     Returns the queries [T, n_heads * row_dim]."""
     _check(proj, "proj", dim=2)
     T, W = proj.shape
@@ -1205,7 +1215,7 @@ def qk_norm_rope_write(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
     lib.call("pyre_qk_norm_rope_write", proj.data_ptr(), W, int(q_col), int(k_col) if write else -1, int(v_col) if write else -1,
              _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(cos) if rotary_dim else None, _ptr(sin) if rotary_dim else None,
              _ptr(v_cos), _ptr(v_sin), q_out.data_ptr(), _ptr(cache_layer), _ptr(slot_mapping) if write else None, T, n_heads,
-             n_kv_heads, qk_dim, v_dim, D, rotary_dim, page_size, _dt(proj.dtype),
+             n_kv_heads, qk_dim, v_dim, D, rotary_dim, int(bool(neighbours)), int(bool(post_norm)), page_size, _dt(proj.dtype),
              cache_layer.shape[0] if write else 0, device_error_flag(proj.device).data_ptr(), _stream())
     return q_out
 
@@ -1425,7 +1435,9 @@ class ScaledSum:
     def __init__(self, terms, dtype: torch.dtype):
         if not 1 <= len(terms) <= 2:
             raise ValueError("a ScaledSum holds one or two terms")
-        self.terms = [(materialize(t) if isinstance(t, (DeferredProduct, ScaledRows)) else t, s) for t, s in terms]
+        # a product not launched yet runs plainly; its fp32 partial sums (K split) stay unrounded
+        terms = [(t.partials() if isinstance(t, DeferredProduct) else t, s) for t, s in terms]
+        self.terms = [(materialize(t) if isinstance(t, ScaledRows) else t, s) for t, s in terms]
         self.dtype = dtype
 
     @property
@@ -1468,12 +1480,14 @@ class ScaledSum:
 
 def add_layernorm(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSums | None", weight: torch.Tensor, eps: float,
                   out_dtype: torch.dtype, rows: "torch.Tensor | None" = None, update_x: bool = True,
-                  act_dtype: "torch.dtype | None" = None, bias: "torch.Tensor | None" = None) -> torch.Tensor:
+                  act_dtype: "torch.dtype | None" = None, bias: "torch.Tensor | None" = None,
+                  weight2: "torch.Tensor | None" = None):
     """out[r] = layernorm(x[src] + delta[src]) * weight (+ bias) with src = rows[r] (or r): the mean is taken off, the
     variance is the mean squared deviation; ``bias`` fp32 [H] or None.  ``x`` is the fp32 residual stream [T, H]; with ``update_x``
     (and no ``rows``) the sum is written back to it.  ``delta``: a ``ScaledSum`` (each term times its gain), a
     plain branch output or partial sums (gain one), or None.  ``out_dtype`` float32 with bfloat16 activations
-    (``act_dtype``) gives the normalised rows in fp32: a norm applied to the stream itself."""
+    (``act_dtype``) gives the normalised rows in fp32: a norm applied to the stream itself.  ``weight2``: a second norm
+    of the SAME rows (no bias) written in the same pass; the result is then the pair."""
     _check(x, "x", torch.float32, 2)
     _check(weight, "weight", torch.float32, 1)
     T, H = x.shape
@@ -1484,6 +1498,10 @@ def add_layernorm(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSum
         _check(bias, "bias", torch.float32, 1)
         if bias.shape[0] != H:
             raise ValueError(f"norm bias has {bias.shape[0]} entries, rows have {H}")
+    if weight2 is not None:
+        _check(weight2, "weight2", torch.float32, 1)
+        if weight2.shape[0] != H or out_dtype != act:
+            raise ValueError("a second norm has as many entries as the rows and writes activations")
     if H * 4 > 48 * 1024:
         raise UnsupportedSize(f"layer norm over rows of {H}: the kernel holds a row of at most 12,288 in shared memory")
     if delta is not None and not isinstance(delta, ScaledSum):
@@ -1498,11 +1516,43 @@ def add_layernorm(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSum
         _check(rows, "rows", torch.int32, 1)
         n_rows, update_x = rows.shape[0], False
     out = torch.empty((n_rows, H), dtype=out_dtype, device=x.device)
+    out2 = torch.empty((n_rows, H), dtype=out_dtype, device=x.device) if weight2 is not None else None
     a = args
-    lib.call("pyre_add_layernorm", x.data_ptr(), a[0], a[1], a[2], a[3], a[4], a[5], a[6], a[7], stride, weight.data_ptr(), _ptr(bias), out.data_ptr(),
+    lib.call("pyre_add_layernorm", x.data_ptr(), a[0], a[1], a[2], a[3], a[4], a[5], a[6], a[7], stride, weight.data_ptr(), _ptr(bias), _ptr(weight2), out.data_ptr(), _ptr(out2),
              int(out_dtype == torch.float32 and act != torch.float32), _ptr(rows), n_rows, H, float(eps),
              int(bool(update_x and delta is not None)), _dt(act), _stream())
+    return out if out2 is None else (out, out2)
+
+
+def stream_rows(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSums | None", dtype: torch.dtype) -> torch.Tensor:
+    """The fp32 stream ``x`` [T, H] with ``delta`` (as in ``add_layernorm``) added, as activations for a product that
+    reads the stream itself: a new tensor in ``dtype``; ``x`` stays as it is."""
+    _check(x, "x", torch.float32, 2)
+    T, H = x.shape
+    if delta is not None and not isinstance(delta, ScaledSum):
+        delta = ScaledSum([(delta, _ones(H, x.device))], dtype)
+    args, stride = ([None, None, 0, None] * 2, 0)
+    if delta is not None:
+        if delta.shape != (T, H):
+            raise ValueError(f"delta shape {delta.shape} != x shape {(T, H)}")
+        args, stride = delta._args(dtype)
+    out = torch.empty((T, H), dtype=dtype, device=x.device)
+    a = args
+    lib.call("pyre_stream_rows", x.data_ptr(), a[0], a[1], a[2], a[3], a[4], a[5], a[6], a[7], stride, out.data_ptr(), T, H,
+             _dt(dtype), _stream())
     return out
+
+
+def stream_set(x: torch.Tensor, base: torch.Tensor, product: "torch.Tensor | PartialSums") -> None:
+    """x = base + product in place on the fp32 stream ``x``: the stream set anew from an fp32 product (a tensor, or the
+    partial sums of one) and a fixed fp32 term of the same shape."""
+    _check(x, "x", torch.float32, 2)
+    _check(base, "base", torch.float32, 2)
+    parts = product.parts if isinstance(product, PartialSums) else product.unsqueeze(0)
+    _check(parts, "product", torch.float32, 3)
+    if base.shape != x.shape or tuple(parts.shape[1:]) != tuple(x.shape):
+        raise ValueError(f"stream {tuple(x.shape)}, base {tuple(base.shape)} and product {tuple(parts.shape[1:])} differ")
+    lib.call("pyre_stream_set", x.data_ptr(), base.data_ptr(), parts.data_ptr(), parts.shape[0], x.numel(), x.numel(), _stream())
 
 
 _ones_cache: dict = {}
@@ -1516,16 +1566,19 @@ def _ones(n: int, device) -> torch.Tensor:
     return t
 
 
+MUL_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu": 2}
+
+
 def act_mul(gate_up: torch.Tensor, kind: str) -> torch.Tensor:
-    """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i] for rows [gates | ups]; ``kind`` as in ``ACTIVATIONS``."""
+    """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i] for rows [gates | ups]; ``kind`` as in ``MUL_ACTIVATIONS``."""
     _check(gate_up, "gate_up", dim=2)
-    if kind not in ACTIVATIONS:
-        raise UnsupportedSize(f"activation {kind!r}: implemented are {sorted(ACTIVATIONS)}")
+    if kind not in MUL_ACTIVATIONS:
+        raise UnsupportedSize(f"activation {kind!r}: implemented are {sorted(MUL_ACTIVATIONS)}")
     T, two_i = gate_up.shape
     if two_i % 2:
         raise ValueError("gate_up must have an even number of columns")
     out = torch.empty((T, two_i // 2), dtype=gate_up.dtype, device=gate_up.device)
-    lib.call("pyre_act_mul", gate_up.data_ptr(), out.data_ptr(), T, two_i // 2, ACTIVATIONS[kind], _dt(gate_up.dtype), _stream())
+    lib.call("pyre_act_mul", gate_up.data_ptr(), out.data_ptr(), T, two_i // 2, MUL_ACTIVATIONS[kind], _dt(gate_up.dtype), _stream())
     return out
 
 
@@ -1536,12 +1589,15 @@ LATENT_MAX_RANK = 512
 def latent_prepare(proj: "torch.Tensor | PartialSums", q_col: int, q_rank: int, c_col: int, rank: int, rope: int, rot: int,
                    wq: "torch.Tensor | None", wc: torch.Tensor, eps: float, cos: "torch.Tensor | None", sin: "torch.Tensor | None",
                    cache_layer: "torch.Tensor | None", slot_mapping: "torch.Tensor | None", page_size: int,
-                   act_dtype: torch.dtype) -> "torch.Tensor | None":
+                   act_dtype: torch.dtype, halves: bool = False, q_out: "torch.Tensor | None" = None, qh_col: int = 0,
+                   dq: int = 0) -> "torch.Tensor | None":
     """From a token's down-projections ``proj`` [T, W] (columns ``q_col``: the query latent of ``q_rank`` entries,
     0 for none; ``c_col``: the key/value latent of ``rank`` entries followed by the shared key part of ``rope``):
     returns rmsnorm(query latent) * wq [T, q_rank] and writes [rmsnorm(latent) * wc | rotate(key part)] to the
-    token's row of ``cache_layer`` [pages, 1, 1, page_size, row].  The rotation turns neighbouring pairs of the
-    first ``rot`` entries by the angles whose cos/sin are given [T, rot / 2]."""
+    token's row of ``cache_layer`` [pages, 1, 1, page_size, row].  The rotation turns neighbouring pairs (``halves``:
+    the pairs (i, i + rot / 2)) of the first ``rot`` entries by the angles whose cos/sin are given [T, rot / 2].
+    ``q_out`` [T, heads, row]: the queries lie in the same projection rows (head h's at ``qh_col + h (dq + rope)``, its
+    rotated part last); their rotated parts are turned and written to ``q_out[t, h, rank:]`` (zeros beyond ``rope``)."""
     parts, n_parts, stride, tensor = None, 0, 0, None
     if isinstance(proj, PartialSums):
         parts, n_parts, stride = proj.parts, proj.n, proj.parts[0].numel()
@@ -1571,15 +1627,23 @@ def latent_prepare(proj: "torch.Tensor | PartialSums", q_col: int, q_rank: int, 
         _check(slot_mapping, "slot_mapping", torch.int32, 1)
         if slot_mapping.shape[0] != T:
             raise ValueError("slot_mapping must have one entry per token")
+    nh = 0
+    if q_out is not None:
+        _check(q_out, "q_out", act_dtype, 3)
+        nh = q_out.shape[1]
+        if q_out.shape[0] != T or qh_col < 0 or qh_col + nh * (dq + rope) > W or (row and q_out.shape[2] != row):
+            raise ValueError("the queries do not lie inside the projection row or do not match the cache's rows")
+        row = row or q_out.shape[2]
     cq = torch.empty((T, q_rank), dtype=act_dtype, device=device) if q_rank else None
     lib.call("pyre_latent_prepare", _ptr(tensor), _ptr(parts), n_parts, stride, W, int(q_col), int(q_rank), int(c_col), int(rank),
              int(rope), int(rot), _ptr(wq), wc.data_ptr(), float(eps), _ptr(cos) if rot else None, _ptr(sin) if rot else None,
              _ptr(cq), _ptr(cache_layer), _ptr(slot_mapping) if cache_layer is not None else None, T, max(row, rank + rope),
-             n_pages, int(page_size), _dt(act_dtype), device_error_flag(device).data_ptr(), _stream())
+             n_pages, int(page_size), int(bool(halves)), _ptr(q_out), int(qh_col), nh, int(dq), _dt(act_dtype), device_error_flag(device).data_ptr(), _stream())
     return cq
 
 
-def latent_rotate_q(q: torch.Tensor, qa: torch.Tensor, cos, sin, n_heads: int, dq: int, rope: int, rot: int, rank: int) -> None:
+def latent_rotate_q(q: torch.Tensor, qa: torch.Tensor, cos, sin, n_heads: int, dq: int, rope: int, rot: int, rank: int,
+                    halves: bool = False) -> None:
     """qa[t, h, rank + i] = rotate(q[t, h, dq + i]) for i < rope (zeros beyond): the rotated tail of the absorbed
     query rows ``qa`` [T, n_heads, row]; ``q`` [T, n_heads * (dq + rope)]."""
     _check(q, "q", dim=2)
@@ -1588,14 +1652,32 @@ def latent_rotate_q(q: torch.Tensor, qa: torch.Tensor, cos, sin, n_heads: int, d
     if q.shape[1] != n_heads * (dq + rope) or tuple(qa.shape[:2]) != (T, n_heads) or row < rank + rope:
         raise ValueError("q or qa do not match the head sizes")
     lib.call("pyre_latent_rotate_q", q.data_ptr(), qa.data_ptr(), _ptr(cos) if rot else None, _ptr(sin) if rot else None, T,
-             n_heads, int(dq), int(rope), int(rot), int(rank), row, _dt(q.dtype), _stream())
+             n_heads, int(dq), int(rope), int(rot), int(rank), row, int(bool(halves)), _dt(q.dtype), _stream())
+
+
+def _latent_extras(qa: torch.Tensor, sink, gate) -> tuple:
+    """(sink pointer, gate pointer, gate row stride) as the latent attention kernels take them."""
+    T, nh, _ = qa.shape
+    if sink is not None:
+        _check(sink, "sink", torch.float32, 1)
+        if sink.shape[0] != nh:
+            raise ValueError(f"{sink.shape[0]} sink scores for {nh} heads")
+    if gate is None:
+        return _ptr(sink), None, 0
+    g, col = gate
+    _check(g, "gate", qa.dtype, 2)
+    if g.shape[0] != T or col < 0 or col + nh > g.shape[1]:
+        raise ValueError("the gates do not lie inside the projection row")
+    return _ptr(sink), g.data_ptr() + col * g.element_size(), g.stride(0)
 
 
 def latent_attention_exact(qa: torch.Tensor, cache_layer: torch.Tensor, block_table: torch.Tensor, seq_of_token: torch.Tensor,
-                           positions: torch.Tensor, rank: int, rope: int, scale: float, window: "int | None") -> torch.Tensor:
+                           positions: torch.Tensor, rank: int, rope: int, scale: float, window: "int | None",
+                           sink: "torch.Tensor | None" = None, gate: "tuple | None" = None) -> torch.Tensor:
     """Exact fp32-arithmetic attention of absorbed queries ``qa`` [T, nh, row] over the latent rows of their
     sequences' pages: score = qa . row[: rank + rope] * scale, output = sum of probabilities times row[: rank];
-    returns [T, nh, rank]."""
+    returns [T, nh, rank].  ``sink``: fp32 scores [nh] of a sink without a value that joins each head's denominator.
+    ``gate`` (tensor [T, W] in the activation dtype, column g): head h's result is multiplied by sigmoid(tensor[t, g + h])."""
     _check(qa, "qa", dim=3)
     _check(cache_layer, "cache_layer", qa.dtype, 5)
     _check(block_table, "block_table", torch.int32, 2)
@@ -1608,9 +1690,11 @@ def latent_attention_exact(qa: torch.Tensor, cache_layer: torch.Tensor, block_ta
     if rank > LATENT_MAX_RANK or (rank + rope) * 16 > 48 * 1024:
         raise UnsupportedSize(f"latent rows of {rank} + {rope}: the kernel takes latents up to {LATENT_MAX_RANK}")
     out = torch.empty((T, nh, rank), dtype=qa.dtype, device=qa.device)
+    sink_ptr, gate_ptr, gate_stride = _latent_extras(qa, sink, gate)
     lib.call("pyre_latent_attention_exact", qa.data_ptr(), cache_layer.data_ptr(), out.data_ptr(), block_table.data_ptr(),
              block_table.stride(0), seq_of_token.data_ptr(), positions.data_ptr(), T, nh, int(rank), int(rope), row, page_size,
-             int(window or 0), float(scale), _dt(qa.dtype), cache_layer.shape[0], device_error_flag(qa.device).data_ptr(), _stream())
+             int(window or 0), float(scale), sink_ptr, gate_ptr, gate_stride, _dt(qa.dtype), cache_layer.shape[0],
+             device_error_flag(qa.device).data_ptr(), _stream())
     return out
 
 
@@ -1625,11 +1709,14 @@ def _grouped_mma_ok(x: torch.Tensor, w: torch.Tensor, x_row_stride: int, x_group
 
 
 def headwise_linear(x: torch.Tensor, w: torch.Tensor, out: "torch.Tensor | None" = None) -> torch.Tensor:
-    """out[t, h, :N] = x[t, h, :K] . w[h]^T for ``x`` [T, H, >= K] and ``w`` [H, N, K]: a product per head.  ``out``
-    [T, H, >= N] may be given (rows wider than N keep their other columns); else [T, H, N] is returned."""
-    _check(x, "x", dim=3)
+    """out[t, h, :N] = x[t, h, :K] . w[h]^T for ``x`` [T, H, >= K] and ``w`` [H, N, K]: a product per head.  ``x`` may be
+    a view with strides of its own over tokens and heads (the heads inside a wider projection row).  ``out`` [T, H, >= N] may be given (rows wider than N keep their other columns); else [T, H, N] is returned."""
+    if not x.is_cuda or x.dim() != 3 or x.stride(2) != 1:
+        raise ValueError("x is [T, H, K] with contiguous entries per head")
+    require_current_device(x.device, "x")
     _check(w, "w", x.dtype, 3)
     T, H, xs = x.shape
+    row_stride, head_stride = x.stride(0), x.stride(1)
     _, N, K = w.shape
     if w.shape[0] != H or xs < K:
         raise ValueError(f"x {tuple(x.shape)} and w {tuple(w.shape)} do not match head by head")
@@ -1639,8 +1726,8 @@ def headwise_linear(x: torch.Tensor, w: torch.Tensor, out: "torch.Tensor | None"
         _check(out, "out", x.dtype, 3)
         if tuple(out.shape[:2]) != (T, H) or out.shape[2] < N:
             raise ValueError("out does not match the heads")
-    lib.call("pyre_grouped_linear", x.data_ptr(), H * xs, xs, w.data_ptr(), N * K, out.data_ptr(), H * out.shape[2], out.shape[2],
-             None, None, None, T, N, K, H, 0, 0, _dt(x.dtype), _grouped_mma_ok(x, w, H * xs, xs, K), _stream())
+    lib.call("pyre_grouped_linear", x.data_ptr(), row_stride, head_stride, w.data_ptr(), N * K, out.data_ptr(), H * out.shape[2], out.shape[2],
+             None, None, None, T, N, K, H, 0, 0, _dt(x.dtype), _grouped_mma_ok(x, w, row_stride, head_stride, K), _stream())
     return out
 
 
@@ -1838,10 +1925,11 @@ def latent_attention_splits(n_tiles: int, n_heads: int, rank: int, span: int, ro
 
 def latent_attention_mma(qa: torch.Tensor, cache_layer: torch.Tensor, block_table: torch.Tensor, cu_seqlens: torch.Tensor,
                          positions: torch.Tensor, n_tiles: int, rank: int, scale: float, window: "int | None", n_splits: int = 1,
-                         max_len: int = 0, out: "torch.Tensor | None" = None) -> torch.Tensor:
+                         max_len: int = 0, out: "torch.Tensor | None" = None, sink: "torch.Tensor | None" = None,
+                         gate: "tuple | None" = None) -> torch.Tensor:
     """bfloat16 attention of absorbed queries ``qa`` [T, nh, row] over latent rows on the tensor cores; ``n_tiles``:
     an upper bound of the row tiles (64 // min(nh, 64) tokens each) of the entries taken (``max_len`` > 0: those of
-    at most that many tokens).  Returns [T, nh, rank]."""
+    at most that many tokens).  ``sink`` and ``gate`` as in ``latent_attention_exact``.  Returns [T, nh, rank]."""
     _check(qa, "qa", torch.bfloat16, 3)
     _check(cache_layer, "cache_layer", torch.bfloat16, 5)
     _check(block_table, "block_table", torch.int32, 2)
@@ -1857,30 +1945,31 @@ def latent_attention_mma(qa: torch.Tensor, cache_layer: torch.Tensor, block_tabl
     if out is None:
         out = torch.empty((T, nh, rank), dtype=qa.dtype, device=qa.device)
     n_splits = int(n_splits)
+    sink_ptr, gate_ptr, gate_stride = _latent_extras(qa, sink, gate)
     part_o = part_ml = None
     if n_splits > 1:
         part_o = torch.empty((T, nh, n_splits, rank), dtype=torch.float32, device=qa.device)
         part_ml = torch.empty((T, nh, n_splits, 2), dtype=torch.float32, device=qa.device)
     lib.call("pyre_latent_attention_mma", qa.data_ptr(), cache_layer.data_ptr(), out.data_ptr(), _ptr(part_o), _ptr(part_ml),
              block_table.data_ptr(), block_table.stride(0), cu_seqlens.data_ptr(), positions.data_ptr(), T, n_seqs, int(n_tiles), nh,
-             int(rank), row, page_size, int(window or 0), float(scale), n_splits, int(max_len), cache_layer.shape[0],
+             int(rank), row, page_size, int(window or 0), float(scale), sink_ptr, gate_ptr, gate_stride, n_splits, int(max_len), cache_layer.shape[0],
              device_error_flag(qa.device).data_ptr(), _stream())
     return out
 
 
 def latent_attention(ctx, qa: torch.Tensor, cache_layer: torch.Tensor, block_table: torch.Tensor, rank: int, rope: int,
-                     scale: float, window: "int | None") -> torch.Tensor:
+                     scale: float, window: "int | None", sink: "torch.Tensor | None" = None, gate: "tuple | None" = None) -> torch.Tensor:
     """Attention of a whole step's absorbed queries over their sequences' latent rows; [T, nh, rank].  bfloat16 with
     rows of a multiple of 16 entries: the tensor-core kernel; everything else: the exact one."""
     T, nh, row = qa.shape
     if not latent_mma_ok(qa.dtype, row):
-        return latent_attention_exact(qa, cache_layer, block_table, ctx.seq_of_token, ctx.positions, rank, rope, scale, window)
+        return latent_attention_exact(qa, cache_layer, block_table, ctx.seq_of_token, ctx.positions, rank, rope, scale, window, sink=sink, gate=gate)
     tq = LATENT_MMA_ROWS // min(nh, LATENT_MMA_ROWS)
     lens = ctx.cu_seqlens_host[1:] - ctx.cu_seqlens_host[:-1]
     n_tiles = int((-(-lens // tq)).sum())
     span = ctx.max_context if not window else min(ctx.max_context, window + tq)
     return latent_attention_mma(qa, cache_layer, block_table, ctx.cu_seqlens, ctx.positions, n_tiles, rank, scale, window,
-                                latent_attention_splits(n_tiles, nh, rank, span, row))
+                                latent_attention_splits(n_tiles, nh, rank, span, row), sink=sink, gate=gate)
 
 
 # ---------------------------------------------------------------------------------- short histories and recurrent states

@@ -34,14 +34,17 @@ def _instantiate(spec: ModelSpec, dtype, device):
     embed = make_part("embed", spec.embed, dtype, device)
     blocks = [make_part("block", b, dtype, device) for b in spec.blocks]
     tail = make_part("tail", spec.tail, dtype, device)
-    return embed, blocks, tail
+    streams = {name: make_part("stream", part, dtype, device) for name, (part, _prefix) in spec.streams.items()}
+    return embed, blocks, tail, streams
 
 
 def tensor_table(spec: ModelSpec) -> dict[str, TensorSpec]:
     """Checkpoint name -> TensorSpec for every tensor of the model, in a fixed order
-    (embedding, layers in order, final norm, head)."""
-    embed, blocks, tail = _instantiate(spec, torch.float32, "meta")
+    (embedding, the model's stream parts, layers in order, final norm, head)."""
+    embed, blocks, tail, streams = _instantiate(spec, torch.float32, "meta")
     table = collect_tensors(embed, spec.embed_prefix)
+    for name, part in streams.items():
+        table.update(collect_tensors(part, spec.streams[name][1]))
     for i, b in enumerate(blocks):
         table.update(collect_tensors(b, spec.block_prefix.format(i=i)))
     table.update(collect_tensors(tail, spec.tail_prefix))
@@ -55,7 +58,7 @@ class Model:
         self.spec = spec
         self.dtype = dtype
         self.device = torch.device(device)
-        self.embed, self.blocks, self.tail = _instantiate(spec, dtype, self.device)
+        self.embed, self.blocks, self.tail, self.streams = _instantiate(spec, dtype, self.device)
         self.vocab_size = spec.vocab_size
         self.calls, self.kv_groups, self.state_groups = self._bind_schedule()
         self.loaded = False
@@ -63,8 +66,8 @@ class Model:
         self.graph_safe = all(all_graph_safe(p) for p in self.parts())
 
     def parts(self) -> list:
-        """The top-level parts: embedding, blocks, tail."""
-        return [self.embed, *self.blocks, self.tail]
+        """The top-level parts: embedding, the model's stream parts, blocks, tail."""
+        return [self.embed, *self.streams.values(), *self.blocks, self.tail]
 
     # ------------------------------------------------------------------ schedule
     def _bind_schedule(self):
@@ -111,7 +114,7 @@ class Model:
                 st_layer = st_layers[st_group]
                 st_layers[st_group] += 1
             calls.append(BoundCall(n, call.block, kv_group, kv_layer, call.write, st_group, st_layer, bool(call.add_embedding),
-                                   tuple(call.add_vector) if call.add_vector is not None else None))
+                                   tuple(call.add_vector) if call.add_vector is not None else None, call.before))
         kv_groups = [KVGroup(s, n) for s, n in zip(kv_specs, kv_layers)]
         state_groups = [StateGroup(s, n) for s, n in zip(st_specs, st_layers)]
         return calls, kv_groups, state_groups
@@ -122,6 +125,8 @@ class Model:
 
     def _bind(self, tensors) -> None:
         load_part(self.embed, tensors, self.spec.embed_prefix)
+        for name, part in self.streams.items():
+            load_part(part, tensors, self.spec.streams[name][1])
         for i, b in enumerate(self.blocks):
             prefix = self.spec.block_prefix.format(i=i)
             load_part(b, tensors, prefix)
@@ -156,7 +161,12 @@ class Model:
         pending = None
         # blocks update the stream in place: an entry that adds the embedding's output again needs a copy of it
         fed = x.clone() if any(call.add_embedding for call in self.calls) else None
+        for part in self.streams.values():
+            if hasattr(part, "begin"):
+                part.begin(ctx, x)
         for call in self.calls:
+            if call.before is not None:
+                x, pending = self.streams[call.before].forward(ctx, x, pending, at_start=call.index == 0)
             if call.add_embedding:
                 from ..kernels import ops
                 ops.add_residual(x, fed)      # a branch output still pending is added by the block's norm, as ever

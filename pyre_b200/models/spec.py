@@ -20,13 +20,15 @@ class LayerCall:
     entry) is added to the stream: a model that runs a span of its layers several times feeds its input in
     again at the start of every repeat.
     ``add_vector``: (name, row) of one of ``ModelSpec.vectors``: before this entry runs, that row of the tensor is
-    added to every token's stream (a model that marks each repeat of a span with a learned vector)."""
+    added to every token's stream (a model that marks each repeat of a span with a learned vector).
+    ``before``: the name of one of ``ModelSpec.streams``: before this entry runs, that stream part runs on the stream."""
 
     block: int
     cache: "int | str | None" = None
     write: bool = True
     add_embedding: bool = False
     add_vector: "tuple | None" = None
+    before: "str | None" = None
 
 
 @dataclass
@@ -53,6 +55,9 @@ class ModelSpec:
     # (``LayerCall.add_vector``); full checkpoint name -> number of rows
     vectors: dict = field(default_factory=dict)
     width: int = 0
+    # stream parts that belong to no block: an entry of the schedule names the one that runs before it
+    # (``LayerCall.before``); name -> (part, prefix of its tensors in the checkpoint)
+    streams: dict = field(default_factory=dict)
 
     def __post_init__(self):
         if not self.schedule:
@@ -64,6 +69,8 @@ class ModelSpec:
                 name, row = call.add_vector
                 if name not in self.vectors or not 0 <= row < self.vectors[name] or self.width <= 0:
                     raise ValueError(f"schedule adds row {row} of {name!r}, which the model's vectors (and width) do not give")
+            if call.before is not None and call.before not in self.streams:
+                raise ValueError(f"schedule runs {call.before!r} before an entry, which is none of the model's streams")
         if self.tail is None:
             if self.final_norm is None or self.head is None:
                 raise ValueError("a model needs a tail: give final_norm and head, or tail")

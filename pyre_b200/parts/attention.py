@@ -17,13 +17,14 @@ def attention_libraries(dtype, row_dim: int) -> list[str]:
     return ["attention_generic"]
 
 
-def attend(ctx, dtype, q, layer, kv, n_heads: int, n_kv_heads: int, row_dim: int, scale: float, window, sink=None):
-    """Softmax attention of every token of the step over its sequence's cached keys and values in ``layer``, by the
-    package's kernels: bfloat16 rows up to 128 on the tensor cores, everything else on the exact fp32 kernel."""
+def attend(ctx, dtype, q, layer, kv, n_heads: int, n_kv_heads: int, row_dim: int, scale: float, window, sink=None, keep_first: int = 0):
+    """Softmax attention of every token of the step over its sequence's cached keys and values in ``layer`` (with a
+    window: the last ``window`` of them and the first ``keep_first``), by the package's kernels: bfloat16 rows up to 128 on the tensor cores, everything else on the exact fp32 kernel."""
     if dtype == torch.bfloat16 and row_dim <= ops.MMA_MAX_HEAD_DIM:
-        return ops.paged_attention_bf16(ctx, q, layer, kv.block_table, n_heads, n_kv_heads, row_dim, scale, window, sink=sink)
+        return ops.paged_attention_bf16(ctx, q, layer, kv.block_table, n_heads, n_kv_heads, row_dim, scale, window, sink=sink,
+                                        keep_first=keep_first)
     return ops.paged_attention_generic(q, layer, kv.block_table, ctx.seq_of_token, ctx.positions, n_heads, n_kv_heads, row_dim,
-                                       scale, window, sink=sink)
+                                       scale, window, sink=sink, keep_first=keep_first)
 
 
 class Attention(Part):
@@ -37,13 +38,16 @@ class Attention(Part):
     ``position``, the PartSpec of the position encoding applied to q and k, and ``names``, the checkpoint's
     names of the four projections (default q_proj, k_proj, v_proj, o_proj: an architecture whose checkpoint
     calls them otherwise says so in its builder, no new part needed).
-    A query at position p sees keys max(0, p - window + 1)..p.
+    A query at position p sees keys max(0, p - window + 1)..p and, with ``keep_first``, the sequence's first
+    ``keep_first`` keys however far back they lie (at their true positions).
 
     Further parameters, all off by default (the stacked, fused path above is untouched by them):
     ``v_head_dim``: a value head's size when it differs from ``head_dim`` (the cache's rows then have one size that
     holds both, ``ops.attention_row_dim``, the rest zero);
     ``qk_norm``: an RMS norm per head over the ``head_dim`` dims of queries and keys before the position encoding,
     ``{"eps": e}``, with weights of ``head_dim`` entries shared by the heads (names ``q_norm`` / ``k_norm``);
+    ``qk_unit``: ``{"eps": e}``: queries and keys are divided by their root mean square over the ``head_dim`` dims per
+    head AFTER the position encoding, without a weight;
     ``sink``: the score of a sink that has no value: exp(sink) joins every softmax denominator; ``"learned"``: a score
     per query head read from the checkpoint (name ``sink``, [n_heads]);
     ``out_gate``: the concatenated heads are multiplied by sigmoid(W_g h) before the output projection (name ``g``);
@@ -67,10 +71,16 @@ class Attention(Part):
                  scale: "float | None" = None, window: "int | None" = None, names: "dict[str, str] | None" = None,
                  v_head_dim: "int | None" = None, qk_norm: "dict | None" = None, sink: "float | None" = None,
                  out_gate: "bool | str" = False, own_kv: bool = True, weight_suffix: str = ".weight",
-                 value_position: "PartSpec | None" = None):
+                 value_position: "PartSpec | None" = None, keep_first: int = 0, qk_unit: "dict | None" = None):
         super().__init__(dtype, device)
         self.v_head_dim = int(v_head_dim) if v_head_dim is not None else int(head_dim)
         self.qk_norm_eps = float(qk_norm["eps"]) if qk_norm is not None else None
+        self.qk_unit_eps = float(qk_unit["eps"]) if qk_unit is not None else None
+        if qk_unit is not None and qk_norm is not None and self.qk_unit_eps != self.qk_norm_eps:
+            raise ops.UnsupportedSize("norms of queries and keys before and after the position encoding share one eps")
+        self.keep_first = int(keep_first) if window is not None else 0
+        if self.keep_first < 0:
+            raise ValueError("keep_first must not be negative")
         self.learned_sink = sink == "learned"
         self.sink = None if sink is None or self.learned_sink else float(sink)
         if out_gate not in (False, True, "head"):
@@ -82,7 +92,8 @@ class Attention(Part):
             raise ops.UnsupportedSize("rotated values: an even value size and half-split pairs")
         # the general path: projections laid out by a ProjectionLayout, unfused small kernels
         self.general = (self.v_head_dim != int(head_dim) or qk_norm is not None or self.out_gate or not self.own_kv
-                        or self.value_position is not None or self.learned_sink)
+                        or self.value_position is not None or self.learned_sink or qk_unit is not None
+                        or (position is not None and position.params.get("pairing") == "interleaved"))
         if self.general and qkv_bias:
             raise ops.UnsupportedSize("projection biases together with v_head_dim, qk_norm, out_gate or own_kv=False are not implemented")
         self.names = dict(self.DEFAULT_NAMES, **(names or {}))
@@ -171,18 +182,18 @@ class Attention(Part):
         return libs
 
     def cache_spec(self):
-        return PagedKVSpec(self.n_kv_heads, self.row_dim, self.window)
+        return PagedKVSpec(self.n_kv_heads, self.row_dim, self.window, keep_first=self.keep_first)
 
     def state_spec(self):
         return None
 
     def launch_key(self, n_rows, max_context):
         # the tensor-core kernel's split count is chosen on the host from these numbers
-        return (ops.attention_splits(n_rows, n_rows, self.n_heads, self.n_kv_heads, max_context, self.window),)
+        return (ops.attention_splits(n_rows, n_rows, self.n_heads, self.n_kv_heads, max_context, self.window and self.window + self.keep_first),)
 
     def _attend(self, ctx, q, layer, kv):
         return attend(ctx, self.dtype, q, layer, kv, self.n_heads, self.n_kv_heads, self.row_dim, self.scale, self.window,
-                      sink=self.sink)
+                      sink=self.sink, keep_first=self.keep_first)
 
     def _forward_general(self, ctx, h, call):
         """Projections in one product [q | k | v | gate]; norm, position encoding and the paged write by the
@@ -197,7 +208,9 @@ class Attention(Part):
         if self.value_position is not None:
             vcos, vsin, _ = self.value_position.rotation(ctx, self.v_head_dim)
             kw["value_tables"] = (vcos, vsin)
-        q = self.position.apply_layout(ctx, proj, self.layout, self.q_norm_w, self.k_norm_w, self.qk_norm_eps or 0.0, kv,
+        if self.qk_unit_eps is not None:
+            kw["post_norm"] = True
+        q = self.position.apply_layout(ctx, proj, self.layout, self.q_norm_w, self.k_norm_w, self.qk_norm_eps or self.qk_unit_eps or 0.0, kv,
                                        layer if call.kv_write else None, **kw)
         a = self._attend(ctx, q, layer, kv)
         if self.head_gate or vcos is not None:

@@ -38,7 +38,9 @@ Interfaces by category (``ctx`` is the StepContext, T its number of tokens):
               ``kernels.ops.ScaledRows`` instead of a tensor (see ``PreNormBlock``)
     stream    forward(ctx, x, pending) -> (x, pending)   a step of a layer that works on the residual stream itself
               after the sublayers (a per-layer input derived from the step's token ids); a block that has one
-              calls it last
+              calls it last.  A stream part may also belong to the model (``ModelSpec.streams``) and run before
+              entries of the schedule that name it; such a part's ``begin(ctx, x)`` sees the embedding's output
+              before the first entry
     head      forward(ctx, h_rows) -> fp32 logits [R, vocab]
     tail      forward(ctx, x, pending) -> fp32 logits [R, vocab] at ``ctx.logit_rows``: everything after the last
               block (the built-in one: a norm over the wanted rows, then a head)
@@ -72,7 +74,8 @@ class PartSpec:
 class PagedKVSpec:
     """What an attention-like mixer needs from the paged cache: per token and layer,
     keys and values of ``n_kv_heads * head_dim`` elements each.  ``window``: only the
-    last ``window`` positions are ever read (None = all), so older pages may be given back.
+    last ``window`` positions are ever read (None = all), so older pages may be given back; ``keep_first``: with a
+    window, the sequence's first positions that are read for ever beside it, whose pages stay.
     ``planes``: 2 = a plane of keys and a plane of values per page; 1 = one plane of rows that serve as both (a
     cache of latent rows from which keys and values are derived)."""
 
@@ -80,6 +83,7 @@ class PagedKVSpec:
     head_dim: int
     window: int | None = None
     planes: int = 2
+    keep_first: int = 0
 
     def bytes_per_token(self, element_size: int) -> int:
         """Bytes of one token's keys and values in one layer of the group."""
@@ -88,8 +92,8 @@ class PagedKVSpec:
     def tokens_held(self, step_tokens: int) -> "int | None":
         """The most tokens of one request whose pages are held at a time, when a step brings it at most
         ``step_tokens`` new ones: None = all of them (no window); with a window, the window of the step's first
-        token and the step's own tokens."""
-        return None if self.window is None else self.window - 1 + step_tokens
+        token, the step's own tokens and the kept first ones."""
+        return None if self.window is None else self.window - 1 + step_tokens + self.keep_first
 
 
 @dataclass(frozen=True)
@@ -152,6 +156,7 @@ class BoundCall:
     state_layer: int = 0
     add_embedding: bool = False   # the embedding's output is added to the stream before this entry runs
     add_vector: "tuple | None" = None   # (tensor name, row): that row is added to every token's stream before the entry
+    before: "str | None" = None         # the model's stream part that runs on the stream before the entry
 
 
 class Part:
@@ -210,19 +215,29 @@ class PositionEncoding(Part):
         return None, None, 0
 
     def apply_layout(self, ctx, proj, layout: ProjectionLayout, q_norm, k_norm, norm_eps: float, kv, cache_layer,
-                     value_tables=None):
+                     value_tables=None, post_norm: bool = False):
         """The same step for projections laid out by a ``ProjectionLayout`` (key and value sizes that differ, rows
         padded to the cache's row size), with an optional RMS norm per head over the query and key dims before
         the encoding (``q_norm`` / ``k_norm``: fp32 weights [qk_dim] or None).  Stores keys and values in
         ``cache_layer`` (None: nothing) and returns the queries [T, n_heads * row_dim].  An encoding that is a
         rotation of leading dims only has to give ``rotation``.  ``value_tables``: (cos, sin) [T, v_dim / 2] of a
-        rotation that the mixer wants on the VALUES before they are cached (given only by a mixer that has one)."""
+        rotation that the mixer wants on the VALUES before they are cached (given only by a mixer that has one).
+        ``post_norm``: after the rotation queries and keys are divided by their root mean square per head (``norm_eps``,
+        no weight; given only by a mixer that wants it)."""
         from ..kernels import ops
         cos, sin, rotary_dim = self.rotation(ctx, layout.qk_dim)
         return ops.qk_norm_rope_write(proj, layout.q_col, layout.k_col, layout.v_col, q_norm, k_norm, norm_eps, cos, sin,
                                       cache_layer, kv.slot_mapping, layout.n_heads, layout.n_kv_heads, layout.qk_dim,
                                       layout.v_dim, layout.row_dim, rotary_dim, kv.page_size,
-                                      *(value_tables or ()))
+                                      *(value_tables or ()), **self._layout_options(post_norm))
+
+    def _layout_options(self, post_norm: bool) -> dict:
+        """Options of the fused rotation + write kernel beyond its defaults (a rotation of neighbouring pairs, a norm
+        after the rotation)."""
+        out = {"neighbours": True} if getattr(self, "pairing", "half") == "interleaved" else {}
+        if post_norm:
+            out["post_norm"] = True
+        return out
 
     @staticmethod
     def store(qkv, bias, heads: HeadGeometry, kv, cache_layer):

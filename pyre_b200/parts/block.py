@@ -110,7 +110,8 @@ register_part("block", "output_norm", OutputNormBlock)
 
 class ParallelBlock(Part):
     """x = x + m * (g1 * mixer(h) + g2 * ffn(h)) with h = norm1(x): ONE norm, both branches read its output, and
-    their results enter the stream together.  ``residual_mult`` is m; ``layer_scale``: g1 and g2 are gains per
+    their results enter the stream together.  ``norm2``: the feed-forward reads norm2(x) instead, a second norm of the
+    same x (one kernel forms both when the norms offer ``forward_pair``).  ``residual_mult`` is m; ``layer_scale``: g1 and g2 are gains per
     feature read from the checkpoint (names ``ls1`` / ``ls2``), else ones.  ``ffn`` None: the layer has the mixer
     only.
 
@@ -119,20 +120,26 @@ class ParallelBlock(Part):
 
     graph_safe = True
 
-    DEFAULT_NAMES = {"norm1": "norm1.", "mixer": "mixer.", "ffn": "ffn.", "ls1": "ls1", "ls2": "ls2"}
+    DEFAULT_NAMES = {"norm1": "norm1.", "norm2": "norm2.", "mixer": "mixer.", "ffn": "ffn.", "ls1": "ls1", "ls2": "ls2"}
 
     def __init__(self, dtype, device, width: int, norm1: PartSpec, mixer: PartSpec, ffn: "PartSpec | None" = None,
-                 residual_mult: float = 1.0, layer_scale: bool = False, names: "dict[str, str] | None" = None):
+                 residual_mult: float = 1.0, layer_scale: bool = False, names: "dict[str, str] | None" = None,
+                 norm2: "PartSpec | None" = None):
         super().__init__(dtype, device)
         self.names = dict(self.DEFAULT_NAMES, **(names or {}))
         self.width, self.residual_mult, self.layer_scale = int(width), float(residual_mult), bool(layer_scale)
         self.norm1 = make_part("norm", norm1, dtype, device)
         self.mixer = make_part("mixer", mixer, dtype, device)
         self.ffn = make_part("ffn", ffn, dtype, device) if ffn is not None else None
+        if norm2 is not None and ffn is None:
+            raise ValueError("a second norm needs the feed-forward that reads it")
+        self.norm2 = make_part("norm", norm2, dtype, device) if norm2 is not None else None
         self.gain1 = self.gain2 = None
 
     def children(self):
         out = {self.names["norm1"]: self.norm1, self.names["mixer"]: self.mixer}
+        if self.norm2 is not None:
+            out[self.names["norm2"]] = self.norm2
         if self.ffn is not None:
             out[self.names["ffn"]] = self.ffn
         return out
@@ -161,10 +168,16 @@ class ParallelBlock(Part):
         from ..kernels import ops
         if pending is not None and isinstance(pending, ops.ScaledSum) and not getattr(self.norm1, "takes_scaled_sum", False):
             pending = ops.materialize(pending)
-        h = self.norm1.forward(ctx, x, delta=pending)
+        if self.norm2 is None:
+            h = h2 = self.norm1.forward(ctx, x, delta=pending)
+        elif hasattr(self.norm1, "forward_pair"):
+            h, h2 = self.norm1.forward_pair(ctx, x, pending, self.norm2)
+        else:
+            h = self.norm1.forward(ctx, x, delta=pending)       # adds what is pending to x, which norm2 reads
+            h2 = self.norm2.forward(ctx, x)
         terms = [(self.mixer.forward(ctx, h, call), self.gain1)]
         if self.ffn is not None:
-            terms.append((self.ffn.forward(ctx, h), self.gain2))
+            terms.append((self.ffn.forward(ctx, h2), self.gain2))
         return x, ops.ScaledSum(terms, self.dtype)
 
 

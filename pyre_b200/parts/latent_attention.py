@@ -25,18 +25,22 @@ class LatentAttention(Part):
     q~_n = U_k,n^T q_plain,n (a product per head), scores against the cached rows themselves, the weighted sum of
     the latents per head, and then the head's value map (a second product per head).  Keys and values are never
     expanded, in prompts or in decoding.  ``window``: a query at position p sees p - window + 1 .. p (None: all).
-    ``position``: the PartSpec of a rotation that gives tables (``rotation(ctx, rope_dim)``) and pairs neighbours
-    (None with ``rope_dim`` 0: attention without positions).  ``q_rank`` None: the queries have no latent of their own,
-    q = W_q h (name ``q``).  Norms, angles, scores and the softmax are fp32."""
+    ``position``: the PartSpec of a rotation that gives tables (``rotation(ctx, rope_dim)``), of neighbouring or
+    half-split pairs (None with ``rope_dim`` 0: attention without positions).  ``q_rank`` None: the queries have no
+    latent of their own, q = W_q h (name ``q``); queries, latent and gates then come from ONE product of h.
+    ``sink``: a score per head read from the checkpoint (name ``sink``, [n_heads]): exp(sink) joins the head's
+    denominator, with no key and no value.  ``head_gate``: head n's output is multiplied by sigmoid(W_g h)_n (name
+    ``g``, [n_heads, width]); the attention kernel applies it where it normalises, since a scalar per head commutes
+    with the head's value map.  Norms, angles, scores and the softmax are fp32."""
 
     DEFAULT_NAMES = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk",
-                     "uv": "uv", "o": "o", "q": "q"}
+                     "uv": "uv", "o": "o", "q": "q", "sink": "sink", "g": "g"}
 
     graph_safe = True
 
     def __init__(self, dtype, device, width: int, n_heads: int, head_dim: int, rope_dim: int, v_head_dim: int,
                  q_rank: "int | None", kv_rank: int, scale: float, eps: float, position: "PartSpec | None" = None,
-                 window: "int | None" = None, names: "dict[str, str] | None" = None):
+                 window: "int | None" = None, names: "dict[str, str] | None" = None, sink: bool = False, head_gate: bool = False):
         super().__init__(dtype, device)
         self.names = dict(self.DEFAULT_NAMES, **(names or {}))
         self.width, self.n_heads, self.head_dim, self.rope_dim = int(width), int(n_heads), int(head_dim), int(rope_dim)
@@ -55,8 +59,11 @@ class LatentAttention(Part):
         if position is None and self.rope_dim:
             raise ValueError("a rotated key part needs a position encoding")
         self.position = make_part("position", position or PartSpec("none"), dtype, device)
-        if self.rope_dim and getattr(self.position, "pairing", "interleaved") != "interleaved":
-            raise ops.UnsupportedSize("the latent attention kernels rotate neighbouring pairs")
+        self.halves = getattr(self.position, "pairing", "interleaved") == "half"
+        self.has_sink, self.head_gate = bool(sink), bool(head_gate)
+        if self.head_gate and self.q_latent:
+            raise ops.UnsupportedSize("a gate per head together with a query latent is not implemented")
+        self.sink = None
         self.w_down = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = self.g_q = self.g_c = None
 
     def children(self):
@@ -75,6 +82,8 @@ class LatentAttention(Part):
             n["dkv_norm"]: TensorSpec((self.kv_rank,), role="vector", init=("normal", 1.0, 0.1)),
             n["uk"]: TensorSpec((H * self.head_dim, self.kv_rank)),
             n["uv"]: TensorSpec((H * self.v_head_dim, self.kv_rank)),
+            **({n["sink"]: TensorSpec((H,), role="vector", init=("normal", 0.0, 1.0))} if self.has_sink else {}),
+            **({n["g"]: TensorSpec((H, self.width))} if self.head_gate else {}),
             n["o"]: TensorSpec((self.width, H * self.v_head_dim)),
         }
 
@@ -84,7 +93,13 @@ class LatentAttention(Part):
             self.w_down = torch.cat([tensors[n["dq"]], tensors[n["dkv"]]], dim=0).contiguous()
             self.w_uq, self.g_q = tensors[n["uq"]], tensors[n["dq_norm"]]
         else:
-            self.w_down, self.w_uq = tensors[n["dkv"]], tensors[n["q"]]
+            # one product of h: [queries | latent and key part | gates], rows up to a multiple of 16 bytes
+            stack = [tensors[n["q"]], tensors[n["dkv"]]] + ([tensors[n["g"]]] if self.head_gate else [])
+            pad = -sum(w.shape[0] for w in stack) % 8
+            if pad:
+                stack.append(torch.zeros((pad, self.width), dtype=stack[0].dtype, device=stack[0].device))
+            self.w_down = torch.cat(stack, dim=0).contiguous()
+        self.sink = tensors[n["sink"]] if self.has_sink else None
         # the key map moves to the query: per head [kv_rank, head_dim], the layout of a linear layer from
         # head_dim to kv_rank
         self.w_uk_t = tensors[n["uk"]].view(H, self.head_dim, self.kv_rank).transpose(1, 2).contiguous()
@@ -113,19 +128,41 @@ class LatentAttention(Part):
         kv = ctx.kv_group(call.kv_group)
         layer = kv.pool[call.kv_layer]
         T, H = ctx.num_tokens, self.n_heads
+        cos, sin, rot = self.position.rotation(ctx, self.rope_dim) if self.rope_dim else (None, None, 0)
+        gate = None
+        if not self.q_latent:
+            with lib.section("qkv"):
+                proj = ops.materialize(ops.linear(h, self.w_down))
+            dk = self.head_dim + self.rope_dim
+            qa = torch.empty((T, H, self.row), dtype=self.dtype, device=proj.device)
+            # the latent's norm, the rotation of key part and queries, the paged write
+            ops.latent_prepare(proj, 0, 0, H * dk, self.kv_rank, self.rope_dim, rot, None, self.g_c, self.eps, cos, sin,
+                               layer if call.kv_write else None, kv.slot_mapping, kv.page_size, self.dtype,
+                               halves=self.halves, q_out=qa if self.row > self.kv_rank else None, qh_col=0, dq=self.head_dim)
+            with lib.section("absorb"):
+                ops.headwise_linear(proj[:, :H * dk].unflatten(1, (H, dk)), self.w_uk_t, out=qa)
+            if self.head_gate:
+                gate = (proj, H * dk + self.kv_rank + self.rope_dim)
+            return self._attend(ctx, qa, layer, kv, gate)
         with lib.section("qkv"):
             down = ops.linear(h, self.w_down, partials_ok=True)
-        cos, sin, rot = self.position.rotation(ctx, self.rope_dim) if self.rope_dim else (None, None, 0)
         cq = ops.latent_prepare(down, 0, self.q_rank, self.q_rank, self.kv_rank, self.rope_dim, rot, self.g_q, self.g_c,
-                                self.eps, cos, sin, layer if call.kv_write else None, kv.slot_mapping, kv.page_size, self.dtype)
+                                self.eps, cos, sin, layer if call.kv_write else None, kv.slot_mapping, kv.page_size, self.dtype,
+                                halves=self.halves)
         with lib.section("q_up"):
-            q = ops.materialize(ops.linear(cq if self.q_latent else h, self.w_uq))
+            q = ops.materialize(ops.linear(cq, self.w_uq))
         qa = torch.empty((T, H, self.row), dtype=self.dtype, device=q.device)
         with lib.section("absorb"):
             ops.headwise_linear(q.view(T, H, self.head_dim + self.rope_dim), self.w_uk_t, out=qa)
         if self.row > self.kv_rank:      # the rotated tail of the rows, and zeros up to the row size
-            ops.latent_rotate_q(q, qa, cos, sin, H, self.head_dim, self.rope_dim, rot, self.kv_rank)
-        lat = ops.latent_attention(ctx, qa, layer, kv.block_table, self.kv_rank, self.rope_dim, self.scale, self.window)
+            ops.latent_rotate_q(q, qa, cos, sin, H, self.head_dim, self.rope_dim, rot, self.kv_rank,
+                                halves=self.halves)
+        return self._attend(ctx, qa, layer, kv, None)
+
+    def _attend(self, ctx, qa, layer, kv, gate):
+        T, H = qa.shape[:2]
+        lat = ops.latent_attention(ctx, qa, layer, kv.block_table, self.kv_rank, self.rope_dim, self.scale, self.window,
+                                   sink=self.sink, gate=gate)
         with lib.section("v_up"):
             heads = ops.headwise_linear(lat, self.w_uv)
         with lib.section("o"):

@@ -15,8 +15,8 @@ class GatedMLP(Part):
     when I is a multiple of 128, their rows alternate in blocks of 64 features so that one
     output tile of the product holds both halves and the activation runs in its epilogue.
     ``names``: the checkpoint's names of the three projections (default gate_proj, up_proj, down_proj);
-    ``weight_suffix``: what follows a projection's name (".weight").  ``activation``: ``silu``, or ``gelu_tanh``
-    (product, then the activation kernel on the stacked [gates | ups])."""
+    ``weight_suffix``: what follows a projection's name (".weight").  ``activation``: ``silu`` or ``relu``
+    (both in the product's epilogue), or ``gelu_tanh`` (product, then the activation kernel on the stacked [gates | ups])."""
 
     DEFAULT_NAMES = {"gate": "gate_proj", "up": "up_proj", "down": "down_proj"}
 
@@ -29,13 +29,14 @@ class GatedMLP(Part):
         self.names = dict(self.DEFAULT_NAMES, **(names or {}))
         self.suffix = str(weight_suffix)
         self.width, self.intermediate = int(width), int(intermediate)
-        if activation not in ops.ACTIVATIONS:
-            raise ops.UnsupportedSize(f"activation {activation!r}: implemented are {sorted(ops.ACTIVATIONS)}")
+        if activation not in ops.MUL_ACTIVATIONS:
+            raise ops.UnsupportedSize(f"activation {activation!r}: implemented are {sorted(ops.MUL_ACTIVATIONS)}")
         self.activation = activation
         self.w_gate_up = self.w_down = None
-        # the product's epilogue knows silu; another activation runs after the product on [gates | ups]
-        self.interleaved = activation == "silu" and dtype == torch.bfloat16 and self.intermediate % (2 * ops.GATED_BLOCK) == 0
-        if activation != "silu":
+        # the product's epilogue knows silu and relu; another activation runs after the product on [gates | ups]
+        self.in_product = activation in ops.GATE_KINDS
+        self.interleaved = self.in_product and dtype == torch.bfloat16 and self.intermediate % (2 * ops.GATED_BLOCK) == 0
+        if not self.in_product:
             self.takes_scaled_rows = False
 
     def tensors(self):
@@ -56,13 +57,13 @@ class GatedMLP(Part):
         self.w_down = tensors[n["down"] + sfx]
 
     def kernel_libraries(self):
-        return ["elementwise"] + (["parallel_block"] if self.activation != "silu" else []) + \
+        return ["elementwise"] + (["parallel_block"] if not self.in_product else []) + \
             (["gemm_f32"] if self.dtype == torch.float32 else ["gemm_tc"])
 
     def forward(self, ctx, h):
         with lib.section("gate_up"):
-            if self.activation == "silu":
-                act = ops.gated_linear(h, self.w_gate_up, self.interleaved)
+            if self.in_product:
+                act = ops.gated_linear(h, self.w_gate_up, self.interleaved, **({} if self.activation == "silu" else {"kind": self.activation}))
             else:
                 act = ops.act_mul(ops.materialize(ops.linear(h, self.w_gate_up)), self.activation)
         with lib.section("down"):

@@ -88,6 +88,13 @@ class LayerNorm(Part):
     def forward(self, ctx, x, delta=None, rows=None, update_x=True, scaled_ok=False):
         return ops.add_layernorm(x, delta, self.weight, self.eps, self.dtype, rows=rows, update_x=update_x, bias=self.bias)
 
+    def forward_pair(self, ctx, x, delta, other: "LayerNorm"):
+        """(this norm of x + delta, ``other``'s norm of the same rows) in one pass: the norms of two branches that read
+        one stream.  ``other`` has this norm's eps and no bias."""
+        if other.eps != self.eps or other.bias is not None:
+            raise ops.UnsupportedSize("two norms in one pass share their eps, and the second has no bias")
+        return ops.add_layernorm(x, delta, self.weight, self.eps, self.dtype, bias=self.bias, weight2=other.weight)
+
     def gated_output(self, ctx, y, gate=None, gate_bias=None):
         """norm(y * sigmoid(gate + gate_bias)) * gain for a sublayer's result ``y`` that is not added to the stream
         here: it comes back as an fp32 branch output (one unrounded part in bfloat16) for the next norm to add."""

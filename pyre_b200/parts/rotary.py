@@ -40,8 +40,8 @@ class Rotary(PositionEncoding):
         if pairing not in ("half", "interleaved"):
             raise ops.UnsupportedSize(f"rotary pairing {pairing!r}: known are 'half' and 'interleaved'")
         # "half" pairs dims (j, j + rotary_dim / 2), "interleaved" pairs neighbours (2j, 2j + 1); the angles are the
-        # same.  The fused q/k/v kernels of ``apply`` rotate half-split pairs only; a mixer with a kernel of its own
-        # takes the tables (``rotation``) and ``pairing``.
+        # same.  The fused q/k/v kernels of ``apply`` rotate half-split pairs only; ``apply_layout`` serves both; a mixer
+        # with a kernel of its own takes the tables (``rotation``) and ``pairing``.
         self.pairing = pairing
         if self.rotary_dim % 2 or self.rotary_dim > self.head_dim:
             raise ops.UnsupportedSize(f"rotary_dim {self.rotary_dim} must be even and <= head_dim")
@@ -98,17 +98,11 @@ class Rotary(PositionEncoding):
             ctx.scratch[self._key] = tab
         return tab
 
-
     def rotation(self, ctx, qk_dim: int):
         if qk_dim != self.head_dim:
             raise ValueError(f"rotary part built for head_dim {self.head_dim}, used with {qk_dim}")
         cos, sin = self.tables(ctx)
         return cos, sin, self.rotary_dim
-
-    def apply_layout(self, ctx, proj, layout, q_norm, k_norm, norm_eps, kv, cache_layer, **kw):
-        if self.pairing != "half":
-            raise ops.UnsupportedSize("the q/k/v kernels rotate half-split pairs only")
-        return super().apply_layout(ctx, proj, layout, q_norm, k_norm, norm_eps, kv, cache_layer, **kw)
 
     def apply(self, ctx, qkv, bias, heads: HeadGeometry, kv, cache_layer):
         if self.pairing != "half":

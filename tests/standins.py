@@ -62,7 +62,7 @@ def qkv_rope_write(qkv, bias, cos, sin, cache_layer, slot_mapping, n_heads, n_kv
 
 
 def paged_attention_generic(q, cache_layer, block_table, seq_of_token, positions, n_heads, n_kv_heads, head_dim, scale,
-                            window=None, out=None, sink=None):
+                            window=None, out=None, sink=None, keep_first=0):
     T = q.shape[0]
     page_size = cache_layer.shape[3]
     n_rep = n_heads // n_kv_heads
@@ -70,9 +70,9 @@ def paged_attention_generic(q, cache_layer, block_table, seq_of_token, positions
     for t in range(T):
         b, p = int(seq_of_token[t]), int(positions[t])
         lo = 0 if not window else max(0, p - window + 1)
-        pos = torch.arange(lo, p + 1)
+        pos = torch.cat([torch.arange(0, min(keep_first, lo)), torch.arange(lo, p + 1)])
         pages = block_table[b].long()[pos // page_size]
-        assert (pages >= 0).all(), f"token {t}: a key in its window lies on a page that was given back"
+        assert (pages >= 0).all(), f"token {t}: a visible key lies on a page that was given back"
         keys = cache_layer[pages, 0, :, pos % page_size, :].float()          # [keys, kv heads, head_dim]
         vals = cache_layer[pages, 1, :, pos % page_size, :].float()
         qt = q[t].float().reshape(n_kv_heads, n_rep, head_dim)
@@ -114,7 +114,7 @@ def linear_act(x, w, kind):
 
 
 def qk_norm_rope_write(proj, q_col, k_col, v_col, q_weight, k_weight, eps, cos, sin, cache_layer, slot_mapping, n_heads,
-                       n_kv_heads, qk_dim, v_dim, row_dim, rotary_dim, page_size, v_cos=None, v_sin=None):
+                       n_kv_heads, qk_dim, v_dim, row_dim, rotary_dim, page_size, v_cos=None, v_sin=None, neighbours=False, post_norm=False):
     T = proj.shape[0]
     x = proj.float()
 
@@ -123,10 +123,9 @@ def qk_norm_rope_write(proj, q_col, k_col, v_col, q_weight, k_weight, eps, cos, 
         if w is not None:
             t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w
         if rotary_dim:
-            half = rotary_dim // 2
-            a, b, rest = t[..., :half], t[..., half:rotary_dim], t[..., rotary_dim:]
-            c, s = cos[:, None, :], sin[:, None, :]
-            t = torch.cat([a * c - b * s, b * c + a * s, rest], dim=-1)
+            t = _turn_pairs(t, cos, sin, rotary_dim, halves=not neighbours)
+        if post_norm:
+            t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
         return torch.nn.functional.pad(t, (0, row_dim - d))
 
     q = heads(q_col, n_heads, qk_dim, q_weight)
@@ -259,10 +258,13 @@ def sgemm_nt(a, w, bias=None, out=None):
     return y if bias is None else y + bias
 
 
-def silu_mul(gate_up, out=None, block=0):
+_GATES = {"silu": torch.nn.functional.silu, "relu": torch.relu}
+
+
+def silu_mul(gate_up, out=None, block=0, kind="silu"):
     assert block == 0, "the float32 path stacks all gates before all ups"
     inter = gate_up.shape[1] // 2
-    return torch.nn.functional.silu(gate_up[:, :inter]) * gate_up[:, inter:]
+    return _GATES[kind](gate_up[:, :inter]) * gate_up[:, inter:]
 
 
 def sample(logits, temperature=None, seeds=None, token_index=None, out=None):
@@ -285,7 +287,7 @@ def _branch(t):
     return t.float()
 
 
-def add_layernorm(x, delta, weight, eps, out_dtype, rows=None, update_x=True, act_dtype=None, bias=None):
+def add_layernorm(x, delta, weight, eps, out_dtype, rows=None, update_x=True, act_dtype=None, bias=None, weight2=None):
     from pyre_b200.kernels import ops
     v = x
     if delta is not None:
@@ -297,38 +299,57 @@ def add_layernorm(x, delta, weight, eps, out_dtype, rows=None, update_x=True, ac
     if rows is not None:
         v = v[rows.long()]
     dev = v - v.mean(-1, keepdim=True)
-    out = dev * torch.rsqrt(dev.pow(2).mean(-1, keepdim=True) + eps) * weight
-    return (out if bias is None else out + bias).to(out_dtype)
+    unit = dev * torch.rsqrt(dev.pow(2).mean(-1, keepdim=True) + eps)
+    out = unit * weight
+    out = (out if bias is None else out + bias).to(out_dtype)
+    return out if weight2 is None else (out, (unit * weight2).to(out_dtype))
+
+
+def stream_rows(x, delta, dtype):
+    from pyre_b200.kernels import ops
+    if delta is None:
+        return x.to(dtype, copy=True)
+    terms = delta.terms if isinstance(delta, ops.ScaledSum) else [(delta, 1.0)]
+    return (x + sum(g * _branch(t) for t, g in terms)).to(dtype)
+
+
+def stream_set(x, base, product):
+    x.copy_(base + _branch(product))
 
 
 def act_mul(gate_up, kind):
     g, u = gate_up.float().chunk(2, dim=1)
-    a = torch.nn.functional.silu(g) if kind == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
+    a = torch.nn.functional.gelu(g, approximate="tanh") if kind == "gelu_tanh" else _GATES[kind](g)
     return (a * u).to(gate_up.dtype)
 
 
-def _turn_pairs(v, cos, sin, rot):
-    """Neighbouring pairs of the first ``rot`` entries of the last axis turn by the token's angles; v [T, ..., n]."""
+def _turn_pairs(v, cos, sin, rot, halves=False):
+    """Neighbouring pairs (``halves``: pairs half apart) of the first ``rot`` entries of the last axis turn by the
+    token's angles; v [T, ..., n]."""
     if not rot:
         return v
     shape = [v.shape[0]] + [1] * (v.dim() - 2) + [rot // 2]
     c, s = cos.view(shape), sin.view(shape)
-    a, b = v[..., 0:rot:2], v[..., 1:rot:2]
+    first, second = (slice(0, rot // 2), slice(rot // 2, rot)) if halves else (slice(0, rot, 2), slice(1, rot, 2))
+    a, b = v[..., first], v[..., second]
     out = v.clone()
-    out[..., 0:rot:2] = a * c - b * s
-    out[..., 1:rot:2] = b * c + a * s
+    out[..., first] = a * c - b * s
+    out[..., second] = b * c + a * s
     return out
 
 
 def latent_prepare(proj, q_col, q_rank, c_col, rank, rope, rot, wq, wc, eps, cos, sin, cache_layer, slot_mapping, page_size,
-                   act_dtype):
+                   act_dtype, halves=False, q_out=None, qh_col=0, dq=0):
     x = _branch(proj)
     T = x.shape[0]
     rms = lambda v, w: v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w
     cq = rms(x[:, q_col:q_col + q_rank], wq).to(act_dtype) if q_rank else None
+    if q_out is not None:
+        nh = q_out.shape[1]
+        latent_rotate_q(x[:, qh_col:qh_col + nh * (dq + rope)], q_out, cos, sin, nh, dq, rope, rot, rank, halves)
     if cache_layer is not None:
         c = rms(x[:, c_col:c_col + rank], wc)
-        r = _turn_pairs(x[:, c_col + rank:c_col + rank + rope], cos, sin, rot)
+        r = _turn_pairs(x[:, c_col + rank:c_col + rank + rope], cos, sin, rot, halves)
         assert cache_layer.shape[1:3] == (1, 1)
         for t in range(T):
             page, off = divmod(int(slot_mapping[t]), page_size)
@@ -337,14 +358,14 @@ def latent_prepare(proj, q_col, q_rank, c_col, rank, rope, rot, wq, wc, eps, cos
     return cq
 
 
-def latent_rotate_q(q, qa, cos, sin, n_heads, dq, rope, rot, rank):
+def latent_rotate_q(q, qa, cos, sin, n_heads, dq, rope, rot, rank, halves=False):
     T = q.shape[0]
-    tail = _turn_pairs(q.float().view(T, n_heads, dq + rope)[..., dq:], cos, sin, rot)
+    tail = _turn_pairs(q.float().reshape(T, n_heads, dq + rope)[..., dq:], cos, sin, rot, halves)
     qa[..., rank:] = 0
     qa[..., rank:rank + rope] = tail.to(qa.dtype)
 
 
-def latent_attention(ctx, qa, cache_layer, block_table, rank, rope, scale, window):
+def latent_attention(ctx, qa, cache_layer, block_table, rank, rope, scale, window, sink=None, gate=None):
     T, nh, row = qa.shape
     page_size = cache_layer.shape[3]
     out = torch.empty((T, nh, rank), dtype=qa.dtype)
@@ -356,7 +377,12 @@ def latent_attention(ctx, qa, cache_layer, block_table, rank, rope, scale, windo
         assert (pages >= 0).all(), f"token {t}: a key in its window lies on a page that was given back"
         rows = cache_layer[pages, 0, 0, pos % page_size, :].float()             # [keys, row]
         scores = qa[t].float()[:, :rank + rope] @ rows[:, :rank + rope].t() * scale
-        out[t] = (torch.softmax(scores, dim=-1) @ rows[:, :rank]).to(qa.dtype)
+        if sink is not None:       # one more term in the denominator, with no value
+            scores = torch.cat([scores, sink.float().view(-1, 1)], dim=-1)
+        p = torch.softmax(scores, dim=-1)[:, :rows.shape[0]]
+        if gate is not None:
+            p = p * torch.sigmoid(gate[0][t, gate[1]:gate[1] + nh].float()).view(-1, 1)
+        out[t] = (p @ rows[:, :rank]).to(qa.dtype)
     return out
 
 
@@ -530,7 +556,7 @@ def install(monkeypatch) -> None:
                          add_row_vector=add_row_vector, gated_norm=gated_norm, scale_to_places=scale_to_places,
                          token_shift_mix=token_shift_mix, wkv_scan=wkv_scan, scale_cap=scale_cap, short_conv=short_conv,
                          ssm_scan=ssm_scan, group_norm_gate=group_norm_gate, diff_combine=diff_combine, rotate_heads=rotate_heads,
-                         side_gate=side_gate, token_gate_add=token_gate_add).items():
+                         side_gate=side_gate, token_gate_add=token_gate_add, stream_rows=stream_rows, stream_set=stream_set).items():
         monkeypatch.setattr(ops, name, fn)
     monkeypatch.setattr(ops, "device_error_flag", lambda device: flag)
     monkeypatch.setattr(ops, "check_device_errors", lambda device="cpu": None)
@@ -581,7 +607,7 @@ def gemm_tc(x, w, out_dtype=torch.bfloat16, plan=None, reduce=True, gated=False,
     if gated:
         assert N % (2 * ops.GATED_BLOCK) == 0
         y = (x.float() @ w.float().t()).view(M, N // (2 * ops.GATED_BLOCK), 2, ops.GATED_BLOCK)
-        return (torch.nn.functional.silu(y[:, :, 0]) * y[:, :, 1]).reshape(M, N // 2).to(torch.bfloat16)
+        return (_GATES["silu" if gated is True else gated](y[:, :, 0]) * y[:, :, 1]).reshape(M, N // 2).to(torch.bfloat16)
     per = -(-kb // splits) * 64
     parts = torch.stack([x[:, s * per:(s + 1) * per].float() @ w[:, s * per:(s + 1) * per].float().t() for s in range(splits)])
     if splits == 1 and reduce:
@@ -591,16 +617,16 @@ def gemm_tc(x, w, out_dtype=torch.bfloat16, plan=None, reduce=True, gated=False,
     return parts.sum(0).to(out_dtype)
 
 
-def silu_mul_any(gate_up, out=None, block=0):
+def silu_mul_any(gate_up, out=None, block=0, kind="silu"):
     if block == 0:
-        return silu_mul(gate_up.float()).to(gate_up.dtype)
+        return silu_mul(gate_up.float(), kind=kind).to(gate_up.dtype)
     T, two_i = gate_up.shape
     y = gate_up.float().view(T, two_i // (2 * block), 2, block)
-    return (torch.nn.functional.silu(y[:, :, 0]) * y[:, :, 1]).reshape(T, two_i // 2).to(gate_up.dtype)
+    return (_GATES[kind](y[:, :, 0]) * y[:, :, 1]).reshape(T, two_i // 2).to(gate_up.dtype)
 
 
 def _attend_entries(q, cache_layer, block_table, cu_seqlens, positions, n_seqs, n_heads, n_kv_heads, head_dim, scale, window,
-                    out, takes, sink=None):
+                    out, takes, sink=None, keep_first=0):
     cu = cu_seqlens.tolist()
     taken = 0
     for b in range(n_seqs):
@@ -610,12 +636,13 @@ def _attend_entries(q, cache_layer, block_table, cu_seqlens, positions, n_seqs, 
         taken += n
         rows = slice(cu[b], cu[b + 1])
         out[rows] = paged_attention_generic(q[rows], cache_layer, block_table[b:b + 1], torch.zeros(n, dtype=torch.int32),
-                                            positions[rows], n_heads, n_kv_heads, head_dim, scale, window, sink=sink)
+                                            positions[rows], n_heads, n_kv_heads, head_dim, scale, window, sink=sink,
+                                            keep_first=keep_first)
     return taken
 
 
 def paged_attention_mma(q, cache_layer, block_table, cu_seqlens, positions, n_seqs, n_heads, n_kv_heads, head_dim, scale,
-                        window=None, n_splits=1, out=None, scratch=None, max_len=0, uniform_len=0, sink=None):
+                        window=None, n_splits=1, out=None, scratch=None, max_len=0, uniform_len=0, sink=None, keep_first=0):
     from pyre_b200.kernels import ops
     assert q.dtype == cache_layer.dtype == torch.bfloat16 and head_dim <= ops.MMA_MAX_HEAD_DIM
     assert 1 <= n_splits <= ops.MAX_SCRATCH_SPLITS
@@ -624,27 +651,27 @@ def paged_attention_mma(q, cache_layer, block_table, cu_seqlens, positions, n_se
     if out is None:
         out = torch.empty_like(q)
     _attend_entries(q, cache_layer, block_table, cu_seqlens, positions, n_seqs, n_heads, n_kv_heads, head_dim, scale, window,
-                    out, lambda n: not (max_len > 0 and n > max_len), sink=sink)
+                    out, lambda n: not (max_len > 0 and n > max_len), sink=sink, keep_first=keep_first)
     return out
 
 
 def attention_prefill(q, cache_layer, block_table, cu_seqlens, positions, n_seqs, n_long_tokens, n_heads, n_kv_heads,
-                      head_dim, scale, window, out, min_len=32, sink=None):
+                      head_dim, scale, window, out, min_len=32, sink=None, keep_first=0):
     from pyre_b200.kernels import ops
     assert head_dim in ops.PREFILL_HEAD_DIMS
     taken = _attend_entries(q, cache_layer, block_table, cu_seqlens, positions, n_seqs, n_heads, n_kv_heads, head_dim, scale,
-                            window, out, lambda n: n >= min_len, sink=sink)
+                            window, out, lambda n: n >= min_len, sink=sink, keep_first=keep_first)
     assert taken == n_long_tokens, "n_long_tokens must count the tokens of the entries this kernel takes"
     return out
 
 
 def attention_prefill_tc(q, cache_layer, block_table, cu_seqlens, positions, n_seqs, n_long_tokens, n_heads, n_kv_heads,
-                         head_dim, scale, window, out, min_len, key_splits=1, sink=None):
+                         head_dim, scale, window, out, min_len, key_splits=1, sink=None, keep_first=0):
     page_size = cache_layer.shape[3]
     assert 1 <= key_splits <= 32
     assert page_size & (page_size - 1) == 0 and page_size >= 4, "the tcgen05 attention takes power-of-two pages"
     return attention_prefill(q, cache_layer, block_table, cu_seqlens, positions, n_seqs, n_long_tokens, n_heads, n_kv_heads,
-                             head_dim, scale, window, out, min_len, sink=sink)
+                             head_dim, scale, window, out, min_len, sink=sink, keep_first=keep_first)
 
 
 def install_bf16(monkeypatch, calls: "dict | None" = None) -> None:
