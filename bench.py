@@ -1084,6 +1084,110 @@ def run_nipudra(args) -> dict:
     return out
 
 
+def run_gadopel(args) -> dict:
+    """``--workload gadopel``: the Gadopel design (random weights) at two sets of layer sizes, two layers that run twice
+    (latent attention with a sink and a gate per head; grouped-query attention over a window beside kept first tokens;
+    each beside a relu-gated feed-forward; the stream fed with the embedding again before each pass), beside the
+    package's closest layers at equal sizes, run as often: Pivinex's latent attention beside a gelu-gated feed-forward,
+    and Tekarax's grouped-query attention with a dense feed-forward.  A 2,048-token prompt step and decode steps at
+    batch 8 and 64 with 2,048 tokens of context, device-timed, and per kernel class the device time of one such step with
+    the fraction of the measured peak."""
+    import numpy as np
+
+    from pyre_b200.config import config_from_dict
+
+    peaks = load_peaks()
+    V = 32768
+    sizes = {
+        # width; heads of 128 + 64, values of 128, latent; key/value heads of the grouped-query layer; window, kept
+        # first tokens; feed-forward
+        "2k": dict(H=2048, nh=16, dn=128, dr=64, dv=128, kr=256, nkv=4, win=1024, keep=64, I=8192),
+        "3.5k": dict(H=3584, nh=28, dn=128, dr=64, dv=128, kr=512, nkv=4, win=4096, keep=128, I=18944),
+    }
+    T, ctx_len, times = PROMPT_LEN, 2048, 2
+    rng = np.random.default_rng(0)
+    out = {"workload": "gadopel", "peaks": peaks, "prompt": T, "decode_context": ctx_len, "sizes": {}}
+    for tag, z in sizes.items():
+        H, nh, dn, dr, dv, kr, nkv, win, keep, I = (z[k] for k in ("H", "nh", "dn", "dr", "dv", "kr", "nkv", "win", "keep", "I"))
+        row, qr = kr + dr, 768
+        scaling = {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}
+        raw_g = {"architecture": "Gadopel", "vocab": V, "width": H, "norm": {"eps": 1e-6}, "loop": {"start": 0, "stop": 2, "times": times}, "layers": [
+            {"type": "latent_attention", "mixer": {"heads": nh, "dim": dn, "rot_dim": dr, "vdim": dv, "kv_rank": kr, "scale": (dn + dr) ** -0.5,
+                                                   "rot": {"dims": dr, "base": 1e6}}, "mlp": {"kind": "dense", "ff": I}},
+            {"type": "attention", "mixer": {"heads": nh, "kv_heads": nkv, "dim": dn, "vdim": dv, "scale": dn ** -0.5, "mask": {"size": win, "keep_first": keep},
+                                            "rot": {"dims": dn, "base": 1e6, "scaling": scaling}}, "mlp": {"kind": "dense", "ff": I}}]}
+        raw_p = {"architecture": "Pivinex", "vocab": V, "width": H, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+                 "loop": {"start": 0, "stop": 1, "times": times}, "layers": [
+            {"type": "latent_attention", "mixer": {"heads": nh, "dim": dn, "rot_dim": dr, "vdim": dv, "q_rank": qr, "kv_rank": kr, "scale": (dn + dr) ** -0.5,
+                                                   "mask": {"size": 1 << 20}, "rot": {"dims": dr, "base": 1e6}}, "mlp": {"kind": "dense", "ff": I}}]}
+        raw_t = {"architecture": "Tekarax", "vocab": V, "width": H, "norm": {"eps": 1e-6}, "loop": {"start": 0, "stop": 1, "times": times}, "layers": [
+            {"type": "attention", "mixer": {"heads": nh, "kv_heads": nkv, "dim": dn, "vdim": dv, "scale": dn ** -0.5,
+                                            "rot": {"dims": dn, "base": 1e6, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+             "mlp": {"kind": "dense", "ff": I}}]}
+        q, kv = nh * dn, nkv * dn
+
+        def pairs(Tn, B, before, window=None, kept=0):
+            """query-key pairs of a step of B entries, ``before`` tokens cached each"""
+            seen = np.arange(before, before + Tn // B) + 1
+            return B * float((np.minimum(seen, window + kept) if window else seen).sum())
+
+        def latent(Tn, B, before, n):
+            cached = B * (before + Tn // B)
+            return {
+                "absorb": {"bytes": n * (nh * dn * kr * 2 + Tn * nh * (dn + kr) * 2), "flops": 2.0 * n * Tn * nh * dn * kr},
+                "latent_attention": {"bytes": n * (cached * row * 2 + Tn * nh * (row + kr) * 2), "flops": 2.0 * n * nh * (kr + dr + kr) * pairs(Tn, B, before)},
+                "v_up": {"bytes": n * (nh * dv * kr * 2 + Tn * nh * (kr + dv) * 2), "flops": 2.0 * n * Tn * nh * kr * dv}}
+
+        def product(rows, cols, Tn, n):
+            return {"bytes": n * (rows * cols * 2 + Tn * (rows + cols) * 2), "flops": 2.0 * n * Tn * rows * cols}
+
+        def tail(Tn, B):
+            return {"head": {"bytes": V * H * 2 + B * (H * 2 + V * 4), "flops": 2.0 * B * H * V}, "embed": {"bytes": Tn * H * (2 + 4), "flops": 0}}
+
+        def gated(Tn, n):
+            return {"gate_up": {"bytes": n * (2 * I * H * 2 + Tn * (H + I) * 2), "flops": 4.0 * n * Tn * H * I}, "down": product(I, H, Tn, n)}
+
+        def work_gadopel(Tn, B, before):
+            cols = nh * (dn + dr) + kr + dr + nh + (q + 2 * kv)
+            per = Tn // B
+            seen = B * min(before + per, win + keep + per)
+            return {
+                "qkv": {"bytes": times * (cols * H * 2 + Tn * (2 * H + cols) * 2), "flops": 2.0 * times * Tn * H * cols},
+                "attention": {"bytes": times * (seen * 2 * kv * 2 + 2 * Tn * q * 2), "flops": 4.0 * times * nh * dn * pairs(Tn, B, before, win, keep)},
+                "o": product(nh * dv, H, Tn, 2 * times),
+                # the embedding's half once per step, the stream's half once per pass; fp32 results
+                "feed_again": {"bytes": (times + 1) * (H * H * 2 + Tn * H * (2 + 4)), "flops": 2.0 * (times + 1) * Tn * H * H},
+                "norm": {"bytes": Tn * H * (2 + 2 + 4 + 4 + 2 + 2), "flops": 0, "per_launch": True},
+                "rotary+write": {"bytes": Tn * (nh * dr + row + q + 2 * kv) * 2 // 2 * 2, "flops": 0, "per_launch": True},
+                **latent(Tn, B, before, times), **gated(Tn, 2 * times), **tail(Tn, B)}
+
+        def work_pivinex(Tn, B, before):
+            cols = qr + kr + dr
+            return {
+                "qkv": product(cols, H, Tn, times), "q_up": product(nh * (dn + dr), qr, Tn, times), "o": product(nh * dv, H, Tn, times),
+                "norm": {"bytes": Tn * H * (2 + 2 + 4 + 4 + 2), "flops": 0, "per_launch": True},
+                "rotary+write": {"bytes": Tn * (cols + qr + row + 2 * nh * dr) * 2 // 2, "flops": 0, "per_launch": True},
+                **latent(Tn, B, before, times), **gated(Tn, times), **tail(Tn, B)}
+
+        def work_tekarax(Tn, B, before):
+            cols = q + 2 * kv + nh
+            return {
+                "qkv": product(cols, H, Tn, times), "o": product(q, H, Tn, times), "up": product(I, H, Tn, times), "down": product(I, H, Tn, times),
+                "attention": {"bytes": times * (B * (before + Tn // B) * 2 * kv * 2 + 2 * Tn * q * 2), "flops": 4.0 * times * nh * dn * pairs(Tn, B, before)},
+                "residual_gate": product(H, H, Tn, 2 * times),
+                "activation": {"bytes": times * Tn * I * 4, "flops": 0},
+                "norm": {"bytes": Tn * H * (2 + 2 + 4 + 4), "flops": 0, "per_launch": True},
+                "gate": {"bytes": Tn * q * (2 + 2), "flops": 0, "per_launch": True},
+                "rotary+write": {"bytes": Tn * (q + 2 * kv) * 2 * 2, "flops": 0, "per_launch": True},
+                **tail(Tn, B)}
+
+        block = {"sizes": dict(z), "models": {}}
+        for name, raw, work in (("gadopel", raw_g, work_gadopel), ("pivinex", raw_p, work_pivinex), ("tekarax", raw_t, work_tekarax)):
+            block["models"][name] = dict(layers=len(raw["layers"]), times=times, **_measure_design(config_from_dict(raw), work, args, peaks, V, T, ctx_len, rng))
+        out["sizes"][tag] = block
+    return out
+
+
 def run_sweep(args) -> dict:
     """Decode throughput over a grid of batch sizes and context lengths and prefill throughput over
     several portion lengths on the 7B shape, each with its fraction of the roofline (device-timed,
@@ -1207,11 +1311,11 @@ def main() -> int:
                     help="leave out the points at longer contexts and at the 14B and 32B shapes")
     ap.add_argument("--no-per-kernel", action="store_true",
                     help="leave out the `kernels` block (device time, bytes or flops and fraction of the peak per kernel class)")
-    ap.add_argument("--workload", choices=["serve14b", "mixed32b", "sweep", "modovik", "pivinex", "tekarax", "nipudra"], default=None,
+    ap.add_argument("--workload", choices=["serve14b", "mixed32b", "sweep", "modovik", "pivinex", "tekarax", "nipudra", "gadopel"], default=None,
                     help="run one of the two other baseline workloads, a sweep over batch sizes, context lengths and "
                          "portion lengths on the 7B shape, the Modovik or the Pivinex design beside the Qwen2.5 decoder at "
                          "equal layer sizes, the Tekarax design beside the closest layers of those two, or the Nipudra design beside the closest "
-                         "layers of Tekarax and Modovik, instead (prints its own JSON line)")
+                         "layers of Tekarax and Modovik, or the Gadopel design beside the closest layers of Pivinex and Tekarax, instead (prints its own JSON line)")
     ap.add_argument("--cache-fraction", type=float, default=1.0,
                     help="serve14b: cache capacity as a fraction of what all requests need at once (< 1 forces preemption)")
     args = ap.parse_args()
@@ -1220,7 +1324,8 @@ def main() -> int:
         return 2
     if args.workload:
         result = run_sweep(args) if args.workload == "sweep" else run_modovik(args) if args.workload == "modovik" else \
-            run_pivinex(args) if args.workload == "pivinex" else run_tekarax(args) if args.workload == "tekarax" else run_nipudra(args) if args.workload == "nipudra" else run_workload(args)
+            run_pivinex(args) if args.workload == "pivinex" else run_tekarax(args) if args.workload == "tekarax" else run_nipudra(args) if args.workload == "nipudra" else \
+            run_gadopel(args) if args.workload == "gadopel" else run_workload(args)
         result["env"] = environment()
         print(json.dumps(result))
         return 0
