@@ -1158,7 +1158,8 @@ def run_gadopel(args) -> dict:
                 # the embedding's half once per step, the stream's half once per pass; fp32 results
                 "feed_again": {"bytes": (times + 1) * (H * H * 2 + Tn * H * (2 + 4)), "flops": 2.0 * (times + 1) * Tn * H * H},
                 "norm": {"bytes": Tn * H * (2 + 2 + 4 + 4 + 2 + 2), "flops": 0, "per_launch": True},
-                "rotary+write": {"bytes": Tn * (nh * dr + row + q + 2 * kv) * 2 // 2 * 2, "flops": 0, "per_launch": True},
+                # rotated parts of the queries, latent rows; whole heads of the grouped-query layer: read and written once
+                "rotary+write": {"bytes": times * Tn * (nh * dr + row + q + 2 * kv) * 4, "flops": 0},
                 **latent(Tn, B, before, times), **gated(Tn, 2 * times), **tail(Tn, B)}
 
         def work_pivinex(Tn, B, before):
@@ -1166,7 +1167,7 @@ def run_gadopel(args) -> dict:
             return {
                 "qkv": product(cols, H, Tn, times), "q_up": product(nh * (dn + dr), qr, Tn, times), "o": product(nh * dv, H, Tn, times),
                 "norm": {"bytes": Tn * H * (2 + 2 + 4 + 4 + 2), "flops": 0, "per_launch": True},
-                "rotary+write": {"bytes": Tn * (cols + qr + row + 2 * nh * dr) * 2 // 2, "flops": 0, "per_launch": True},
+                "rotary+write": {"bytes": times * Tn * (cols + qr + row + 2 * nh * dr) * 2, "flops": 0},
                 **latent(Tn, B, before, times), **gated(Tn, times), **tail(Tn, B)}
 
         def work_tekarax(Tn, B, before):
@@ -1178,7 +1179,7 @@ def run_gadopel(args) -> dict:
                 "activation": {"bytes": times * Tn * I * 4, "flops": 0},
                 "norm": {"bytes": Tn * H * (2 + 2 + 4 + 4), "flops": 0, "per_launch": True},
                 "gate": {"bytes": Tn * q * (2 + 2), "flops": 0, "per_launch": True},
-                "rotary+write": {"bytes": Tn * (q + 2 * kv) * 2 * 2, "flops": 0, "per_launch": True},
+                "rotary+write": {"bytes": times * Tn * (q + 2 * kv) * 2 * 2, "flops": 0},
                 **tail(Tn, B)}
 
         block = {"sizes": dict(z), "models": {}}

@@ -324,6 +324,72 @@ __global__ void qk_norm_rope_write_kernel(const T* proj, long long row_stride, i
     for (int d = lane; d < D; d += 32) dst[d] = from_f32<T>(d < dk ? __fmul_rn(n[d], rstd) : 0.f);
 }
 
+// The same for neighbouring pairs without a norm before the rotation, in vectors of four entries per lane (dk, dv, D, rot
+// and every column multiples of 4, at most 256 entries a row): both entries of a pair lie in one lane, so a head goes
+// from one load to one store through registers.
+template <typename T>
+__global__ void qk_neighbours_write_kernel(const T* proj, long long row_stride, int q_col, int k_col, int v_col, float eps,
+                                           const float* cos_t, const float* sin_t, T* q_out, T* cache, const int* slot_mapping,
+                                           int n_tokens, int nh, int nkv, int dk, int dv, int D, int rot, int post_norm, int page_size,
+                                           long long n_pages, int* err_flag) {
+    pdl_trigger();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const int per_token = nh + (k_col >= 0 ? 2 * nkv : 0);
+    const long long item = (long long)blockIdx.x * warps + warp;
+    if (item >= (long long)n_tokens * per_token) return;
+    const int t = (int)(item / per_token), h = (int)(item - (long long)t * per_token);
+    const bool is_q = h < nh, is_k = !is_q && h < nh + nkv;
+    const T* src = proj + (size_t)t * row_stride;
+    T* dst;
+    if (is_q) {
+        src += q_col + (size_t)h * dk;
+        dst = q_out + ((size_t)t * nh + h) * D;
+    } else {
+        const int slot = (cache && slot_mapping) ? pyre_checked_slot(slot_mapping[t], n_pages, page_size, err_flag) : -1;
+        if (slot < 0) return;
+        const int page = slot / page_size, off = slot - page * page_size, kvh = is_k ? h - nh : h - nh - nkv;
+        src += is_k ? k_col + (size_t)kvh * dk : v_col + (size_t)kvh * dv;
+        dst = cache + ((((size_t)page * 2 + (is_k ? 0 : 1)) * nkv + kvh) * page_size + off) * D;
+    }
+    const bool turn = is_q || is_k;
+    const int n = turn ? dk : dv;
+    float v[2][4];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        const int d = 4 * (lane + 32 * c);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[c][k] = 0.f;
+        if (d >= n) continue;
+        const Vec<T, 4> in = load_vec<T, 4>(src + d);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[c][k] = to_f32<T>(in.v[k]);
+        if (turn && d < rot) {
+            const Vec<float, 2> cs = load_vec<float, 2>(cos_t + (size_t)t * (rot / 2) + d / 2), sn = load_vec<float, 2>(sin_t + (size_t)t * (rot / 2) + d / 2);
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const float a = v[c][2 * k], b = v[c][2 * k + 1];
+                v[c][2 * k] = __fadd_rn(__fmul_rn(a, cs.v[k]), __fmul_rn(-b, sn.v[k]));
+                v[c][2 * k + 1] = __fadd_rn(__fmul_rn(b, cs.v[k]), __fmul_rn(a, sn.v[k]));
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) ss = fmaf(v[c][k], v[c][k], ss);
+    }
+    float rstd = 1.f;
+    if (turn && post_norm) rstd = 1.0f / sqrtf(warp_sum(ss) / (float)dk + eps);
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        const int d = 4 * (lane + 32 * c);
+        if (d >= D) continue;
+        Vec<T, 4> o;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) o.v[k] = from_f32<T>(__fmul_rn(v[c][k], rstd));
+        store_vec<T, 4>(dst + d, o);
+    }
+}
+
 PYRE_API int pyre_qk_norm_rope_write(const void* proj, long long row_stride, int q_col, int k_col, int v_col,
                                      const float* q_w, const float* k_w, float eps, const float* cos_t, const float* sin_t,
                                      const float* vcos_t, const float* vsin_t, void* q_out, void* cache, const int* slot_mapping, int n_tokens, int nh, int nkv,
@@ -339,6 +405,17 @@ PYRE_API int pyre_qk_norm_rope_write(const void* proj, long long row_stride, int
     const long long items = (long long)n_tokens * (nh + (k_col >= 0 ? 2 * nkv : 0));
     const int blocks = (int)ceil_div_ll(items, warps);
     const size_t smem = (size_t)warps * D * sizeof(float);
+    const int kv_cols = k_col >= 0 ? k_col | v_col : 0;
+    if (neighbours && !q_w && !k_w && !vcos_t && D <= 256 && ((dk | dv | D | rot | q_col | kv_cols | (int)(row_stride & 3)) & 3) == 0 &&
+        (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache | (uintptr_t)cos_t | (uintptr_t)sin_t) & 15) == 0 &&
+        (dtype == PYRE_BF16 || dtype == PYRE_F32)) {
+        if (dtype == PYRE_BF16)
+            pyre_launch(qk_neighbours_write_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), 0, stream, (const __nv_bfloat16*)proj, row_stride, q_col, k_col, v_col, eps, cos_t, sin_t, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, post_norm, page_size, n_pages, err_flag);
+        else
+            pyre_launch(qk_neighbours_write_kernel<float>, dim3(blocks), dim3(warps * 32), 0, stream, (const float*)proj, row_stride, q_col, k_col, v_col, eps, cos_t, sin_t, (float*)q_out, (float*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, post_norm, page_size, n_pages, err_flag);
+        PYRE_LAUNCH_CHECK();
+        return 0;
+    }
     if (dtype == PYRE_BF16)
         pyre_launch(qk_norm_rope_write_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, stream, (const __nv_bfloat16*)proj, row_stride, q_col, k_col, v_col, q_w, k_w, eps, cos_t, sin_t, vcos_t, vsin_t, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, neighbours, post_norm, page_size, n_pages, err_flag);
     else if (dtype == PYRE_F32)

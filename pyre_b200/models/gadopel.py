@@ -48,7 +48,9 @@ def build_gadopel(cfg: GadopelConfig) -> ModelSpec:
                 "names": {"q": "q", "k": "k", "v": "v", "o": "o"}})
         params = {"width": cfg.width, "norm1": norm(), "mixer": mixer,
                   "names": {"norm1": "norm1", "norm2": "norm2", "mixer": "mix.", "ffn": "mlp."}}
-        if L.ff:
+        if not L.ff:
+            params["spare_norm2"] = True
+        else:
             params["norm2"] = norm()
             params["ffn"] = PartSpec("gated_mlp", {"width": cfg.width, "intermediate": L.ff, "activation": "relu",
                                                    "names": {"gate": "gate", "up": "up", "down": "down"}, "weight_suffix": ""})

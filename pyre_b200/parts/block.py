@@ -111,7 +111,8 @@ register_part("block", "output_norm", OutputNormBlock)
 class ParallelBlock(Part):
     """x = x + m * (g1 * mixer(h) + g2 * ffn(h)) with h = norm1(x): ONE norm, both branches read its output, and
     their results enter the stream together.  ``norm2``: the feed-forward reads norm2(x) instead, a second norm of the
-    same x (one kernel forms both when the norms offer ``forward_pair``).  ``residual_mult`` is m; ``layer_scale``: g1 and g2 are gains per
+    same x (one kernel forms both when the norms offer ``forward_pair``); ``spare_norm2``: the layer has no feed-forward,
+    but its checkpoint may hold a second norm's weight all the same.  ``residual_mult`` is m; ``layer_scale``: g1 and g2 are gains per
     feature read from the checkpoint (names ``ls1`` / ``ls2``), else ones.  ``ffn`` None: the layer has the mixer
     only.
 
@@ -124,7 +125,7 @@ class ParallelBlock(Part):
 
     def __init__(self, dtype, device, width: int, norm1: PartSpec, mixer: PartSpec, ffn: "PartSpec | None" = None,
                  residual_mult: float = 1.0, layer_scale: bool = False, names: "dict[str, str] | None" = None,
-                 norm2: "PartSpec | None" = None):
+                 norm2: "PartSpec | None" = None, spare_norm2: bool = False):
         super().__init__(dtype, device)
         self.names = dict(self.DEFAULT_NAMES, **(names or {}))
         self.width, self.residual_mult, self.layer_scale = int(width), float(residual_mult), bool(layer_scale)
@@ -134,6 +135,7 @@ class ParallelBlock(Part):
         if norm2 is not None and ffn is None:
             raise ValueError("a second norm needs the feed-forward that reads it")
         self.norm2 = make_part("norm", norm2, dtype, device) if norm2 is not None else None
+        self.spare_norm2 = bool(spare_norm2) and self.norm2 is None
         self.gain1 = self.gain2 = None
 
     def children(self):
@@ -146,9 +148,10 @@ class ParallelBlock(Part):
 
     def tensors(self):
         from ..weights.specs import TensorSpec
+        spare = {self.names["norm2"]: TensorSpec((self.width,), role="vector", init=("normal", 1.0, 0.1), optional=True)} if self.spare_norm2 else {}
         if not self.layer_scale:
-            return {}
-        t = {self.names["ls1"]: TensorSpec((self.width,), role="vector", init=("normal", 1.0, 0.1))}
+            return spare
+        t = {**spare, self.names["ls1"]: TensorSpec((self.width,), role="vector", init=("normal", 1.0, 0.1))}
         # a layer without a feed-forward has no use for the second gain; a checkpoint may hold it all the same
         t[self.names["ls2"]] = TensorSpec((self.width,), role="vector", init=("normal", 1.0, 0.1), optional=self.ffn is None)
         return t

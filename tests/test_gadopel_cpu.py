@@ -66,7 +66,8 @@ def test_tensor_names_and_cache_groups():
     table = tensor_table(spec)
     assert {"embed", "head", "loop.in", "final.norm", "l0.norm1", "l0.norm2", "l0.mix.q", "l0.mix.v", "l0.mlp.gate", "l1.mix.dkv.norm",
             "l1.mix.sink", "l1.mix.g", "l1.mix.uk", "l1.mix.uv", "l1.mix.o", "l2.mix.k", "l3.norm1"} <= set(table)
-    assert not {"l2.norm2", "l3.norm2", "l2.mlp.up", "l0.mix.sink", "l0.mix.g", "l1.mix.k", "l1.mix.dq", "l0.mix.q_norm"} & set(table)
+    assert table["l2.norm2"].optional and table["l3.norm2"].optional and not table["l0.norm2"].optional      # layers without a feed-forward
+    assert not {"l2.mlp.up", "l0.mix.sink", "l0.mix.g", "l1.mix.k", "l1.mix.dq", "l0.mix.q_norm"} & set(table)
     assert table["loop.in"].shape == (96, 192) and table["l1.mix.q"].shape == (3 * 24, 96) and table["l1.mix.dkv"].shape == (48, 96)
     assert table["l1.mix.sink"].shape == (3,) and table["l1.mix.g"].shape == (3, 96) and table["l1.mix.uv"].shape == (72, 40)
     assert table["l0.mix.k"].shape == (48, 96) and table["l0.mix.v"].shape == (72, 96) and table["l0.mix.o"].shape == (96, 144)
@@ -195,6 +196,18 @@ def test_the_models_of_these_tests_show_a_fault(folders, monkeypatch, fault):
         monkeypatch.setattr(GP, "visible", lambda T, window=None, keep=0: visible(T, window + dw, keep + dk) if window else visible(T))
     wrong = GH.plain_logits(d, ids)
     assert np.abs(wrong - plain["A4"]).max() > 30 * (1e-4 + 2e-4 * np.abs(plain["A4"]).max())
+
+
+def test_a_layer_without_a_feed_forward_may_hold_its_second_norm(tmp_path, monkeypatch, folders):
+    from safetensors.torch import load_file, save_file
+    d, reqs, plain = folders["A"]
+    state = load_file(str(d / "model.safetensors"))
+    assert "l2.norm2" not in state
+    state["l2.norm2"] = torch.full((96,), 3.0)
+    (tmp_path / "config.json").write_text((d / "config.json").read_text())
+    save_file(state, str(tmp_path / "model.safetensors"))
+    got = _replay_on_cpu(monkeypatch, tmp_path, H.trace_whole({"A2": reqs["A2"]}), 16)
+    GH.compare(got, {"A2": plain["A2"]}, "float32", "whole")
 
 
 def test_random_model_folder_loads(tmp_path, monkeypatch):

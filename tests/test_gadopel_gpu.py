@@ -89,10 +89,12 @@ def test_the_relu_gate_in_every_form_of_the_gated_product(ops, dtype, T, K, I):
 @pytest.mark.parametrize("dtype", BOTH)
 @pytest.mark.parametrize("neighbours", [False, True])
 @pytest.mark.parametrize("nh,nkv,dk,dv,rot,D,page,norm", [(6, 3, 16, 24, 8, 32, 16, False), (5, 5, 20, 28, 12, 32, 8, False), (4, 2, 64, 48, 64, 64, 32, False),
-                                                        (4, 1, 128, 128, 96, 128, 16, True), (2, 1, 48, 40, 0, 48, 4, False), (3, 1, 200, 64, 130, 208, 16, True)])
+                                                        (4, 1, 128, 128, 96, 128, 16, True), (2, 1, 48, 40, 0, 48, 4, False), (3, 1, 200, 64, 130, 208, 16, True),
+                                                        (4, 1, 128, 128, 96, 128, 16, False), (2, 2, 256, 64, 128, 256, 16, False), (3, 3, 12, 12, 4, 16, 8, False)])
 def test_rotation_then_unit_heads_then_the_paged_write(ops, dtype, neighbours, nh, nkv, dk, dv, rot, D, page, norm):
     T, n_pages, eps = 9, 7, 1e-3          # a large eps: where it stands matters
-    W = nh * dk + nkv * (dk + dv) + 3
+    pad = 3 if norm or dk == 20 else 4      # rows of four-entry vectors, and rows that are not
+    W = nh * dk + nkv * (dk + dv) + pad
     proj = bf16_exact(T, W, scale=0.1, seed=dk)
     pos = torch.tensor([0, 1, 2, 3, 77, 78, 500, 511, 600])
     scaling = {"factor": 8.0, "original": 64, "fast": 4.0, "slow": 0.5} if neighbours else None
@@ -110,7 +112,7 @@ def test_rotation_then_unit_heads_then_the_paged_write(ops, dtype, neighbours, n
         return GP.unit_rms(v, eps)
     want_q = turned(proj[:, :nh * dk].view(T, nh, dk))
     want_k = turned(proj[:, nh * dk:nh * dk + nkv * dk].view(T, nkv, dk))
-    want_v = proj[:, nh * dk + nkv * dk:W - 3].view(T, nkv, dv)
+    want_v = proj[:, nh * dk + nkv * dk:W - pad].view(T, nkv, dv)
     got = q.view(T, nh, D)
     close(got[..., :dk], want_q, dtype, "queries", atol32=2e-4)
     flat = cache.permute(0, 3, 1, 2, 4).reshape(-1, 2, nkv, D)[slots.cuda()]
