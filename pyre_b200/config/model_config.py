@@ -965,3 +965,223 @@ class GadopelConfig(ModelConfig):
         for _ in range(self.loop_times):
             order += [(i, i == self.loop_start) for i in range(self.loop_start, self.loop_stop)]
         return order + [(i, False) for i in range(self.loop_stop, len(self.layers))]
+
+
+@dataclass(frozen=True)
+class GugidraLayer:
+    """One layer of a Gugidra model: which mixer (``kind``: "gla" or "parallel") with its sizes, and its feed-forward:
+    ``mlp_kind`` "dense" (``ff`` wide), "moe" (``experts`` experts of ``ff``, ``top`` per token, plus a shared one of
+    ``shared_ff`` when that is positive) or "" (none)."""
+
+    kind: str
+    heads: int                     # gla: heads; parallel: query heads of the attention
+    dim: int                       # query/key entries per head
+    vdim: int                      # value entries per head (parallel: the attention's values are its keys, vdim = dim)
+    tau: float = 0.0               # gla: root taken of the decay's sigmoid
+    decay_rank: int = 0            # gla: inner size of the decay's two-layer map (0: read from the tensor's shape)
+    kv_heads: int = 0              # parallel: key/value heads of the attention
+    scale: float = 0.0             # parallel: factor on q . k
+    rot_dims: int = 0              # parallel: leading entries of a head that are rotated
+    rot_base: float = 10000.0
+    left_scale: float = 1.0        # parallel: factor on the attention's result
+    memory_heads: int = 0          # parallel: heads of the matrix memory, with
+    memory_dim: int = 0            # so many query/key
+    memory_vdim: int = 0           # and value entries each
+    gate_cap: float = 0.0          # parallel: bound of the memory's gate logits
+    right_scale: float = 1.0       # parallel: factor on the memory's result
+    mlp_kind: str = ""
+    ff: int = 0
+    limit: float = 0.0             # bound of the clamped gate
+    experts: int = 0
+    top: int = 0
+    group_count: int = 1           # the experts form so many equal groups, of which
+    group_keep: int = 1            # so many can be chosen from
+    shared_ff: int = 0
+    shared_limit: float = 0.0
+
+
+@dataclass(frozen=True)
+class GugidraConfig(ModelConfig):
+    """A Gugidra decoder: a scaled embedding; layers with an RMS norm (gain stored around zero) before AND after each
+    sublayer; gated linear attention, or attention and a matrix memory side by side, in any order; clamped gated
+    feed-forwards, dense or routed in groups; a span of layers that runs several times in a row, each pass with a cache and
+    state of its own, a learned vector added before it and the embedding's output before every one but the first; a final
+    norm and a head with soft-capped logits.  ``config.json`` keys: ``vocab``, ``width``, ``norm.eps``, ``embedding.scale``,
+    ``logit_softcap``, ``loop {start, stop, times}`` (absent: no repeated span) and ``layers``, a list of ``{"type", "mixer":
+    {...}, "mlp": {"kind": "dense", "ff", "limit"} | {"kind": "moe", "expert": {"ff", "limit"}, "router": {experts, top,
+    groups: {count, keep}}, "shared": {"ff", "limit"}} | null}`` with the mixers ``gla {heads, dim, vdim, tau}`` and ``parallel
+    {left: {heads, kv_heads, dim, vdim, scale, rot: {dims, base}}, right: {heads, dim, vdim, gate_cap}, left_scale,
+    right_scale}``.  A size that the file does not give (the inner size of a gla layer's decay map) is read from the shape
+    of the layer's tensor (``with_tensor_shapes``)."""
+
+    architecture: ClassVar[str] = "Gugidra"
+    KINDS: ClassVar[tuple] = ("gla", "parallel")
+
+    vocab: int
+    width: int
+    norm_eps: float
+    layers: tuple
+    embedding_scale: float = 1.0
+    logit_softcap: float = 0.0
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 0            # 0: no repeated span
+
+    def __post_init__(self):
+        _positive("vocab", self.vocab)
+        _positive("width", self.width)
+        if not self.norm_eps > 0:
+            raise ConfigError(f"config.json: norm.eps must be positive, got {self.norm_eps}")
+        if not self.layers:
+            raise ConfigError("config.json: layers is empty")
+        if self.logit_softcap < 0:
+            raise ConfigError("config.json: logit_softcap must not be negative")
+        if self.loop_times < 0 or (self.loop_times and not 0 <= self.loop_start < self.loop_stop <= len(self.layers)):
+            raise ConfigError(f"config.json: loop (start {self.loop_start}, stop {self.loop_stop}, times {self.loop_times}) must lie "
+                              f"within the {len(self.layers)} layers")
+        for i, L in enumerate(self.layers):
+            where = f"config.json: layers[{i}]"
+            if L.kind not in self.KINDS:
+                raise ConfigError(f"{where}.type {L.kind!r}: known are {', '.join(self.KINDS)}")
+            if min(L.heads, L.dim, L.vdim) <= 0:
+                raise ConfigError(f"{where}.mixer: heads, dim and vdim must be positive")
+            if L.kind == "gla" and (not L.tau > 0 or L.decay_rank < 0):
+                raise ConfigError(f"{where}.mixer.tau must be positive")
+            if L.kind == "parallel":
+                if L.kv_heads <= 0 or L.heads % L.kv_heads:
+                    raise ConfigError(f"{where}.mixer.left.kv_heads ({L.kv_heads}) must divide heads ({L.heads})")
+                if L.vdim != L.dim:
+                    raise ConfigError(f"{where}.mixer.left.vdim ({L.vdim}) must be dim ({L.dim}): the values are the keys")
+                if not L.scale > 0:
+                    raise ConfigError(f"{where}.mixer.left.scale must be positive")
+                if L.rot_dims < 0 or L.rot_dims % 2 or L.rot_dims > L.dim or (L.rot_dims and not L.rot_base > 0):
+                    raise ConfigError(f"{where}.mixer.left.rot: dims ({L.rot_dims}) must be even and at most dim ({L.dim}), base positive")
+                if min(L.memory_heads, L.memory_dim, L.memory_vdim) <= 0 or not L.gate_cap > 0:
+                    raise ConfigError(f"{where}.mixer.right: heads, dim, vdim and gate_cap must be positive")
+            if L.mlp_kind not in ("", "dense", "moe"):
+                raise ConfigError(f"{where}.mlp.kind {L.mlp_kind!r}: known are 'dense' and 'moe'")
+            if L.mlp_kind and (L.ff <= 0 or not L.limit > 0):
+                raise ConfigError(f"{where}.mlp: ff and limit must be positive")
+            if L.mlp_kind == "moe":
+                if L.experts <= 0 or L.group_count <= 0 or L.experts % L.group_count or not 0 < L.group_keep <= L.group_count:
+                    raise ConfigError(f"{where}.mlp.router.groups: {L.experts} experts do not form {L.group_count} groups of which {L.group_keep} are kept")
+                if not 0 < L.top <= L.group_keep * (L.experts // L.group_count):
+                    raise ConfigError(f"{where}.mlp.router: {L.group_keep} of {L.group_count} groups of {L.experts} experts cannot give top {L.top}")
+                if L.shared_ff < 0 or (L.shared_ff and not L.shared_limit > 0):
+                    raise ConfigError(f"{where}.mlp.shared: ff and limit must be positive")
+
+    @classmethod
+    def from_dict(cls, raw: dict[str, Any]) -> "GugidraConfig":
+        norm = raw.get("norm")
+        if not isinstance(norm, dict):
+            raise ConfigError("config.json: required key 'norm' (with 'eps') is missing")
+        layers_raw = raw.get("layers")
+        if not isinstance(layers_raw, (list, tuple)):
+            raise ConfigError("config.json: required key 'layers' is missing")
+        layers = []
+        for i, entry in enumerate(layers_raw):
+            where = f"layers[{i}]"
+            if not isinstance(entry, dict) or not isinstance(entry.get("mixer"), dict):
+                raise ConfigError(f"config.json: {where} needs 'type' and 'mixer'")
+            m, kind = entry["mixer"], str(entry.get("type"))
+            if kind == "gla":
+                fields = dict(kind=kind, heads=_require(m, "heads"), dim=_require(m, "dim"), vdim=_require(m, "vdim"),
+                              tau=_require(m, "tau", float), decay_rank=int(m.get("decay_rank") or 0))
+            elif kind == "parallel":
+                left, right = m.get("left"), m.get("right")
+                if not isinstance(left, dict) or not isinstance(right, dict):
+                    raise ConfigError(f"config.json: {where}.mixer needs 'left' and 'right'")
+                rot = left.get("rot") or {}
+                fields = dict(kind=kind, heads=_require(left, "heads"), dim=_require(left, "dim"), scale=_require(left, "scale", float))
+                fields.update(kv_heads=int(left.get("kv_heads") or fields["heads"]), vdim=int(left.get("vdim") or fields["dim"]),
+                              rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)),
+                              left_scale=float(m.get("left_scale", 1.0)), right_scale=float(m.get("right_scale", 1.0)),
+                              memory_heads=_require(right, "heads"), memory_dim=_require(right, "dim"),
+                              memory_vdim=_require(right, "vdim"), gate_cap=_require(right, "gate_cap", float))
+            else:
+                raise ConfigError(f"config.json: {where}.type {kind!r}: known are {', '.join(cls.KINDS)}")
+            mlp = entry.get("mlp")
+            if mlp is not None:
+                if not isinstance(mlp, dict):
+                    raise ConfigError(f"config.json: {where}.mlp must be an object or null")
+                fields["mlp_kind"] = str(mlp.get("kind", "dense"))
+                if fields["mlp_kind"] == "moe":
+                    expert, router = mlp.get("expert"), mlp.get("router")
+                    if not isinstance(expert, dict) or not isinstance(router, dict):
+                        raise ConfigError(f"config.json: {where}.mlp needs 'expert' and 'router'")
+                    groups, shared = router.get("groups") or {}, mlp.get("shared") or {}
+                    fields.update(ff=_require(expert, "ff"), limit=_require(expert, "limit", float), experts=_require(router, "experts"),
+                                  top=_require(router, "top"), group_count=int(groups.get("count", 1)), group_keep=int(groups.get("keep", 1)))
+                    if shared:
+                        fields.update(shared_ff=_require(shared, "ff"), shared_limit=_require(shared, "limit", float))
+                        _positive(f"{where}.mlp.shared.ff", fields["shared_ff"])
+                else:
+                    fields.update(ff=_require(mlp, "ff"), limit=_require(mlp, "limit", float))
+            layers.append(GugidraLayer(**fields))
+        loop, span = raw.get("loop"), {}
+        if loop is not None:
+            if not isinstance(loop, dict):
+                raise ConfigError("config.json: loop must be an object or null")
+            span = dict(loop_start=_require(loop, "start"), loop_stop=_require(loop, "stop"), loop_times=_require(loop, "times"))
+            _positive("loop.times", span["loop_times"])
+        return cls(vocab=_require(raw, "vocab"), width=_require(raw, "width"), norm_eps=_require(norm, "eps", float), layers=tuple(layers),
+                   embedding_scale=float((raw.get("embedding") or {}).get("scale", 1.0)), logit_softcap=float(raw.get("logit_softcap") or 0.0),
+                   **span)
+
+    def to_dict(self) -> dict[str, Any]:
+        layers = []
+        for L in self.layers:
+            if L.kind == "gla":
+                mixer = {"heads": L.heads, "dim": L.dim, "vdim": L.vdim, "tau": L.tau}
+                if L.decay_rank:
+                    mixer["decay_rank"] = L.decay_rank
+            else:
+                left = {"heads": L.heads, "kv_heads": L.kv_heads, "dim": L.dim, "vdim": L.vdim, "scale": L.scale,
+                        "rot": {"dims": L.rot_dims, "base": L.rot_base}}
+                right = {"heads": L.memory_heads, "dim": L.memory_dim, "vdim": L.memory_vdim, "gate_cap": L.gate_cap}
+                mixer = {"left": left, "right": right, "left_scale": L.left_scale, "right_scale": L.right_scale}
+            mlp = None
+            if L.mlp_kind == "dense":
+                mlp = {"kind": "dense", "ff": L.ff, "limit": L.limit}
+            elif L.mlp_kind == "moe":
+                mlp = {"kind": "moe", "expert": {"ff": L.ff, "limit": L.limit}, "router": {"experts": L.experts, "top": L.top}}
+                if L.group_count > 1:
+                    mlp["router"]["groups"] = {"count": L.group_count, "keep": L.group_keep}
+                if L.shared_ff:
+                    mlp["shared"] = {"ff": L.shared_ff, "limit": L.shared_limit}
+            layers.append({"type": L.kind, "mixer": mixer, "mlp": mlp})
+        out = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
+               "embedding": {"scale": self.embedding_scale}, "layers": layers}
+        if self.logit_softcap:
+            out["logit_softcap"] = self.logit_softcap
+        if self.has_loop():
+            out["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        return out
+
+    def has_loop(self) -> bool:
+        return self.loop_times > 0
+
+    def layer_order(self) -> list:
+        """(layer index, number of the pass that begins here or None) in the order the layers run."""
+        if not self.has_loop():
+            return [(i, None) for i in range(len(self.layers))]
+        order = [(i, None) for i in range(self.loop_start)]
+        for t in range(self.loop_times):
+            order += [(i, t if i == self.loop_start else None) for i in range(self.loop_start, self.loop_stop)]
+        return order + [(i, None) for i in range(self.loop_stop, len(self.layers))]
+
+    def needs_tensor_shapes(self) -> bool:
+        return any(L.kind == "gla" and not L.decay_rank for L in self.layers)
+
+    def with_tensor_shapes(self, shape_of) -> "GugidraConfig":
+        """The configuration with the sizes that only the weights give filled in; ``shape_of(name)`` returns the
+        shape of a checkpoint tensor (or None)."""
+        layers = []
+        for i, L in enumerate(self.layers):
+            if L.kind == "gla" and not L.decay_rank:
+                shape = shape_of(f"l{i}.mix.a1")
+                if shape is None or len(shape) != 2:
+                    raise ConfigError(f"config.json: layers[{i}] gives no decay_rank and the weights hold no l{i}.mix.a1 to read it from")
+                L = dataclasses.replace(L, decay_rank=int(shape[0]))
+            layers.append(L)
+        return dataclasses.replace(self, layers=tuple(layers))

@@ -223,6 +223,8 @@ PYRE_API int pyre_activation(const void* in, void* out, long long n, int kind, i
 //   proj [T, row_stride]: the token's projections; queries at column q_col (nh heads of dk), keys at
 //         k_col (nkv heads of dk), values at v_col (nkv heads of dv); k_col < 0: no keys or values (a layer
 //         that reads another layer's cache)
+//   q_b [nh dk], k_b [nkv dk], v_b [nkv dv] fp32 or null: added to the projections before anything else
+//         (v_col may equal k_col: a layer whose values are its keys before norm and rotation)
 //   q_w, k_w [dk] fp32 or null: the weight of the RMS norm over a head's dk dims (shared by all heads),
 //         n = (v * (1 / sqrt(mean(v^2) + eps))) * w; null: no norm
 //   rotation (pairs (j, j + rot / 2), j < rot / 2, after the norm):
@@ -236,6 +238,7 @@ PYRE_API int pyre_activation(const void* in, void* out, long long n, int kind, i
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void qk_norm_rope_write_kernel(const T* proj, long long row_stride, int q_col, int k_col, int v_col,
+                                          const float* q_b, const float* k_b, const float* v_b,
                                           const float* q_w, const float* k_w, float eps, const float* cos_t,
                                           const float* sin_t, const float* vcos_t, const float* vsin_t, T* q_out, T* cache,
                                           const int* slot_mapping, int n_tokens, int nh, int nkv, int dk, int dv, int D,
@@ -262,28 +265,31 @@ __global__ void qk_norm_rope_write_kernel(const T* proj, long long row_stride, i
     }
     if (!is_q && !is_k) {      // a value head: copied (or turned by its own tables), the rest of the row zero
         const T* src = in + v_col + (size_t)(h - nh - nkv) * dv;
+        const float* vb = v_b ? v_b + (size_t)(h - nh - nkv) * dv : nullptr;
+        auto val = [&](int d) -> float { return vb ? __fadd_rn(to_f32<T>(src[d]), vb[d]) : to_f32<T>(src[d]); };
         if (vcos_t) {
             const int vh = dv / 2;
             const float* ct = vcos_t + (size_t)t * vh;
             const float* st = vsin_t + (size_t)t * vh;
             for (int d = lane; d < D; d += 32) {
                 float o = 0.f;
-                if (d < vh) o = __fadd_rn(__fmul_rn(to_f32<T>(src[d]), ct[d]), __fmul_rn(-to_f32<T>(src[d + vh]), st[d]));
-                else if (d < 2 * vh) o = __fadd_rn(__fmul_rn(to_f32<T>(src[d]), ct[d - vh]), __fmul_rn(to_f32<T>(src[d - vh]), st[d - vh]));
-                else if (d < dv) o = to_f32<T>(src[d]);
+                if (d < vh) o = __fadd_rn(__fmul_rn(val(d), ct[d]), __fmul_rn(-val(d + vh), st[d]));
+                else if (d < 2 * vh) o = __fadd_rn(__fmul_rn(val(d), ct[d - vh]), __fmul_rn(val(d - vh), st[d - vh]));
+                else if (d < dv) o = val(d);
                 dst[d] = from_f32<T>(o);
             }
             return;
         }
-        for (int d = lane; d < D; d += 32) dst[d] = d < dv ? src[d] : from_f32<T>(0.f);
+        for (int d = lane; d < D; d += 32) dst[d] = from_f32<T>(d < dv ? val(d) : 0.f);
         return;
     }
     const T* src = in + (is_q ? q_col + (size_t)h * dk : k_col + (size_t)(h - nh) * dk);
     const float* w = is_q ? q_w : k_w;
+    const float* qkb = is_q ? (q_b ? q_b + (size_t)h * dk : nullptr) : (k_b ? k_b + (size_t)(h - nh) * dk : nullptr);
     float* n = head_smem + warp * D;
     float ss = 0.f;
     for (int d = lane; d < dk; d += 32) {
-        const float v = to_f32<T>(src[d]);
+        const float v = qkb ? __fadd_rn(to_f32<T>(src[d]), qkb[d]) : to_f32<T>(src[d]);
         n[d] = v;
         ss = fmaf(v, v, ss);
     }
@@ -328,7 +334,8 @@ __global__ void qk_norm_rope_write_kernel(const T* proj, long long row_stride, i
 // and every column multiples of 4, at most 256 entries a row): both entries of a pair lie in one lane, so a head goes
 // from one load to one store through registers.
 template <typename T>
-__global__ void qk_neighbours_write_kernel(const T* proj, long long row_stride, int q_col, int k_col, int v_col, float eps,
+__global__ void qk_neighbours_write_kernel(const T* proj, long long row_stride, int q_col, int k_col, int v_col,
+                                           const float* q_b, const float* k_b, const float* v_b, float eps,
                                            const float* cos_t, const float* sin_t, T* q_out, T* cache, const int* slot_mapping,
                                            int n_tokens, int nh, int nkv, int dk, int dv, int D, int rot, int post_norm, int page_size,
                                            long long n_pages, int* err_flag) {
@@ -341,15 +348,19 @@ __global__ void qk_neighbours_write_kernel(const T* proj, long long row_stride, 
     const int t = (int)(item / per_token), h = (int)(item - (long long)t * per_token);
     const bool is_q = h < nh, is_k = !is_q && h < nh + nkv;
     const T* src = proj + (size_t)t * row_stride;
+    const float* bias = nullptr;
     T* dst;
     if (is_q) {
         src += q_col + (size_t)h * dk;
+        if (q_b) bias = q_b + (size_t)h * dk;
         dst = q_out + ((size_t)t * nh + h) * D;
     } else {
         const int slot = (cache && slot_mapping) ? pyre_checked_slot(slot_mapping[t], n_pages, page_size, err_flag) : -1;
         if (slot < 0) return;
         const int page = slot / page_size, off = slot - page * page_size, kvh = is_k ? h - nh : h - nh - nkv;
         src += is_k ? k_col + (size_t)kvh * dk : v_col + (size_t)kvh * dv;
+        if (is_k && k_b) bias = k_b + (size_t)kvh * dk;
+        if (!is_k && v_b) bias = v_b + (size_t)kvh * dv;
         dst = cache + ((((size_t)page * 2 + (is_k ? 0 : 1)) * nkv + kvh) * page_size + off) * D;
     }
     const bool turn = is_q || is_k;
@@ -365,6 +376,11 @@ __global__ void qk_neighbours_write_kernel(const T* proj, long long row_stride, 
         const Vec<T, 4> in = load_vec<T, 4>(src + d);
 #pragma unroll
         for (int k = 0; k < 4; ++k) v[c][k] = to_f32<T>(in.v[k]);
+        if (bias) {
+            const Vec<float, 4> b = load_vec<float, 4>(bias + d);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) v[c][k] = __fadd_rn(v[c][k], b.v[k]);
+        }
         if (turn && d < rot) {
             const Vec<float, 2> cs = load_vec<float, 2>(cos_t + (size_t)t * (rot / 2) + d / 2), sn = load_vec<float, 2>(sin_t + (size_t)t * (rot / 2) + d / 2);
 #pragma unroll
@@ -391,6 +407,7 @@ __global__ void qk_neighbours_write_kernel(const T* proj, long long row_stride, 
 }
 
 PYRE_API int pyre_qk_norm_rope_write(const void* proj, long long row_stride, int q_col, int k_col, int v_col,
+                                     const float* q_b, const float* k_b, const float* v_b,
                                      const float* q_w, const float* k_w, float eps, const float* cos_t, const float* sin_t,
                                      const float* vcos_t, const float* vsin_t, void* q_out, void* cache, const int* slot_mapping, int n_tokens, int nh, int nkv,
                                      int dk, int dv, int D, int rot, int neighbours, int post_norm, int page_size, int dtype, long long n_pages,
@@ -407,19 +424,19 @@ PYRE_API int pyre_qk_norm_rope_write(const void* proj, long long row_stride, int
     const size_t smem = (size_t)warps * D * sizeof(float);
     const int kv_cols = k_col >= 0 ? k_col | v_col : 0;
     if (neighbours && !q_w && !k_w && !vcos_t && D <= 256 && ((dk | dv | D | rot | q_col | kv_cols | (int)(row_stride & 3)) & 3) == 0 &&
-        (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache | (uintptr_t)cos_t | (uintptr_t)sin_t) & 15) == 0 &&
-        (dtype == PYRE_BF16 || dtype == PYRE_F32)) {
+        (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache | (uintptr_t)cos_t | (uintptr_t)sin_t |
+          (uintptr_t)q_b | (uintptr_t)k_b | (uintptr_t)v_b) & 15) == 0 && (dtype == PYRE_BF16 || dtype == PYRE_F32)) {
         if (dtype == PYRE_BF16)
-            pyre_launch(qk_neighbours_write_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), 0, stream, (const __nv_bfloat16*)proj, row_stride, q_col, k_col, v_col, eps, cos_t, sin_t, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, post_norm, page_size, n_pages, err_flag);
+            pyre_launch(qk_neighbours_write_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), 0, stream, (const __nv_bfloat16*)proj, row_stride, q_col, k_col, v_col, q_b, k_b, v_b, eps, cos_t, sin_t, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, post_norm, page_size, n_pages, err_flag);
         else
-            pyre_launch(qk_neighbours_write_kernel<float>, dim3(blocks), dim3(warps * 32), 0, stream, (const float*)proj, row_stride, q_col, k_col, v_col, eps, cos_t, sin_t, (float*)q_out, (float*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, post_norm, page_size, n_pages, err_flag);
+            pyre_launch(qk_neighbours_write_kernel<float>, dim3(blocks), dim3(warps * 32), 0, stream, (const float*)proj, row_stride, q_col, k_col, v_col, q_b, k_b, v_b, eps, cos_t, sin_t, (float*)q_out, (float*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, post_norm, page_size, n_pages, err_flag);
         PYRE_LAUNCH_CHECK();
         return 0;
     }
     if (dtype == PYRE_BF16)
-        pyre_launch(qk_norm_rope_write_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, stream, (const __nv_bfloat16*)proj, row_stride, q_col, k_col, v_col, q_w, k_w, eps, cos_t, sin_t, vcos_t, vsin_t, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, neighbours, post_norm, page_size, n_pages, err_flag);
+        pyre_launch(qk_norm_rope_write_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, stream, (const __nv_bfloat16*)proj, row_stride, q_col, k_col, v_col, q_b, k_b, v_b, q_w, k_w, eps, cos_t, sin_t, vcos_t, vsin_t, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, neighbours, post_norm, page_size, n_pages, err_flag);
     else if (dtype == PYRE_F32)
-        pyre_launch(qk_norm_rope_write_kernel<float>, dim3(blocks), dim3(warps * 32), smem, stream, (const float*)proj, row_stride, q_col, k_col, v_col, q_w, k_w, eps, cos_t, sin_t, vcos_t, vsin_t, (float*)q_out, (float*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, neighbours, post_norm, page_size, n_pages, err_flag);
+        pyre_launch(qk_norm_rope_write_kernel<float>, dim3(blocks), dim3(warps * 32), smem, stream, (const float*)proj, row_stride, q_col, k_col, v_col, q_b, k_b, v_b, q_w, k_w, eps, cos_t, sin_t, vcos_t, vsin_t, (float*)q_out, (float*)cache, slot_mapping, n_tokens, nh, nkv, dk, dv, D, rot, neighbours, post_norm, page_size, n_pages, err_flag);
     else return PYRE_ERR_BAD_ARG;
     PYRE_LAUNCH_CHECK();
     return 0;
@@ -428,11 +445,12 @@ PYRE_API int pyre_qk_norm_rope_write(const void* proj, long long row_stride, int
 // ---------------------------------------------------------------------------
 // A sigmoid gate on a mixer's heads: out[t, h, j] = a[t, h, j] * sigmoid(gate[t, h, j]) for j < dv, where a
 // head of `a` has a_dim >= dv columns (the rest is dropped) and the gate lies in the token's projection row
-// at column g_col (g_col < 0: no gate, the heads are only narrowed to dv columns).
+// at column g_col (g_col < 0: no gate, the heads are only narrowed to dv columns).  Everything is multiplied by `scale`; a
+// row of `out` starts out_stride elements after the one before (the heads of a mixer beside those of another one).
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void sigmoid_gate_kernel(const T* a, int a_dim, const T* proj, long long row_stride, int g_col, T* out,
-                                    int n_tokens, int nh, int dv) {
+                                    long long out_stride, float scale, int n_tokens, int nh, int dv) {
     pdl_trigger();
     pdl_wait();
     const size_t n = (size_t)n_tokens * nh * dv, stride = (size_t)gridDim.x * blockDim.x;
@@ -440,14 +458,14 @@ __global__ void sigmoid_gate_kernel(const T* a, int a_dim, const T* proj, long l
         const size_t t = i / ((size_t)nh * dv);
         const int c = (int)(i - t * nh * dv), h = c / dv, j = c - h * dv;
         const float g = g_col >= 0 ? act_sigmoid(to_f32<T>(proj[t * row_stride + g_col + c])) : 1.0f;
-        out[i] = from_f32<T>(to_f32<T>(a[(t * nh + h) * a_dim + j]) * g);
+        out[t * out_stride + c] = from_f32<T>(to_f32<T>(a[(t * nh + h) * a_dim + j]) * g * scale);
     }
 }
 
 // the same in vectors of VEC elements along a head (dv, a_dim, g_col and row_stride multiples of VEC, aligned pointers)
 template <typename T, int VEC>
 __global__ void sigmoid_gate_vec_kernel(const T* a, int a_dim, const T* proj, long long row_stride, int g_col, T* out,
-                                        int n_tokens, int nh, int dv) {
+                                        long long out_stride, float scale, int n_tokens, int nh, int dv) {
     pdl_trigger();
     pdl_wait();
     const int per_head = dv / VEC;
@@ -459,28 +477,31 @@ __global__ void sigmoid_gate_vec_kernel(const T* a, int a_dim, const T* proj, lo
         if (g_col >= 0) {
             const Vec<T, VEC> gt = load_vec<T, VEC>(proj + t * row_stride + g_col + h * dv + j);
 #pragma unroll
-            for (int k = 0; k < VEC; ++k) o.v[k] = from_f32<T>(to_f32<T>(v.v[k]) * act_sigmoid(to_f32<T>(gt.v[k])));
+            for (int k = 0; k < VEC; ++k) o.v[k] = from_f32<T>(to_f32<T>(v.v[k]) * act_sigmoid(to_f32<T>(gt.v[k])) * scale);
+        } else if (scale != 1.0f) {
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) o.v[k] = from_f32<T>(to_f32<T>(v.v[k]) * scale);
         } else {
             o = v;
         }
-        store_vec<T, VEC>(out + (t * nh + h) * dv + j, o);
+        store_vec<T, VEC>(out + t * out_stride + h * dv + j, o);
     }
 }
 
 PYRE_API int pyre_sigmoid_gate(const void* a, int a_dim, const void* proj, long long row_stride, int g_col, void* out,
-                               int n_tokens, int nh, int dv, int dtype, cudaStream_t stream) {
+                               long long out_stride, float scale, int n_tokens, int nh, int dv, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (a_dim < dv || dv <= 0 || nh <= 0 || (g_col >= 0 && !proj)) return PYRE_ERR_BAD_ARG;
+    if (a_dim < dv || dv <= 0 || nh <= 0 || (g_col >= 0 && !proj) || out_stride < (long long)nh * dv) return PYRE_ERR_BAD_ARG;
     {
         const int vec = dtype == PYRE_BF16 ? 8 : 4;
-        if (dv % vec == 0 && a_dim % vec == 0 && (g_col < 0 || (g_col % vec == 0 && row_stride % vec == 0)) &&
+        if (dv % vec == 0 && a_dim % vec == 0 && out_stride % vec == 0 && (g_col < 0 || (g_col % vec == 0 && row_stride % vec == 0)) &&
             (((uintptr_t)a | (uintptr_t)out | (uintptr_t)proj) & 15) == 0 && (dtype == PYRE_BF16 || dtype == PYRE_F32)) {
             const long long items = (long long)n_tokens * nh * (dv / vec);
             const int blocks = (int)min((long long)148 * 16, ceil_div_ll(items, 256));
             if (dtype == PYRE_BF16)
-                pyre_launch(sigmoid_gate_vec_kernel<__nv_bfloat16, 8>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)a, a_dim, (const __nv_bfloat16*)proj, row_stride, g_col, (__nv_bfloat16*)out, n_tokens, nh, dv);
+                pyre_launch(sigmoid_gate_vec_kernel<__nv_bfloat16, 8>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)a, a_dim, (const __nv_bfloat16*)proj, row_stride, g_col, (__nv_bfloat16*)out, out_stride, scale, n_tokens, nh, dv);
             else
-                pyre_launch(sigmoid_gate_vec_kernel<float, 4>, dim3(blocks), dim3(256), 0, stream, (const float*)a, a_dim, (const float*)proj, row_stride, g_col, (float*)out, n_tokens, nh, dv);
+                pyre_launch(sigmoid_gate_vec_kernel<float, 4>, dim3(blocks), dim3(256), 0, stream, (const float*)a, a_dim, (const float*)proj, row_stride, g_col, (float*)out, out_stride, scale, n_tokens, nh, dv);
             PYRE_LAUNCH_CHECK();
             return 0;
         }
@@ -488,9 +509,9 @@ PYRE_API int pyre_sigmoid_gate(const void* a, int a_dim, const void* proj, long 
     const long long n = (long long)n_tokens * nh * dv;
     const int blocks = (int)min((long long)4096, ceil_div_ll(n, 256));
     if (dtype == PYRE_BF16)
-        pyre_launch(sigmoid_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)a, a_dim, (const __nv_bfloat16*)proj, row_stride, g_col, (__nv_bfloat16*)out, n_tokens, nh, dv);
+        pyre_launch(sigmoid_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)a, a_dim, (const __nv_bfloat16*)proj, row_stride, g_col, (__nv_bfloat16*)out, out_stride, scale, n_tokens, nh, dv);
     else if (dtype == PYRE_F32)
-        pyre_launch(sigmoid_gate_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)a, a_dim, (const float*)proj, row_stride, g_col, (float*)out, n_tokens, nh, dv);
+        pyre_launch(sigmoid_gate_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)a, a_dim, (const float*)proj, row_stride, g_col, (float*)out, out_stride, scale, n_tokens, nh, dv);
     else return PYRE_ERR_BAD_ARG;
     PYRE_LAUNCH_CHECK();
     return 0;

@@ -201,5 +201,8 @@ __device__ __forceinline__ int pyre_checked_page(int page, long long, int*) { re
 __device__ __forceinline__ int pyre_checked_slot(int slot, long long, int, int*) { return slot; }
 #endif
 
+// The clamped gate of a feed-forward: z sigmoid(CLAMPED_GLU_SLOPE z) (u + 1) for z = min(gate, limit), u = clamp(up, -limit, limit)
+constexpr float CLAMPED_GLU_SLOPE = 1.702f;
+
 static inline int ceil_div(int a, int b) { return (a + b - 1) / b; }
 static inline long long ceil_div_ll(long long a, long long b) { return (a + b - 1) / b; }

@@ -455,10 +455,11 @@ PYRE_API int pyre_qkv_rope_write(const void* qkv, const float* partials, int n_p
 }
 
 // ---------------------------------------------------------------------------
-// out[t, i] = act(gu[t, i]) * gu[t, I + i] in fp32; act: silu, z / (1 + exp(-z)), or (relu) max(z, 0).
+// out[t, i] = act(gu[t, i]) * gu[t, I + i] in fp32; kind 0: silu, z / (1 + exp(-z)); 1: relu, max(z, 0); 2: the clamped form
+// z sigmoid(1.702 z) (u + 1) with z = min(gate, limit), u = clamp(up, -limit, limit).
 // ---------------------------------------------------------------------------
 template <typename T, int VEC>
-__global__ void silu_mul_kernel(const T* gu, T* out, int n_tokens, int I, int block, int relu) {
+__global__ void silu_mul_kernel(const T* gu, T* out, int n_tokens, int I, int block, int kind, float limit) {
     pdl_trigger();
     pdl_wait();
     const size_t per_row = (size_t)(I / VEC);
@@ -475,9 +476,13 @@ __global__ void silu_mul_kernel(const T* gu, T* out, int n_tokens, int I, int bl
         Vec<T, VEC> o;
 #pragma unroll
         for (int k = 0; k < VEC; ++k) {
-            const float z = to_f32<T>(g.v[k]);
-            const float s = relu ? fmaxf(z, 0.f) : z / (1.0f + expf(-z));
-            o.v[k] = from_f32<T>(__fmul_rn(s, to_f32<T>(u.v[k])));
+            float z = to_f32<T>(g.v[k]), up = to_f32<T>(u.v[k]);
+            if (kind == 2) {
+                z = fminf(z, limit);
+                up = fminf(fmaxf(up, -limit), limit) + 1.0f;
+            }
+            const float s = kind == 1 ? fmaxf(z, 0.f) : z / (1.0f + expf(kind == 2 ? -CLAMPED_GLU_SLOPE * z : -z));
+            o.v[k] = from_f32<T>(__fmul_rn(s, up));
         }
         store_vec<T, VEC>(out + t * (size_t)I + i, o);
     }
@@ -485,15 +490,17 @@ __global__ void silu_mul_kernel(const T* gu, T* out, int n_tokens, int I, int bl
 
 // block: 0 for gate_up = [gates | ups]; n > 0 for gates and ups interleaved in blocks of n features
 // (n a multiple of 8 that divides I).
-PYRE_API int pyre_silu_mul(const void* gu, void* out, int n_tokens, int I, int block, int relu, int dtype, cudaStream_t stream) {
+PYRE_API int pyre_silu_mul(const void* gu, void* out, int n_tokens, int I, int block, int kind, float limit, int dtype,
+                           cudaStream_t stream) {
     if (n_tokens <= 0 || I <= 0) return 0;
+    if (kind < 0 || kind > 2 || (kind == 2 && !(limit > 0.f))) return PYRE_ERR_BAD_ARG;
     if (block < 0 || (block > 0 && (block % 8 || I % block))) return PYRE_ERR_BAD_ARG;
     const int threads = 256;
 #define LAUNCH(TT, V)                                                                                      \
     do {                                                                                                   \
         long long total = (long long)n_tokens * (I / V);                                                   \
         int blocks = (int)min((long long)pyre_sm_count() * 16, ceil_div_ll(total, threads));                           \
-        pyre_launch(silu_mul_kernel<TT, V>, dim3(blocks), dim3(threads), 0, stream, (const TT*)gu, (TT*)out, n_tokens, I, block, relu);      \
+        pyre_launch(silu_mul_kernel<TT, V>, dim3(blocks), dim3(threads), 0, stream, (const TT*)gu, (TT*)out, n_tokens, I, block, kind, limit);      \
     } while (0)
     if (dtype == PYRE_F32) { if (I % 4 == 0) LAUNCH(float, 4); else LAUNCH(float, 1); }
     else if (dtype == PYRE_BF16) { if (I % 8 == 0) LAUNCH(__nv_bfloat16, 8); else if (I % 4 == 0) LAUNCH(__nv_bfloat16, 4); else LAUNCH(__nv_bfloat16, 1); }

@@ -175,7 +175,9 @@ struct GemmParams {
     int out_f32;
     int x_is_constant;            // 1: X holds weights (may be loaded before the kernels before this one finish); 0: Y does
     int gated;                    // 1: the weight rows are gate/up rows interleaved in blocks of 64 (gate rows, then the up
-                                  // rows of the same features); the epilogue writes silu(gate) * up (2: relu(gate) * up), half as many features
+                                  // rows of the same features); the epilogue writes silu(gate) * up (2: relu(gate) * up; 3: the clamped
+                                  // form with gate_limit, see gated_value), half as many features
+    float gate_limit;
     int act;                      // 1 (row store, one split, bf16 out, FOLD == 1 variants): out = gelu_tanh(product), applied to the
                                   // product rounded to bfloat16, as an activation kernel of its own would read it
     int* err_flag;
@@ -241,8 +243,15 @@ struct SmemLayout {
 // drains its own 128 accumulator rows.  Barriers: the first CTA's "full" barriers count the bytes of both CTAs'
 // loads; the MMA commits arrive on the "empty" and "accumulator full" barriers of both; the epilogue warps of
 // both arrive on the first CTA's "accumulator empty" barriers.
-// the activation of a gated product: gate 1 silu, 2 relu
-__device__ __forceinline__ float gate_of(float z, int gate) { return gate == 2 ? fmaxf(z, 0.f) : z / (1.0f + expf(-z)); }
+// one output of a gated product from its gate z and up v: gate 1 silu(z) v, 2 relu(z) v, 3 (clamped) z' sigmoid(1.702 z') (v' + 1)
+// with z' = min(z, limit), v' = clamp(v, -limit, limit)
+__device__ __forceinline__ float gated_value(float z, float v, int gate, float limit) {
+    if (gate == 3) {
+        z = fminf(z, limit);
+        v = fminf(fmaxf(v, -limit), limit) + 1.0f;
+    }
+    return __fmul_rn(gate == 2 ? fmaxf(z, 0.f) : z / (1.0f + expf(gate == 3 ? -CLAMPED_GLU_SLOPE * z : -z)), v);
+}
 
 // the tanh form of gelu on a product that is rounded to bfloat16 first: 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
 __device__ __forceinline__ float gelu_tanh_of_bf16(float acc) {
@@ -555,7 +564,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                                 for (int e = 0; e < 2; ++e) {
                                     const float z = __bfloat162float(__float2bfloat16_rn(__uint_as_float(g[2 * q + e]) * row_scale));
                                     const float v = __bfloat162float(__float2bfloat16_rn(__uint_as_float(u[2 * q + e]) * row_scale));
-                                    o[e] = __fmul_rn(gate_of(z, p.gated), v);
+                                    o[e] = gated_value(z, v, p.gated, p.gate_limit);
                                 }
                                 __nv_bfloat162 pr = __floats2bfloat162_rn(o[0], o[1]);
                                 w[cc / 2 + q] = *reinterpret_cast<uint32_t*>(&pr);
@@ -607,7 +616,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                                         const float z = __bfloat162float(__float2bfloat16_rn(__uint_as_float(r[4 * q4 + e]) * rs));
                                         const float v = __bfloat162float(__float2bfloat16_rn(uu[e] * rs));
                                         ((__nv_bfloat16*)p.out)[(long long)y * p.stride_y + feature] =
-                                            __float2bfloat16_rn(__fmul_rn(gate_of(z, p.gated), v));
+                                            __float2bfloat16_rn(gated_value(z, v, p.gated, p.gate_limit));
                                     }
                                 }
                             }
@@ -1148,7 +1157,7 @@ int launch_rows(const CUtensorMap& mx, const CUtensorMap& my, const GemmParams& 
 // which operand holds weights: its first tiles are fetched before the kernel waits for the
 // kernels before it in the stream (programmatic dependent launch).  gated: the weight operand holds gate
 // and up rows interleaved in blocks of 64 (64 gate rows, the up rows of the same features, ...); the output is
-// silu(gate product) * (up product) (gated == 3: relu), half as many features: row store (weights = Y, bn 256, out[x, j]) or
+// silu(gate product) * (up product) (gated == 3: relu; 4: the clamped form), half as many features: row store (weights = Y, bn 256, out[x, j]) or
 // transposed store (weights = X, bn <= 128, out[y * stride_y + j]); one split, bf16 out.  pair: two CTAs of a
 // cluster share each 256 x bn tile (row store, bn 128, 160, 192, 208, 224 or 256).
 //
@@ -1179,14 +1188,15 @@ struct PyreGemmFix {
 
 static int gemm_tc_impl(const void* X, int x_rows, long long ldx, const void* Y, int y_rows, long long ldy, int K,
                         void* out, int out_f32, long long stride_x, long long stride_y, long long split_stride,
-                        int splits, int bn, int x_is_constant, int gated, int pair, int* err_flag, const PyreGemmFix* fx,
+                        int splits, int bn, int x_is_constant, int gated, float gate_limit, int pair, int* err_flag, const PyreGemmFix* fx,
                         cudaStream_t stream) {
     if (x_rows <= 0 || y_rows <= 0) return 0;
     // gated == 2: no gate, but gelu_tanh on the product, in the epilogue of a row store of one split (bf16 out)
     // gated == 3: the gate's activation is relu instead of silu
-    if (gated < 0 || gated > 3) return PYRE_ERR_BAD_ARG;
+    // gated == 4: the clamped form (gated_value's gate 3) with gate_limit
+    if (gated < 0 || gated > 4 || (gated == 4 && !(gate_limit > 0.f))) return PYRE_ERR_BAD_ARG;
     const int act = gated == 2 ? 1 : 0;
-    const int gate = gated == 3 ? 2 : 1;
+    const int gate = gated == 4 ? 3 : gated == 3 ? 2 : 1;
     if (act) {
         gated = 0;
         if (splits != 1 || out_f32 || stride_y != 1 || stride_x == 1 || (fx && fx->fix != 0)) return PYRE_ERR_BAD_ARG;
@@ -1243,7 +1253,7 @@ static int gemm_tc_impl(const void* X, int x_rows, long long ldx, const void* Y,
     p.x_rows = x_rows; p.y_rows = y_rows; p.K = K;
     p.k_blocks_per_split = (total_kb + splits - 1) / splits;
     p.stride_x = stride_x; p.stride_y = stride_y; p.split_stride = split_stride;
-    p.out = out; p.out_f32 = out_f32; p.x_is_constant = x_is_constant; p.err_flag = err_flag; p.gated = gated ? gate : 0; p.act = act;
+    p.out = out; p.out_f32 = out_f32; p.x_is_constant = x_is_constant; p.err_flag = err_flag; p.gated = gated ? gate : 0; p.gate_limit = gate_limit; p.act = act;
     p.scale_ssq = nullptr; p.scale_tiles = 0; p.scale_n = 0.f; p.scale_eps = 0.f; p.fix = 0; p.tile_counters = nullptr;
     p.resid = nullptr; p.norm_w = nullptr; p.h_out = nullptr; p.ssq_out = nullptr; p.bias = nullptr; p.cos_t = p.sin_t = nullptr;
     p.q_out = nullptr; p.kv_cache = nullptr; p.slot_mapping = nullptr; p.nh = p.nkv = p.hd = p.rot = p.page_size = 0; p.n_pages = 0;
@@ -1324,8 +1334,8 @@ static int gemm_tc_impl(const void* X, int x_rows, long long ldx, const void* Y,
 
 PYRE_API int pyre_gemm_tc(const void* X, int x_rows, long long ldx, const void* Y, int y_rows, long long ldy, int K,
                           void* out, int out_f32, long long stride_x, long long stride_y, long long split_stride,
-                          int splits, int bn, int x_is_constant, int gated, int pair, int* err_flag,
+                          int splits, int bn, int x_is_constant, int gated, float gate_limit, int pair, int* err_flag,
                           const PyreGemmFix* fx, cudaStream_t stream) {
     return gemm_tc_impl(X, x_rows, ldx, Y, y_rows, ldy, K, out, out_f32, stride_x, stride_y, split_stride, splits, bn,
-                        x_is_constant, gated, pair, err_flag, fx, stream);
+                        x_is_constant, gated, gate_limit, pair, err_flag, fx, stream);
 }

@@ -376,14 +376,18 @@ PYRE_API int pyre_grouped_linear(const void* x, long long x_row_stride, long lon
 // with the largest choice scores are chosen (the lowest index wins a tie), and each chosen output's weight is its
 // plain score s times `scale` (not renormalised).  `sigmoid` != 0: the scores are s = sigmoid(z), each output by itself,
 // instead of the softmax.  `bias` (fp32 [n_out] or null) is added to the logits before anything else.  `renorm` != 0: the
-// chosen outputs' weights are divided by their sum (with softmax scores: the softmax over the chosen logits alone).
+// chosen outputs' weights are divided by their sum + renorm_eps (with softmax scores: the softmax over the chosen logits alone).
+// `groups` > 1: the outputs form so many equal groups of neighbours; a group's score is the sum of its two largest choice
+// scores (of its one, if it has only one), and only outputs of the `keep` groups with the largest scores (the lowest index
+// wins a tie) can be chosen.
 // One block per token, one warp per output in turn.
 //   idx_out [T, top] int32, weight_out [T, top] fp32
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void route_kernel(const T* h, const float* w, const float* correction, const float* bias, int* idx_out,
-                             float* weight_out, int H, int n_out, int top, float scale, int sigmoid, int renorm) {
-    extern __shared__ float z_smem[];   // [n_out] logits, then scores; [n_out] choice scores
+                             float* weight_out, int H, int n_out, int top, float scale, int sigmoid, int renorm, float renorm_eps,
+                             int groups, int keep) {
+    extern __shared__ float z_smem[];   // [n_out] logits, then scores; [n_out] choice scores; [groups] group scores
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -433,6 +437,27 @@ __global__ void route_kernel(const T* h, const float* w, const float* correction
             choice[e] = s + (correction ? correction[e] : 0.f);
         }
         __syncwarp();
+        if (groups > 1) {
+            const int size = n_out / groups;
+            float* gs = choice + n_out;
+            for (int g = lane; g < groups; g += 32) {
+                float first = -INFINITY, second = -INFINITY;
+                for (int e = g * size; e < (g + 1) * size; ++e) {
+                    const float c = choice[e];
+                    if (c > first) { second = first; first = c; }
+                    else if (c > second) second = c;
+                }
+                gs[g] = size > 1 ? first + second : first;
+            }
+            __syncwarp();
+            for (int g = lane; g < groups; g += 32) {      // a group stays if fewer than `keep` groups come before it
+                int before = 0;
+                for (int o = 0; o < groups; ++o) before += (gs[o] > gs[g] || (gs[o] == gs[g] && o < g)) ? 1 : 0;
+                if (before >= keep)
+                    for (int e = g * size; e < (g + 1) * size; ++e) choice[e] = -INFINITY;
+            }
+            __syncwarp();
+        }
         for (int k = 0; k < top; ++k) {
             float best = -INFINITY;
             int at = 0x7fffffff;
@@ -446,6 +471,7 @@ __global__ void route_kernel(const T* h, const float* w, const float* correction
                 const int oa = __shfl_xor_sync(0xffffffffu, at, o);
                 if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
             }
+            if (at >= n_out) at = 0;      // scores that are no numbers choose nothing
             if (lane == 0) {
                 idx_out[(size_t)t * top + k] = at;
                 weight_out[(size_t)t * top + k] = z[at] * scale;
@@ -456,24 +482,26 @@ __global__ void route_kernel(const T* h, const float* w, const float* correction
         if (renorm && lane == 0) {
             float total = 0.f;
             for (int k = 0; k < top; ++k) total += weight_out[(size_t)t * top + k];
-            for (int k = 0; k < top; ++k) weight_out[(size_t)t * top + k] = weight_out[(size_t)t * top + k] / total;
+            for (int k = 0; k < top; ++k) weight_out[(size_t)t * top + k] = weight_out[(size_t)t * top + k] / (total + renorm_eps);
         }
     }
 }
 
 PYRE_API int pyre_route(const void* h, const float* w, const float* correction, const float* bias, int* idx_out, float* weight_out,
-                        int n_tokens, int H, int n_out, int top, float scale, int sigmoid, int renorm, int dtype, cudaStream_t stream) {
+                        int n_tokens, int H, int n_out, int top, float scale, int sigmoid, int renorm, float renorm_eps, int groups,
+                        int keep, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (H <= 0 || n_out <= 0 || top <= 0 || top > n_out) return PYRE_ERR_BAD_ARG;
-    const size_t smem = (size_t)2 * n_out * sizeof(float);
+    if (groups < 0 || (groups > 1 && (n_out % groups || keep <= 0 || top > (long long)keep * (n_out / groups)))) return PYRE_ERR_BAD_ARG;
+    const size_t smem = ((size_t)2 * n_out + max(groups, 0)) * sizeof(float);
     if (smem > 48 * 1024) return PYRE_ERR_UNSUPPORTED;
     const int threads = n_tokens >= 512 ? 256 : 1024;      // few tokens: more warps per token's outputs
     if (dtype == PYRE_BF16)
         pyre_launch(route_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), smem, stream, (const __nv_bfloat16*)h, w, correction,
-                    bias, idx_out, weight_out, H, n_out, top, scale, sigmoid, renorm);
+                    bias, idx_out, weight_out, H, n_out, top, scale, sigmoid, renorm, renorm_eps, groups, keep);
     else if (dtype == PYRE_F32)
         pyre_launch(route_kernel<float>, dim3(n_tokens), dim3(threads), smem, stream, (const float*)h, w, correction, bias, idx_out,
-                    weight_out, H, n_out, top, scale, sigmoid, renorm);
+                    weight_out, H, n_out, top, scale, sigmoid, renorm, renorm_eps, groups, keep);
     else return PYRE_ERR_BAD_ARG;
     PYRE_LAUNCH_CHECK();
     return 0;

@@ -211,7 +211,8 @@ PYRE_API int pyre_scaled_sum(const void* y0, const float* p0, int n0, const floa
 // ---------------------------------------------------------------------------
 // out[r, i] = act(gu[r, i]) * gu[r, I + i]: the elementwise half of a gated feed-forward whose product left
 // [gates | ups] per row.  kind 0: silu, z / (1 + exp(-z)); kind 1: the tanh form of gelu,
-// 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))); kind 2: relu, max(z, 0).
+// 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))); kind 2: relu, max(z, 0); kind 3: the clamped form
+// z sigmoid(1.702 z) (u + 1) with z = min(gate, limit), u = clamp(up, -limit, limit).
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ float gate_act(float z, int kind) {
     if (kind == 0) return z / (1.0f + expf(-z));
@@ -220,31 +221,45 @@ __device__ __forceinline__ float gate_act(float z, int kind) {
     return 0.5f * z * (1.0f + tanhf(u));
 }
 
-template <typename T>
-__global__ void act_mul_kernel(const T* gu, T* out, size_t n_rows, int I, int kind) {
+__device__ __forceinline__ float gated_pair(float z, float u, int kind, float limit) {
+    if (kind == 3) {
+        z = fminf(z, limit);
+        return __fmul_rn(z / (1.0f + expf(-CLAMPED_GLU_SLOPE * z)), fminf(fmaxf(u, -limit), limit) + 1.0f);
+    }
+    return __fmul_rn(gate_act(z, kind), u);
+}
+
+// VEC neighbouring features per thread (I a multiple of VEC, pointers aligned)
+template <typename T, int VEC>
+__global__ void act_mul_kernel(const T* gu, T* out, size_t n_rows, int I, int kind, float limit) {
     pdl_trigger();
     pdl_wait();
-    const size_t total = n_rows * (size_t)I;
+    const size_t per_row = (size_t)(I / VEC), total = n_rows * per_row;
     const size_t stride = (size_t)gridDim.x * blockDim.x;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += stride) {
-        const size_t r = idx / I;
-        const int i = (int)(idx - r * I);
+        const size_t r = idx / per_row;
+        const int i = (int)(idx - r * per_row) * VEC;
         const T* row = gu + r * (size_t)(2 * I);
-        out[idx] = from_f32<T>(__fmul_rn(gate_act(to_f32<T>(row[i]), kind), to_f32<T>(row[I + i])));
+        const Vec<T, VEC> g = load_vec<T, VEC>(row + i), u = load_vec<T, VEC>(row + I + i);
+        Vec<T, VEC> o;
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) o.v[k] = from_f32<T>(gated_pair(to_f32<T>(g.v[k]), to_f32<T>(u.v[k]), kind, limit));
+        store_vec<T, VEC>(out + r * (size_t)I + i, o);
     }
 }
 
-PYRE_API int pyre_act_mul(const void* gu, void* out, int n_rows, int I, int kind, int dtype, cudaStream_t stream) {
+PYRE_API int pyre_act_mul(const void* gu, void* out, int n_rows, int I, int kind, float limit, int dtype, cudaStream_t stream) {
     if (n_rows <= 0 || I <= 0) return 0;
-    if (kind < 0 || kind > 2) return PYRE_ERR_BAD_ARG;
-    const long long total = (long long)n_rows * I;
+    if (kind < 0 || kind > 3 || (kind == 3 && !(limit > 0.f))) return PYRE_ERR_BAD_ARG;
+    const int vec = dtype == PYRE_BF16 ? 8 : 4;
+    const bool wide = I % vec == 0 && aligned16({gu, out});
+    const long long total = (long long)n_rows * (wide ? I / vec : I);
     const int blocks = (int)min((long long)pyre_sm_count() * 16, ceil_div_ll(total, 256));
-    if (dtype == PYRE_BF16)
-        pyre_launch(act_mul_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out,
-                    (size_t)n_rows, I, kind);
-    else if (dtype == PYRE_F32)
-        pyre_launch(act_mul_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, (float*)out, (size_t)n_rows, I, kind);
+#define LAUNCH(T, V) pyre_launch(act_mul_kernel<T, V>, dim3(blocks), dim3(256), 0, stream, (const T*)gu, (T*)out, (size_t)n_rows, I, kind, limit)
+    if (dtype == PYRE_BF16) { if (wide) LAUNCH(__nv_bfloat16, 8); else LAUNCH(__nv_bfloat16, 1); }
+    else if (dtype == PYRE_F32) { if (wide) LAUNCH(float, 4); else LAUNCH(float, 1); }
     else return PYRE_ERR_BAD_ARG;
+#undef LAUNCH
     PYRE_LAUNCH_CHECK();
     return 0;
 }

@@ -58,12 +58,20 @@ class StepContext:
     feed_src: "torch.Tensor | None" = None
     entries: list = field(default_factory=list)
     new_lens: list = field(default_factory=list)
+    _lengths: "list | None" = None
 
     def kv_group(self, index: int) -> KVView:
         return self.kv_groups[index]
 
     def state_group(self, index: int) -> StateView:
         return self.state_groups[index]
+
+    @property
+    def entry_lengths(self) -> list:
+        """Tokens that each entry brings."""
+        if self._lengths is None:
+            self._lengths = np.diff(self.cu_seqlens_host).tolist()
+        return self._lengths
 
     @property
     def max_new_tokens_per_seq(self) -> int:

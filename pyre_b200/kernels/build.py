@@ -42,6 +42,7 @@ LIBRARIES = {
     "grouped": "grouped.cu",
     "wkv": "wkv.cu",
     "seqmix": "seqmix.cu",
+    "matrix_state": "matrix_state.cu",
 }
 
 HEADERS = ["common.cuh", "attention_mma_noalloc.h"]

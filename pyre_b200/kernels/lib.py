@@ -30,11 +30,11 @@ SIGNATURES: dict[str, tuple[str, list]] = {
     "pyre_add_residual": ("elementwise", [P, P, LL, I, P]),
     "pyre_rope_table": ("elementwise", [P, P, P, P, I, I, P]),
     "pyre_qkv_rope_write": ("elementwise", [P, P, I, LL, P, P, P, P, P, P, I, I, I, I, I, I, I, LL, P, P]),
-    "pyre_silu_mul": ("elementwise", [P, P, I, I, I, I, I, P]),
+    "pyre_silu_mul": ("elementwise", [P, P, I, I, I, I, F, I, P]),
     "pyre_sum_partials": ("elementwise", [P, I, LL, P, LL, I, P]),
     "pyre_feed_tokens": ("elementwise", [P, P, P, P, I, P]),
     "pyre_delay": ("elementwise", [LL, P]),
-    "pyre_gemm_tc": ("gemm_tc", [P, I, LL, P, I, LL, I, P, I, LL, LL, LL, I, I, I, I, I, P, P, P]),
+    "pyre_gemm_tc": ("gemm_tc", [P, I, LL, P, I, LL, I, P, I, LL, LL, LL, I, I, I, I, F, I, P, P, P]),
     "pyre_scale_rows": ("elementwise", [P, P, I, P, I, I, F, P]),
     "pyre_sample": ("sampling", [P, LL, P, P, P, P, I, I, P, P]),
     "pyre_sample_slices": ("sampling", [I]),
@@ -46,8 +46,8 @@ SIGNATURES: dict[str, tuple[str, list]] = {
     "pyre_cast_rows": ("blockops", [P, P, LL, I, P]),
     "pyre_norm_add": ("blockops", [P, P, P, I, LL, P, P, I, I, F, I, P]),
     "pyre_activation": ("blockops", [P, P, LL, I, I, P]),
-    "pyre_qk_norm_rope_write": ("blockops", [P, LL, I, I, I, P, P, F, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, LL, P, P]),
-    "pyre_sigmoid_gate": ("blockops", [P, I, P, LL, I, P, I, I, I, I, P]),
+    "pyre_qk_norm_rope_write": ("blockops", [P, LL, I, I, I, P, P, P, P, P, F, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, LL, P, P]),
+    "pyre_sigmoid_gate": ("blockops", [P, I, P, LL, I, P, LL, F, I, I, I, I, P]),
     "pyre_rmsnorm_gate": ("blockops", [P, P, P, LL, I, P, I, I, F, I, P]),
     "pyre_head_gate": ("blockops", [P, I, P, LL, I, P, P, P, I, I, I, I, P]),
     "pyre_bias_act": ("blockops", [P, P, P, LL, I, I, I, P]),
@@ -55,19 +55,24 @@ SIGNATURES: dict[str, tuple[str, list]] = {
     "pyre_gated_norm": ("blockops", [P, P, I, LL, P, P, P, P, P, P, I, I, F, I, I, P]),
     "pyre_token_shift_mix": ("wkv", [P, P, LL, LL, P, P, P, P, P, I, I, I, I, P]),
     "pyre_wkv_scan": ("wkv", [P, P, P, P, P, P, P, P, P, LL, LL, P, P, P, P, P, I, I, I, I, I, F, I, P]),
+    "pyre_channel_decay": ("matrix_state", [P, LL, I, I, P, P, F, P, I, I, I, P]),
+    "pyre_state_scan": ("matrix_state", [P, LL, I, I, I, F, P, P, I, LL, P, F, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, P]),
+    "pyre_state_record_floats": ("matrix_state", [I, I, I]),
+    "pyre_state_chunked": ("matrix_state", [P, LL, I, I, I, F, P, P, I, LL, P, F, P, LL, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P]),
+    "pyre_heads_finish": ("matrix_state", [P, P, P, I, P, LL, I, I, F, P, LL, I, I, I, F, I, P]),
     "pyre_linear_attention_scan": ("linear_attention", [P, LL, I, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, P]),
     "pyre_linear_attention_chunked": ("linear_attention", [P, LL, I, I, I, P, P, P, P, P, I, I, I, I, I, I, I, P]),
     "pyre_add_layernorm": ("parallel_block", [P, P, P, I, P, P, P, I, P, LL, P, P, P, P, P, I, P, I, I, F, I, I, P]),
     "pyre_scaled_sum": ("parallel_block", [P, P, I, P, P, P, I, P, LL, P, I, I, I, P]),
     "pyre_stream_rows": ("parallel_block", [P, P, P, I, P, P, P, I, P, LL, P, I, I, I, P]),
     "pyre_stream_set": ("parallel_block", [P, P, P, I, LL, LL, P]),
-    "pyre_act_mul": ("parallel_block", [P, P, I, I, I, I, P]),
+    "pyre_act_mul": ("parallel_block", [P, P, I, I, I, F, I, P]),
     "pyre_latent_prepare": ("latent_attention", [P, P, I, LL, I, I, I, I, I, I, I, P, P, F, P, P, P, P, P, I, I, LL, I, I, P, I, I, I, I, P, P]),
     "pyre_latent_rotate_q": ("latent_attention", [P, P, P, P, I, I, I, I, I, I, I, I, I, P]),
     "pyre_latent_attention_exact": ("latent_attention", [P, P, P, P, I, P, P, I, I, I, I, I, I, I, F, P, P, LL, I, LL, P, P]),
     "pyre_latent_attention_mma": ("latent_attention", [P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, F, P, P, LL, I, I, LL, P, P]),
     "pyre_grouped_linear": ("grouped", [P, LL, LL, P, LL, P, LL, LL, P, P, P, I, I, I, I, I, I, I, I, P]),
-    "pyre_route": ("grouped", [P, P, P, P, P, P, I, I, I, I, F, I, I, I, P]),
+    "pyre_route": ("grouped", [P, P, P, P, P, P, I, I, I, I, F, I, I, F, I, I, I, P]),
     "pyre_scale_to_places": ("grouped", [P, P, P, P, I, I, I, I, P]),
     "pyre_group_pairs": ("grouped", [P, I, I, I, P, P, P, P]),
     "pyre_combine_pairs": ("grouped", [P, P, P, P, P, I, I, I, I, P]),
@@ -105,6 +110,7 @@ DEFAULT_CLASS = {
     "pyre_latent_rotate_q": "rotary+write", "pyre_latent_attention_exact": "latent_attention", "pyre_latent_attention_mma": "latent_attention", "pyre_grouped_linear": "grouped_product",
     "pyre_route": "router", "pyre_group_pairs": "router", "pyre_combine_pairs": "router", "pyre_scale_to_places": "router",
     "pyre_head_gate": "gate", "pyre_bias_act": "activation", "pyre_add_row_vector": "norm", "pyre_gated_norm": "norm",
+    "pyre_channel_decay": "decay", "pyre_state_scan": "recurrence", "pyre_state_chunked": "recurrence", "pyre_heads_finish": "gate",
     "pyre_token_shift_mix": "recurrence", "pyre_wkv_scan": "recurrence",
     "pyre_scale_cap": "scale", "pyre_short_conv": "short_conv", "pyre_ssm_scan": "recurrence", "pyre_group_norm_gate": "gate",
     "pyre_diff_combine": "gate", "pyre_rotate_heads": "rotary+write", "pyre_side_gate": "activation", "pyre_token_gate_add": "router",

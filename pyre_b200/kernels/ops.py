@@ -92,9 +92,23 @@ class DeferredProduct:
             return gemm_tc(self.x, self.w, self.dtype, reduce=False)
 
 
-def materialize(t: "torch.Tensor | PartialSums | DeferredProduct | ScaledRows | ScaledSum") -> torch.Tensor:
+class BiasedRows:
+    """A branch output y + bias that is not formed yet: ``y`` a tensor or any lazy form, ``bias`` fp32 [N].  The norm on a
+    branch's result (``gated_norm``) adds the bias itself, unrounded; anything else calls ``materialize``."""
+
+    def __init__(self, y, bias: torch.Tensor):
+        self.y, self.bias = y, bias
+
+    @property
+    def shape(self):
+        return self.y.shape
+
+
+def materialize(t: "torch.Tensor | PartialSums | DeferredProduct | ScaledRows | ScaledSum | BiasedRows") -> torch.Tensor:
     """A plain tensor in the activation dtype from a tensor or any of the lazy forms a branch output or a
     norm's output may take."""
+    if isinstance(t, BiasedRows):
+        return bias_act(materialize(t.y), t.bias, None)
     if isinstance(t, ScaledSum):
         return t.tensor()
     if isinstance(t, DeferredProduct):
@@ -191,6 +205,8 @@ def add_rmsnorm(x: torch.Tensor, delta: "torch.Tensor | None", weight: torch.Ten
 
     ``scaled_ok``: the caller's consumer takes ``ScaledRows``.  Then a deferred product is launched with the
     residual add and the norm's preparation as its fix-up, and no norm kernel runs at all."""
+    if isinstance(delta, BiasedRows):
+        delta = materialize(delta)
     _check(x, "x", torch.float32, 2)
     _check(weight, "weight", torch.float32, 1)
     T, H = x.shape
@@ -310,7 +326,7 @@ def qkv_rope_write(qkv: torch.Tensor, bias: "torch.Tensor | None", cos: torch.Te
     return q_out
 
 
-def silu_mul(gate_up: torch.Tensor, out: "torch.Tensor | None" = None, block: int = 0, kind: str = "silu") -> torch.Tensor:
+def silu_mul(gate_up: torch.Tensor, out: "torch.Tensor | None" = None, block: int = 0, kind: str = "silu", limit: float = 0.0) -> torch.Tensor:
     """out[t, i] = act(gate[t, i]) * up[t, i], act ``silu`` or ``relu`` (``kind``).  ``block == 0``: gate_up = [all gates | all ups];
     ``block == n``: gates and ups alternate in blocks of n features (n gates, their n ups, ...)."""
     _check(gate_up, "gate_up", dim=2)
@@ -324,7 +340,7 @@ def silu_mul(gate_up: torch.Tensor, out: "torch.Tensor | None" = None, block: in
         out = torch.empty((T, inter), dtype=gate_up.dtype, device=gate_up.device)
     if kind not in GATE_KINDS:
         raise UnsupportedSize(f"gate activation {kind!r}: this kernel knows {sorted(GATE_KINDS)}")
-    lib.call("pyre_silu_mul", gate_up.data_ptr(), out.data_ptr(), T, inter, int(block), int(kind == "relu"), _dt(gate_up.dtype), _stream())
+    lib.call("pyre_silu_mul", gate_up.data_ptr(), out.data_ptr(), T, inter, int(block), {"silu": 0, "relu": 1, "clamped": 2}[kind], float(limit), _dt(gate_up.dtype), _stream())
     return out
 
 
@@ -786,7 +802,7 @@ def tc_gemm_plan(M: int, N: int, K: int) -> tuple[bool, int, int]:
     return False, whole[1], whole[2]
 
 
-GATE_KINDS = {"silu": 1, "relu": 3}     # gates that a gated product applies in its epilogue: the kernel's argument
+GATE_KINDS = {"silu": 1, "relu": 3, "clamped": 4}     # gates that a gated product applies in its epilogue: the kernel's argument
 GATED_BLOCK = 64     # gate and up rows of a fused feed-forward weight alternate in blocks of this many features
 
 
@@ -810,7 +826,7 @@ def _scale_fields(fx: "lib.GemmFix", x: "ScaledRows") -> None:
 
 def gemm_tc(x: "torch.Tensor | ScaledRows", w: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16,
             plan: "tuple[bool, int, int] | None" = None, reduce: bool = True, gated: "bool | str" = False,
-            pair: "bool | None" = None, checked: bool = False) -> torch.Tensor:
+            pair: "bool | None" = None, checked: bool = False, limit: float = 0.0) -> torch.Tensor:
     """y = x w^T on the tensor cores (tcgen05, TMEM accumulators, TMA-fed), bf16 in, fp32 accumulate.
 
     With a split K the kernel leaves fp32 partial sums [splits, M, N]; ``reduce`` adds
@@ -818,7 +834,8 @@ def gemm_tc(x: "torch.Tensor | ScaledRows", w: torch.Tensor, out_dtype: torch.dt
     as ``PartialSums`` for a consumer kernel that adds them itself.
 
     ``gated``: w holds gate and up rows alternating in blocks of ``GATED_BLOCK`` features; the
-    result is silu(x gate^T) * (x up^T), [M, N / 2] bf16 (``gated="relu"``: relu instead).  The activation runs in the product's
+    result is silu(x gate^T) * (x up^T), [M, N / 2] bf16 (``gated="relu"``: relu instead;
+    ``"clamped"``: the clamped form with ``limit``, see ``act_mul``).  The activation runs in the product's
     epilogue (whole tiles, one split: the usual case in both orientations), otherwise after it.
 
     ``x`` may be ``ScaledRows``: the result rows are scaled by the tokens' 1/rms in the epilogue, before the
@@ -861,15 +878,15 @@ def gemm_tc(x: "torch.Tensor | ScaledRows", w: torch.Tensor, out_dtype: torch.dt
         if not weights_as_rows and bn == 256 and splits == 1 and N % 256 == 0:
             out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
             lib.call("pyre_gemm_tc", x.data_ptr(), M, x.stride(0), w.data_ptr(), N, w.stride(0), K, out.data_ptr(), 0,
-                     N // 2, 1, 0, 1, bn, 0, GATE_KINDS[gate], pair, err.data_ptr(), fx, _stream())
+                     N // 2, 1, 0, 1, bn, 0, GATE_KINDS[gate], float(limit), pair, err.data_ptr(), fx, _stream())
             return out
         if weights_as_rows and bn <= 128 and splits == 1 and N % 128 == 0:
             out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
             lib.call("pyre_gemm_tc", w.data_ptr(), N, w.stride(0), x.data_ptr(), M, x.stride(0), K, out.data_ptr(), 0,
-                     1, N // 2, 0, 1, bn, 1, GATE_KINDS[gate], 0, err.data_ptr(), fx, _stream())
+                     1, N // 2, 0, 1, bn, 1, GATE_KINDS[gate], float(limit), 0, err.data_ptr(), fx, _stream())
             return out
         return silu_mul(gemm_tc(scaled if scaled is not None else x, w, torch.bfloat16, (weights_as_rows, bn, splits), pair=bool(pair)),
-                        block=GATED_BLOCK, kind=gate)
+                        block=GATED_BLOCK, kind=gate, limit=limit)
     if splits == 1 and reduce:
         out = torch.empty((M, N), dtype=out_dtype, device=x.device)
         target, split_stride = out, 0
@@ -879,10 +896,10 @@ def gemm_tc(x: "torch.Tensor | ScaledRows", w: torch.Tensor, out_dtype: torch.dt
     f32 = int(target.dtype == torch.float32)
     if weights_as_rows:
         lib.call("pyre_gemm_tc", w.data_ptr(), N, w.stride(0), x.data_ptr(), M, x.stride(0), K, target.data_ptr(), f32,
-                 1, N, split_stride, splits, bn, 1, 0, 0, err.data_ptr(), fx, _stream())
+                 1, N, split_stride, splits, bn, 1, 0, 0.0, 0, err.data_ptr(), fx, _stream())
     else:
         lib.call("pyre_gemm_tc", x.data_ptr(), M, x.stride(0), w.data_ptr(), N, w.stride(0), K, target.data_ptr(), f32,
-                 N, 1, split_stride, splits, bn, 0, 0, pair, err.data_ptr(), fx, _stream())
+                 N, 1, split_stride, splits, bn, 0, 0, 0.0, pair, err.data_ptr(), fx, _stream())
     if target.dim() == 2:
         return target
     if not reduce:
@@ -913,13 +930,13 @@ def _launch_with_fixup(prod: DeferredProduct, fx: "lib.GemmFix", rows_out: "torc
             parts = torch.empty((splits, M, N), dtype=torch.float32, device=x.device)
             fx.tile_counters = _tile_counters(x.device).data_ptr()
             lib.call("pyre_gemm_tc", w.data_ptr(), N, w.stride(0), x.data_ptr(), M, x.stride(0), K, parts.data_ptr(), 1,
-                     1, N, M * N, splits, bn, 1, 0, 0, err, ctypes.byref(fx), _stream())
+                     1, N, M * N, splits, bn, 1, 0, 0.0, 0, err, ctypes.byref(fx), _stream())
         else:
             if splits != 1 or rows_out is None:
                 raise UnsupportedSize("a product of many tokens folds only with one split and the residual fix-up")
             pair = int(CTA_PAIRS and bn in (128, 160, 192, 208, 224, 256))
             lib.call("pyre_gemm_tc", x.data_ptr(), M, x.stride(0), w.data_ptr(), N, w.stride(0), K, rows_out.data_ptr(), 0,
-                     N, 1, 0, 1, bn, 0, 0, pair, err, ctypes.byref(fx), _stream())
+                     N, 1, 0, 1, bn, 0, 0, 0.0, pair, err, ctypes.byref(fx), _stream())
 
 
 def folds_residual(M: int, N: int, K: int) -> bool:
@@ -1068,14 +1085,14 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor, block: int = GATED_
     return torch.stack([gate.view(inter // block, block, K), up.view(inter // block, block, K)], dim=1).reshape(2 * inter, K).contiguous()
 
 
-def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, interleaved: bool, kind: str = "silu") -> torch.Tensor:
-    """act(x gate^T) * (x up^T), act silu or relu (``kind``), for the stacked weight of a gated feed-forward: [gates | ups] rows, or
+def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, interleaved: bool, kind: str = "silu", limit: float = 0.0) -> torch.Tensor:
+    """act(x gate^T) * (x up^T), act silu or relu (``kind``; ``"clamped"`` with ``limit``: see ``act_mul``), for the stacked weight of a gated feed-forward: [gates | ups] rows, or
     (``interleaved``) blocks of ``GATED_BLOCK`` gate rows and up rows in turn, which lets the bfloat16
     tensor-core product apply the activation in its epilogue."""
     rows = x.rows if isinstance(x, ScaledRows) else x
     if interleaved and x.dtype == torch.bfloat16 and USE_TC_GEMM and tc_gemm_supported(rows, w_gate_up):
-        return gemm_tc(x, w_gate_up, torch.bfloat16, gated=kind, checked=True)
-    return silu_mul(linear(x, w_gate_up), block=GATED_BLOCK if interleaved else 0, kind=kind)
+        return gemm_tc(x, w_gate_up, torch.bfloat16, gated=kind, checked=True, limit=limit)
+    return silu_mul(linear(x, w_gate_up), block=GATED_BLOCK if interleaved else 0, kind=kind, limit=limit)
 
 
 # ---------------------------------------------------------------------------------- layers that are no pre-norm block
@@ -1098,6 +1115,8 @@ def norm_add(x: torch.Tensor, y: "torch.Tensor | PartialSums | DeferredProduct",
     """x[t] += rmsnorm(y[t]) * weight in place on the fp32 stream ``x`` [T, H]: the norm sits on a branch's OUTPUT
     ``y`` (activation dtype, or fp32 partial sums that the kernel adds).  ``want_next``: also return the new stream
     as activations (what the next branch reads), written in the same pass."""
+    if isinstance(y, BiasedRows):
+        y = materialize(y)
     _check(x, "x", torch.float32, 2)
     _check(weight, "weight", torch.float32, 1)
     T, H = x.shape
@@ -1138,7 +1157,7 @@ def linear_act(x: torch.Tensor, w: torch.Tensor, kind: str) -> torch.Tensor:
             out = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
             pair = int(CTA_PAIRS and bn in (128, 160, 192, 208, 224, 256))
             lib.call("pyre_gemm_tc", x.data_ptr(), M, x.stride(0), w.data_ptr(), N, w.stride(0), K, out.data_ptr(), 0,
-                     N, 1, 0, 1, bn, 0, 2, pair, device_error_flag(x.device).data_ptr(), None, _stream())
+                     N, 1, 0, 1, bn, 0, 2, 0.0, pair, device_error_flag(x.device).data_ptr(), None, _stream())
             return out
     return activation(materialize(linear(x, w)), kind)
 
@@ -1161,7 +1180,7 @@ def qk_norm_rope_write(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
                        cache_layer: "torch.Tensor | None", slot_mapping: "torch.Tensor | None", n_heads: int,
                        n_kv_heads: int, qk_dim: int, v_dim: int, row_dim: int, rotary_dim: int, page_size: int,
                        v_cos: "torch.Tensor | None" = None, v_sin: "torch.Tensor | None" = None, neighbours: bool = False,
-                       post_norm: bool = False) -> torch.Tensor:
+                       post_norm: bool = False, biases: "tuple | None" = None) -> torch.Tensor:
     """Per-head RMS norm of queries and keys (weights [qk_dim], shared by the heads; None: no norm), rotation of
     the first ``rotary_dim`` dims of each head, and the paged write, for heads whose query/key size ``qk_dim`` and
     value size ``v_dim`` differ from the cache's row size ``row_dim`` (the rest of a row is zero).
@@ -1171,6 +1190,8 @@ def qk_norm_rope_write(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
     half-split pairs, by these tables, and cached so (``head_gate`` turns a head's weighted sum back).
     ``neighbours``: the rotation's pairs are (2i, 2i + 1) instead of (i, i + rotary_dim / 2).  ``post_norm``: after the
     rotation every query and key head is divided by its root mean square over ``qk_dim`` (with ``eps``, no weight).
+    ``biases``: (q, k, v) fp32 vectors (each may be None) added to the projections before anything else.  ``v_col`` may
+    be ``k_col``: the values are then the keys as projected.
     Returns the queries [T, n_heads * row_dim]."""
     _check(proj, "proj", dim=2)
     T, W = proj.shape
@@ -1211,8 +1232,15 @@ def qk_norm_rope_write(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
         _check(sin, "sin", torch.float32, 2)
         if tuple(cos.shape) != (T, half) or tuple(sin.shape) != (T, half):
             raise ValueError(f"cos/sin must be [{T}, {half}], got {tuple(cos.shape)}")
+    q_b, k_b, v_b = biases or (None, None, None)
+    for b, name, n in ((q_b, "q", n_heads * qk_dim), (k_b, "k", n_kv_heads * qk_dim), (v_b, "v", n_kv_heads * v_dim)):
+        if b is not None:
+            _check(b, name + " bias", torch.float32, 1)
+            if b.shape[0] != n:
+                raise ValueError(f"{name} bias has {b.shape[0]} entries, the heads have {n}")
     q_out = torch.empty((T, n_heads * D), dtype=proj.dtype, device=proj.device)
     lib.call("pyre_qk_norm_rope_write", proj.data_ptr(), W, int(q_col), int(k_col) if write else -1, int(v_col) if write else -1,
+             _ptr(q_b), _ptr(k_b), _ptr(v_b),
              _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(cos) if rotary_dim else None, _ptr(sin) if rotary_dim else None,
              _ptr(v_cos), _ptr(v_sin), q_out.data_ptr(), _ptr(cache_layer), _ptr(slot_mapping) if write else None, T, n_heads,
              n_kv_heads, qk_dim, v_dim, D, rotary_dim, int(bool(neighbours)), int(bool(post_norm)), page_size, _dt(proj.dtype),
@@ -1220,9 +1248,23 @@ def qk_norm_rope_write(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q
     return q_out
 
 
-def sigmoid_gate(a: torch.Tensor, a_dim: int, proj: "torch.Tensor | None", g_col: int, n_heads: int, v_dim: int) -> torch.Tensor:
+def _rows_out(out: "torch.Tensor | None", col: int, T: int, width: int, dtype, device) -> tuple:
+    """(tensor, pointer, row stride) of ``width`` columns from ``col`` of the rows of ``out`` [T, >= col + width]; ``out``
+    None: a new tensor [T, width]."""
+    if out is None:
+        out = torch.empty((T, width), dtype=dtype, device=device)
+        return out, out.data_ptr(), width
+    _check(out, "out", dtype, 2)
+    if out.shape[0] != T or col < 0 or col + width > out.shape[1]:
+        raise ValueError(f"{width} columns from {col} do not lie inside the rows of {tuple(out.shape)}")
+    return out, out.data_ptr() + col * out.element_size(), out.shape[1]
+
+
+def sigmoid_gate(a: torch.Tensor, a_dim: int, proj: "torch.Tensor | None", g_col: int, n_heads: int, v_dim: int,
+                 out: "torch.Tensor | None" = None, out_col: int = 0, scale: float = 1.0) -> torch.Tensor:
     """out[t, h, j] = a[t, h, j] * sigmoid(proj[t, g_col + h v_dim + j]) for j < v_dim; a head of ``a`` has ``a_dim``
-    columns, of which the first ``v_dim`` count.  ``proj`` None: no gate, the heads are only narrowed.
+    columns, of which the first ``v_dim`` count.  ``proj`` None: no gate, the heads are only narrowed.  Everything is
+    multiplied by ``scale``.  ``out`` [T, W]: written to its columns from ``out_col`` on instead of a new tensor.
     Returns [T, n_heads * v_dim]."""
     _check(a, "a", dim=2)
     T = a.shape[0]
@@ -1232,9 +1274,9 @@ def sigmoid_gate(a: torch.Tensor, a_dim: int, proj: "torch.Tensor | None", g_col
         _check(proj, "proj", a.dtype, 2)
         if proj.shape[0] != T or g_col < 0 or g_col + n_heads * v_dim > proj.shape[1]:
             raise ValueError("the gate does not lie inside the projection row")
-    out = torch.empty((T, n_heads * v_dim), dtype=a.dtype, device=a.device)
+    out, at, stride = _rows_out(out, out_col, T, n_heads * v_dim, a.dtype, a.device)
     lib.call("pyre_sigmoid_gate", a.data_ptr(), int(a_dim), _ptr(proj), proj.shape[1] if proj is not None else 0,
-             int(g_col) if proj is not None else -1, out.data_ptr(), T, n_heads, v_dim, _dt(a.dtype), _stream())
+             int(g_col) if proj is not None else -1, at, stride, float(scale), T, n_heads, v_dim, _dt(a.dtype), _stream())
     return out
 
 
@@ -1303,6 +1345,10 @@ def gated_norm(y: "torch.Tensor | PartialSums | DeferredProduct", y_bias: "torch
     ``gate`` None: no gate.  ``out_bias`` fp32 [H]: added after the gain (a norm with a bias)."""
     _check(weight, "weight", torch.float32, 1)
     H = weight.shape[0]
+    if isinstance(y, BiasedRows):
+        if y_bias is not None:
+            raise ValueError("a branch output that carries its bias gets no second one")
+        y, y_bias = y.y, y.bias
     if isinstance(y, DeferredProduct):
         y = y.partials()
     parts, n_parts, stride = None, 0, 0
@@ -1488,6 +1534,8 @@ def add_layernorm(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSum
     plain branch output or partial sums (gain one), or None.  ``out_dtype`` float32 with bfloat16 activations
     (``act_dtype``) gives the normalised rows in fp32: a norm applied to the stream itself.  ``weight2``: a second norm
     of the SAME rows (no bias) written in the same pass; the result is then the pair."""
+    if isinstance(delta, BiasedRows):
+        delta = materialize(delta)
     _check(x, "x", torch.float32, 2)
     _check(weight, "weight", torch.float32, 1)
     T, H = x.shape
@@ -1527,6 +1575,8 @@ def add_layernorm(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSum
 def stream_rows(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSums | None", dtype: torch.dtype) -> torch.Tensor:
     """The fp32 stream ``x`` [T, H] with ``delta`` (as in ``add_layernorm``) added, as activations for a product that
     reads the stream itself: a new tensor in ``dtype``; ``x`` stays as it is."""
+    if isinstance(delta, BiasedRows):
+        delta = materialize(delta)
     _check(x, "x", torch.float32, 2)
     T, H = x.shape
     if delta is not None and not isinstance(delta, ScaledSum):
@@ -1566,11 +1616,12 @@ def _ones(n: int, device) -> torch.Tensor:
     return t
 
 
-MUL_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu": 2}
+MUL_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu": 2, "clamped": 3}
 
 
-def act_mul(gate_up: torch.Tensor, kind: str) -> torch.Tensor:
-    """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i] for rows [gates | ups]; ``kind`` as in ``MUL_ACTIVATIONS``."""
+def act_mul(gate_up: torch.Tensor, kind: str, limit: float = 0.0) -> torch.Tensor:
+    """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i] for rows [gates | ups]; ``kind`` as in ``MUL_ACTIVATIONS``.
+    ``"clamped"``: z sigmoid(1.702 z) (u + 1) with z = min(gate, limit) and u = clamp(up, -limit, limit)."""
     _check(gate_up, "gate_up", dim=2)
     if kind not in MUL_ACTIVATIONS:
         raise UnsupportedSize(f"activation {kind!r}: implemented are {sorted(MUL_ACTIVATIONS)}")
@@ -1578,7 +1629,7 @@ def act_mul(gate_up: torch.Tensor, kind: str) -> torch.Tensor:
     if two_i % 2:
         raise ValueError("gate_up must have an even number of columns")
     out = torch.empty((T, two_i // 2), dtype=gate_up.dtype, device=gate_up.device)
-    lib.call("pyre_act_mul", gate_up.data_ptr(), out.data_ptr(), T, two_i // 2, MUL_ACTIVATIONS[kind], _dt(gate_up.dtype), _stream())
+    lib.call("pyre_act_mul", gate_up.data_ptr(), out.data_ptr(), T, two_i // 2, MUL_ACTIVATIONS[kind], float(limit), _dt(gate_up.dtype), _stream())
     return out
 
 
@@ -1754,11 +1805,13 @@ def expert_linear(x: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, src: 
 
 
 def route(h: torch.Tensor, w: torch.Tensor, correction: "torch.Tensor | None", top: int, scale: float, sigmoid: bool = False,
-          bias: "torch.Tensor | None" = None, renormalise: bool = False):
+          bias: "torch.Tensor | None" = None, renormalise: bool = False, renorm_eps: float = 0.0, groups: int = 1, keep: int = 1):
     """Router of a routed feed-forward: fp32 logits w h (+ ``bias``) over all router outputs, softmax scores s
     (``sigmoid``: each output's own sigmoid instead); the ``top`` outputs with the largest s + correction are chosen
     (lowest index on ties), weights s * scale; ``renormalise``: divided by their sum over the chosen (with softmax
-    scores that is the softmax over the chosen logits alone).
+    scores that is the softmax over the chosen logits alone), the sum plus ``renorm_eps``.  ``groups`` > 1: the outputs
+    form so many equal groups of neighbours, a group's score is the sum of its two largest s + correction, and only
+    outputs of the ``keep`` best groups can be chosen.
     Returns (idx int32 [T, top], weight fp32 [T, top])."""
     _check(h, "h", dim=2)
     _check(w, "w", torch.float32, 2)
@@ -1774,12 +1827,14 @@ def route(h: torch.Tensor, w: torch.Tensor, correction: "torch.Tensor | None", t
         _check(bias, "bias", torch.float32, 1)
         if bias.shape[0] != n_out:
             raise ValueError("one bias per router output")
-    if n_out * 8 > 48 * 1024:
+    if groups > 1 and (n_out % groups or not 0 < keep <= groups or top > keep * (n_out // groups)):
+        raise ValueError(f"{keep} of {groups} groups of {n_out} router outputs cannot give {top}")
+    if n_out * 8 + groups * 4 > 48 * 1024:
         raise UnsupportedSize(f"{n_out} router outputs: the kernel takes up to 6,144")
     idx = torch.empty((T, top), dtype=torch.int32, device=h.device)
     weight = torch.empty((T, top), dtype=torch.float32, device=h.device)
     lib.call("pyre_route", h.data_ptr(), w.data_ptr(), _ptr(correction), _ptr(bias), idx.data_ptr(), weight.data_ptr(), T, H, n_out,
-             int(top), float(scale), int(bool(sigmoid)), int(bool(renormalise)), _dt(h.dtype), _stream())
+             int(top), float(scale), int(bool(sigmoid)), int(bool(renormalise)), float(renorm_eps), int(groups), int(keep), _dt(h.dtype), _stream())
     return idx, weight
 
 
@@ -2085,6 +2140,141 @@ def group_norm_gate(y: torch.Tensor, groups: int, weight: "torch.Tensor | None",
     lib.call("pyre_group_norm_gate", y.data_ptr(), _ptr(proj), proj.shape[1] if proj is not None else 0,
              int(g_col) if proj is not None else -1, GATE_ACTIVATIONS[gate], int(bool(gate_first)), _ptr(weight), float(post),
              out.data_ptr(), T, W, int(groups), float(eps), _dt(out_dtype), _stream())
+    return out
+
+
+# ---------------------------------------------------------------------------------- matrix states with decays that depend on the token
+STATE_MAX_DIM = 256            # query/key entries per head
+STATE_CHUNK_MIN_LEN = 32       # bfloat16 entries with at least this many tokens run in blocks on the tensor cores
+STATE_CHUNK_WARPS = 2          # tiles of 16 value columns per CTA of that kernel
+USE_STATE_CHUNKS = True
+
+
+def memory_state_floats(n_heads: int, qk_dim: int, v_dim: int) -> int:
+    """Floats of one request's slot of a matrix memory: S [heads, qk_dim, v_dim], n [heads, qk_dim] and copies of the
+    running maximum (one per 16 value columns and one for n)."""
+    return n_heads * (qk_dim * v_dim + qk_dim + -(-v_dim // 16) + 1)
+
+
+def channel_decay(proj: torch.Tensor, col: int, rank: int, weight: torch.Tensor, bias: torch.Tensor, tau: float) -> torch.Tensor:
+    """Log decays of gated linear attention, fp32 [T, C]: logsigmoid(inner w + bias) / tau with ``inner`` the ``rank``
+    columns of ``proj`` from ``col`` on and ``weight`` fp32 [rank, C] (the map's transpose)."""
+    _check(proj, "proj", dim=2)
+    _check(weight, "weight", torch.float32, 2)
+    _check(bias, "bias", torch.float32, 1)
+    T, C = proj.shape[0], weight.shape[1]
+    if weight.shape[0] != rank or bias.shape[0] != C or col < 0 or col + rank > proj.shape[1]:
+        raise ValueError("the decay's map does not match the projection row")
+    out = torch.empty((T, C), dtype=torch.float32, device=proj.device)
+    lib.call("pyre_channel_decay", proj.data_ptr(), proj.shape[1], int(col), int(rank), weight.data_ptr(), bias.data_ptr(), float(tau),
+             out.data_ptr(), T, C, _dt(proj.dtype), _stream())
+    return out
+
+
+def _matrix_state(kind: int, proj, q_col, k_col, v_col, q_scale, logd, gates, gate_bias, cap, state_layer, slots, cu_seqlens, n_heads,
+                  qk_dim, v_dim, lens, chunked):
+    _check(proj, "proj", dim=2)
+    _check(state_layer, "state_layer", torch.float32)
+    _check(slots, "slots", torch.int32, 1)
+    _check(cu_seqlens, "cu_seqlens", torch.int32, 1)
+    T, W = proj.shape
+    n_seqs = cu_seqlens.shape[0] - 1
+    slot_floats = state_layer[0].numel()
+    if min(q_col, k_col, v_col) < 0 or max(q_col, k_col) + n_heads * qk_dim > W or v_col + n_heads * v_dim > W:
+        raise ValueError("queries, keys or values do not lie inside the projection row")
+    if slots.shape[0] < n_seqs:
+        raise ValueError("slots do not match the batch")
+    if qk_dim > STATE_MAX_DIM:
+        raise UnsupportedSize(f"heads of {qk_dim}: the recurrence takes up to {STATE_MAX_DIM}")
+    o = torch.empty((T, n_heads * v_dim), dtype=torch.float32, device=proj.device)
+    den = torch.empty((T, n_heads), dtype=torch.float32, device=proj.device) if kind == 1 else None
+    parts, n_parts = (None, 0) if gates is None else (gates.parts, gates.n) if isinstance(gates, PartialSums) else (gates, 1)
+    record = 0
+    if USE_STATE_CHUNKS and chunked is not False and lens is not None and proj.dtype == torch.bfloat16:
+        record = lib.call_value("pyre_state_record_floats", int(qk_dim), int(v_dim), kind)
+    blocks = sum(-(-int(n) // 16) for n in lens if n >= STATE_CHUNK_MIN_LEN) if record else 0
+    if blocks:
+        scratch = torch.empty(blocks * n_heads * record, dtype=torch.float32, device=proj.device)
+        lib.call("pyre_state_chunked", proj.data_ptr(), W, int(q_col), int(k_col), int(v_col), float(q_scale), _ptr(logd), _ptr(parts), n_parts,
+                 T * 2 * n_heads, _ptr(gate_bias), float(cap), state_layer.data_ptr(), slot_floats, slots.data_ptr(), cu_seqlens.data_ptr(),
+                 o.data_ptr(), _ptr(den), scratch.data_ptr(), T, n_seqs, n_heads, qk_dim, v_dim, STATE_CHUNK_MIN_LEN, blocks, kind,
+                 STATE_CHUNK_WARPS, _stream())
+    if not blocks or any(n < STATE_CHUNK_MIN_LEN for n in lens):
+        lib.call("pyre_state_scan", proj.data_ptr(), W, int(q_col), int(k_col), int(v_col), float(q_scale), _ptr(logd), _ptr(parts), n_parts,
+                 T * 2 * n_heads, _ptr(gate_bias), float(cap), state_layer.data_ptr(), slot_floats, slots.data_ptr(), cu_seqlens.data_ptr(),
+                 o.data_ptr(), _ptr(den), T, n_seqs, n_heads, qk_dim, v_dim, STATE_CHUNK_MIN_LEN - 1 if blocks else 0, kind,
+                 _dt(proj.dtype), _stream())
+    return o, den
+
+
+def gated_linear_attention(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_scale: float, logd: torch.Tensor,
+                           state_layer: torch.Tensor, slots: torch.Tensor, cu_seqlens: torch.Tensor, n_heads: int, qk_dim: int,
+                           v_dim: int, lens=None, chunked: "bool | None" = None) -> torch.Tensor:
+    """Linear attention with a decay per key channel over the step's entries, continuing each request's state: per head
+    S_t = diag(exp(logd_t)) S_(t-1) + k_t v_t^T, o_t = S_t^T (q_scale q_t), with q, k, v columns of ``proj`` and ``logd``
+    fp32 [T, heads * qk_dim].  ``state_layer`` [slots, ...] fp32 holds S [heads, qk_dim, v_dim] at slot ``slots[b]`` of
+    entry b and is left updated.  ``lens``: the entries' token counts on the host; with them bfloat16 entries of
+    ``STATE_CHUNK_MIN_LEN`` tokens or more run in blocks of 16 tokens on the tensor cores (query/key sizes up to 128,
+    ``chunked=False``: not); everything else walks token by token, bit-identical under any cutting.
+    Returns fp32 [T, heads * v_dim]."""
+    _check(logd, "logd", torch.float32, 2)
+    if tuple(logd.shape) != (proj.shape[0], n_heads * qk_dim):
+        raise ValueError("one log decay per token, head and key channel")
+    if state_layer[0].numel() < n_heads * qk_dim * v_dim:
+        raise ValueError("the state does not lie inside the slot")
+    return _matrix_state(0, proj, q_col, k_col, v_col, q_scale, logd, None, None, 0.0, state_layer, slots, cu_seqlens, n_heads, qk_dim,
+                         v_dim, lens, chunked)[0]
+
+
+def matrix_memory(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_scale: float, gates: "torch.Tensor | PartialSums",
+                  gate_bias: torch.Tensor, cap: float, state_layer: torch.Tensor, slots: torch.Tensor, cu_seqlens: torch.Tensor,
+                  n_heads: int, qk_dim: int, v_dim: int, lens=None, chunked: "bool | None" = None):
+    """A matrix memory with exponential gates over the step's entries, continuing each request's state.  ``gates`` fp32
+    [T, 2 heads] (or partial sums of it): raw logits, input gates first; with ``gate_bias`` added and capped by
+    cap tanh(z / cap) they are the log input gate i and, through logsigmoid, the log forget gate f.  Per head, with a
+    running maximum m_t = max(f + m_(t-1), i):  S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k v^T, n_t likewise
+    with k alone.  ``state_layer`` [slots, >= memory_state_floats] fp32.  Returns (S_t^T q_t fp32 [T, heads * v_dim],
+    max(|n_t . q_t|, exp(-m_t)) + 1e-6 fp32 [T, heads]); the consumer divides.  ``lens``, ``chunked``: as in
+    ``gated_linear_attention``."""
+    shape = tuple(gates.shape)
+    if shape != (proj.shape[0], 2 * n_heads) or (gates.parts if isinstance(gates, PartialSums) else gates).dtype != torch.float32:
+        raise ValueError(f"gates {shape}: fp32, two per token and head")
+    _check(gates.parts if isinstance(gates, PartialSums) else gates, "gates")
+    _check(gate_bias, "gate_bias", torch.float32, 1)
+    if gate_bias.shape[0] != 2 * n_heads or not cap > 0:
+        raise ValueError("one bias per gate, and a positive cap")
+    if state_layer[0].numel() < memory_state_floats(n_heads, qk_dim, v_dim):
+        raise ValueError("the state does not lie inside the slot")
+    return _matrix_state(1, proj, q_col, k_col, v_col, q_scale, None, gates, gate_bias, cap, state_layer, slots, cu_seqlens, n_heads,
+                         qk_dim, v_dim, lens, chunked)
+
+
+def heads_finish(o: torch.Tensor, den: "torch.Tensor | None", weight: torch.Tensor, eps: float, proj: "torch.Tensor | None", g_col: int,
+                 n_heads: int, v_dim: int, out_dtype: torch.dtype, gate: str = "silu", post: float = 1.0,
+                 out: "torch.Tensor | None" = None, out_col: int = 0) -> torch.Tensor:
+    """A recurrent mixer's heads made ready for its output projection: u = o / den (``den`` None: o) per head, divided by
+    its root mean square over ``v_dim``, times ``weight`` (fp32 [v_dim], shared by the heads, or [n_heads * v_dim]), times
+    act(proj[t, g_col:]) (``gate`` silu or sigmoid; ``proj`` None: none) and ``post``.  ``out`` [T, W]: written to its
+    columns from ``out_col`` on.  Returns [T, n_heads * v_dim] in ``out_dtype`` (or ``out``)."""
+    _check(o, "o", torch.float32, 2)
+    _check(weight, "weight", torch.float32, 1)
+    T, W = o.shape
+    if W != n_heads * v_dim or weight.shape[0] not in (v_dim, W):
+        raise ValueError("the heads or the gain do not match the rows")
+    if den is not None:
+        _check(den, "den", torch.float32, 2)
+        if tuple(den.shape) != (T, n_heads):
+            raise ValueError("one denominator per token and head")
+    if gate not in GATE_ACTIVATIONS:
+        raise UnsupportedSize(f"gate {gate!r}: implemented are {sorted(GATE_ACTIVATIONS)}")
+    if proj is not None:
+        _check(proj, "proj", out_dtype, 2)
+        if proj.shape[0] != T or g_col < 0 or g_col + W > proj.shape[1]:
+            raise ValueError("the gate does not lie inside the projection row")
+    out, at, stride = _rows_out(out, out_col, T, W, out_dtype, o.device)
+    lib.call("pyre_heads_finish", o.data_ptr(), _ptr(den), weight.data_ptr(), weight.shape[0], _ptr(proj), proj.shape[1] if proj is not None else 0,
+             int(g_col) if proj is not None else -1, GATE_ACTIVATIONS[gate] if proj is not None else 0, float(post), at, stride, T,
+             n_heads, v_dim, float(eps), _dt(out_dtype), _stream())
     return out
 
 

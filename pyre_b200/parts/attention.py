@@ -3,11 +3,14 @@ pyre/model.py:296-342 and pyre/kernels/paged_attn.py for reading pages in place)
 
 from __future__ import annotations
 
+import dataclasses
+
 import torch
 
 from ..kernels import lib, ops
 from ..weights.specs import TensorSpec
-from .base import HeadGeometry, PagedKVSpec, Part, PartSpec, ProjectionLayout, make_part, register_part
+from .base import HeadGeometry, PagedKVSpec, PartSpec, ProjectionLayout, make_part, register_part
+from .stacked import StackedMixer, stack_rows
 
 
 def attention_libraries(dtype, row_dim: int) -> list[str]:
@@ -27,7 +30,7 @@ def attend(ctx, dtype, q, layer, kv, n_heads: int, n_kv_heads: int, row_dim: int
                                        scale, window, sink=sink, keep_first=keep_first)
 
 
-class Attention(Part):
+class Attention(StackedMixer):
     """q, k, v projections (stacked into one product); the position encoding (a sub-part, which adds the
     bias, encodes positions into q and k in its own way and writes keys and values to the pages of this
     call's cache layer); attention of every token of the step over its sequence's cached keys; output projection.
@@ -57,7 +60,10 @@ class Attention(Part):
     back by the query's position before the gate (the sum then depends on position differences only);
     ``own_kv=False``: the mixer has no key and value projections (and no key norm): it reads the cache layer that
     another entry of the schedule writes (``LayerCall(cache=..., write=False)``);
-    ``weight_suffix``: what follows a projection's name in the checkpoint (".weight").
+    ``value_is_key``: there is no value projection: a token's value is its key as projected (with its bias), before norm
+    and rotation;
+    ``weight_suffix`` / ``bias_suffix``: what follows a projection's name in the checkpoint (".weight", ".bias").
+    With any of these the mixer is a ``StackedMixer``: it may also stand beside other mixers.
     """
 
     DEFAULT_NAMES = {"q": "q_proj", "k": "k_proj", "v": "v_proj", "o": "o_proj", "g": "g_proj", "q_norm": "q_norm.weight",
@@ -71,8 +77,12 @@ class Attention(Part):
                  scale: "float | None" = None, window: "int | None" = None, names: "dict[str, str] | None" = None,
                  v_head_dim: "int | None" = None, qk_norm: "dict | None" = None, sink: "float | None" = None,
                  out_gate: "bool | str" = False, own_kv: bool = True, weight_suffix: str = ".weight",
-                 value_position: "PartSpec | None" = None, keep_first: int = 0, qk_unit: "dict | None" = None):
+                 value_position: "PartSpec | None" = None, keep_first: int = 0, qk_unit: "dict | None" = None,
+                 value_is_key: bool = False, bias_suffix: str = ".bias"):
         super().__init__(dtype, device)
+        self.value_is_key, self.bias_suffix, self.has_o_bias = bool(value_is_key), str(bias_suffix), bool(o_bias)
+        if self.value_is_key and (not own_kv or (v_head_dim is not None and int(v_head_dim) != int(head_dim))):
+            raise ValueError("values that are the keys need keys of the mixer's own and value heads of the keys' size")
         self.v_head_dim = int(v_head_dim) if v_head_dim is not None else int(head_dim)
         self.qk_norm_eps = float(qk_norm["eps"]) if qk_norm is not None else None
         self.qk_unit_eps = float(qk_unit["eps"]) if qk_unit is not None else None
@@ -93,9 +103,8 @@ class Attention(Part):
         # the general path: projections laid out by a ProjectionLayout, unfused small kernels
         self.general = (self.v_head_dim != int(head_dim) or qk_norm is not None or self.out_gate or not self.own_kv
                         or self.value_position is not None or self.learned_sink or qk_unit is not None
+                        or self.value_is_key or self.has_o_bias
                         or (position is not None and position.params.get("pairing") == "interleaved"))
-        if self.general and qkv_bias:
-            raise ops.UnsupportedSize("projection biases together with v_head_dim, qk_norm, out_gate or own_kv=False are not implemented")
         self.names = dict(self.DEFAULT_NAMES, **(names or {}))
         self.width, self.n_heads, self.n_kv_heads, self.head_dim = int(width), int(n_heads), int(n_kv_heads), int(head_dim)
         if self.n_heads % self.n_kv_heads:
@@ -104,8 +113,6 @@ class Attention(Part):
         self.row_dim = ops.attention_row_dim(self.head_dim, self.v_head_dim, dtype) if self.general else self.head_dim
         if self.row_dim % 16 or not 16 <= self.row_dim <= 256:
             raise ops.UnsupportedSize(f"head_dim {head_dim}: the attention kernels take multiples of 16 from 16 to 256")
-        if o_bias:
-            raise ops.UnsupportedSize("an output-projection bias is not implemented")
         if window is not None and window <= 0:
             raise ValueError("window must be positive or None")
         self.qkv_bias = bool(qkv_bias)
@@ -113,12 +120,15 @@ class Attention(Part):
         self.window = window
         self.heads = HeadGeometry(self.n_heads, self.n_kv_heads, self.head_dim)
         self.position = make_part("position", position or PartSpec("none"), dtype, device)
-        self.w_qkv = self.b_qkv = self.w_o = None
-        self.w_proj = self.q_norm_w = self.k_norm_w = None
+        self.w_qkv = self.b_qkv = None
+        self.q_norm_w = self.k_norm_w = self.biases = None
+        self.heads_width = self.n_heads * self.v_head_dim
         q_cols, kv_cols = self.n_heads * self.head_dim, self.n_kv_heads * self.head_dim
         self.layout = ProjectionLayout(self.n_heads, self.n_kv_heads, self.head_dim, self.v_head_dim, self.row_dim, 0,
-                                       q_cols if self.own_kv else -1, q_cols + kv_cols if self.own_kv else -1)
-        self.g_col = q_cols + (kv_cols + self.n_kv_heads * self.v_head_dim if self.own_kv else 0)
+                                       q_cols if self.own_kv else -1,
+                                       -1 if not self.own_kv else q_cols if self.value_is_key else q_cols + kv_cols)
+        v_cols = 0 if self.value_is_key else self.n_kv_heads * self.v_head_dim
+        self.g_col = q_cols + (kv_cols + v_cols if self.own_kv else 0)
 
     def children(self):
         # a position encoding with tensors of its own would find them under the mixer's prefix
@@ -131,10 +141,11 @@ class Attention(Part):
         if self.general:
             sfx = self.suffix
             vq, vkv = self.n_heads * self.v_head_dim, self.n_kv_heads * self.v_head_dim
-            t[n["q"] + sfx] = TensorSpec((q, self.width))
-            if self.own_kv:
-                t[n["k"] + sfx] = TensorSpec((kv, self.width))
-                t[n["v"] + sfx] = TensorSpec((vkv, self.width))
+            own = [("q", q)] + ([("k", kv)] if self.own_kv else []) + ([("v", vkv)] if self.own_kv and not self.value_is_key else [])
+            for key, rows in own:
+                t[n[key] + sfx] = TensorSpec((rows, self.width))
+                if self.qkv_bias:
+                    t[n[key] + self.bias_suffix] = TensorSpec((rows,), role="vector")
             if self.qk_norm_eps is not None:
                 t[n["q_norm"]] = TensorSpec((self.head_dim,), role="vector", init=("normal", 1.0, 0.1))
                 if self.own_kv:
@@ -144,6 +155,8 @@ class Attention(Part):
             if self.learned_sink:
                 t[n["sink"]] = TensorSpec((self.n_heads,), role="vector", init=("normal", 0.0, 1.0))
             t[n["o"] + sfx] = TensorSpec((self.width, vq))
+            if self.has_o_bias:
+                t[n["o"] + self.bias_suffix] = TensorSpec((self.width,), role="vector")
             return t
         # checkpoint order: weight then bias per projection, the output projection last
         for key, rows in (("q", q), ("k", kv), ("v", kv)):
@@ -157,10 +170,13 @@ class Attention(Part):
         n = self.names
         if self.general:
             sfx = self.suffix
-            stack = [tensors[n["q"] + sfx]] + ([tensors[n["k"] + sfx], tensors[n["v"] + sfx]] if self.own_kv else [])
-            if self.out_gate:
-                stack.append(tensors[n["g"] + sfx])
-            self.w_proj = torch.cat(stack, dim=0).contiguous() if len(stack) > 1 else stack[0]
+            own = ["q"] + (["k"] if self.own_kv else []) + (["v"] if self.own_kv and not self.value_is_key else [])
+            self.w_in = stack_rows([tensors[n[key] + sfx] for key in own + (["g"] if self.out_gate else [])])
+            if self.qkv_bias:
+                b = {key: tensors[n[key] + self.bias_suffix] for key in own}
+                self.biases = (b["q"], b.get("k"), b.get("k") if self.value_is_key else b.get("v"))
+            if self.has_o_bias:
+                self.b_o = tensors[n["o"] + self.bias_suffix]
             if self.qk_norm_eps is not None:
                 self.q_norm_w = tensors[n["q_norm"]]
                 self.k_norm_w = tensors[n["k_norm"]] if self.own_kv else None
@@ -195,36 +211,42 @@ class Attention(Part):
         return attend(ctx, self.dtype, q, layer, kv, self.n_heads, self.n_kv_heads, self.row_dim, self.scale, self.window,
                       sink=self.sink, keep_first=self.keep_first)
 
-    def _forward_general(self, ctx, h, call):
-        """Projections in one product [q | k | v | gate]; norm, position encoding and the paged write by the
-        encoding's ``apply_layout``; attention over cache rows of ``row_dim``; the gate; the output projection."""
+    def head_rows(self, ctx, h, proj, col, call, out=None, out_col=0, scale=1.0):
+        """From the projections [q | k | v | gate] at column ``col``: biases, norm, position encoding and the paged write by
+        the encoding's ``apply_layout``; attention over cache rows of ``row_dim``; the gate."""
         kv = ctx.kv_group(call.kv_group)
         layer = kv.pool[call.kv_layer]
         if self.own_kv != bool(call.kv_write):
             raise ValueError("a mixer with its own keys and values writes its cache layer; one without reads another's")
-        with lib.section("qkv"):
-            proj = ops.materialize(ops.linear(h, self.w_proj))
+        layout, g_col = self.layout, self.g_col + col
+        if col:
+            layout = dataclasses.replace(layout, q_col=layout.q_col + col, k_col=layout.k_col + col if self.own_kv else -1,
+                                         v_col=layout.v_col + col if self.own_kv else -1)
         kw, vcos, vsin = {}, None, None
         if self.value_position is not None:
             vcos, vsin, _ = self.value_position.rotation(ctx, self.v_head_dim)
             kw["value_tables"] = (vcos, vsin)
         if self.qk_unit_eps is not None:
             kw["post_norm"] = True
-        q = self.position.apply_layout(ctx, proj, self.layout, self.q_norm_w, self.k_norm_w, self.qk_norm_eps or self.qk_unit_eps or 0.0, kv,
+        if self.biases is not None:
+            kw["biases"] = self.biases
+        q = self.position.apply_layout(ctx, proj, layout, self.q_norm_w, self.k_norm_w, self.qk_norm_eps or self.qk_unit_eps or 0.0, kv,
                                        layer if call.kv_write else None, **kw)
         a = self._attend(ctx, q, layer, kv)
         if self.head_gate or vcos is not None:
             if self.out_gate and not self.head_gate:
                 raise ops.UnsupportedSize("rotated values with a gate per entry are not implemented")
-            a = ops.head_gate(a, self.row_dim, proj if self.head_gate else None, self.g_col, self.n_heads, self.v_head_dim, vcos, vsin)
-        elif self.out_gate or self.row_dim != self.v_head_dim:
-            a = ops.sigmoid_gate(a, self.row_dim, proj if self.out_gate else None, self.g_col, self.n_heads, self.v_head_dim)
-        with lib.section("o"):
-            return ops.linear(a, self.w_o, partials_ok=True)
+            a = ops.head_gate(a, self.row_dim, proj if self.head_gate else None, g_col, self.n_heads, self.v_head_dim, vcos, vsin)
+            return a if out is None and scale == 1.0 else ops.sigmoid_gate(a, self.v_head_dim, None, -1, self.n_heads, self.v_head_dim,
+                                                                           out=out, out_col=out_col, scale=scale)
+        if self.out_gate or self.row_dim != self.v_head_dim or out is not None or scale != 1.0:
+            a = ops.sigmoid_gate(a, self.row_dim, proj if self.out_gate else None, g_col, self.n_heads, self.v_head_dim,
+                                 out=out, out_col=out_col, scale=scale)
+        return a
 
     def forward(self, ctx, h, call):
         if self.general:
-            return self._forward_general(ctx, h, call)
+            return super().forward(ctx, h, call)
         kv = ctx.kv_group(call.kv_group)
         layer = kv.pool[call.kv_layer]
         with lib.section("qkv"):

@@ -183,6 +183,9 @@ class Part:
         """Take the tensors named by ``tensors()`` (already on the device, already in
         their roles' dtypes) and by ``shared_tensors()``."""
 
+    def loaded(self) -> None:
+        """The part and its sub-parts have taken their tensors: a part that packs what its sub-parts hold does so here."""
+
     def kernel_libraries(self) -> list[str]:
         return []
 
@@ -215,7 +218,7 @@ class PositionEncoding(Part):
         return None, None, 0
 
     def apply_layout(self, ctx, proj, layout: ProjectionLayout, q_norm, k_norm, norm_eps: float, kv, cache_layer,
-                     value_tables=None, post_norm: bool = False):
+                     value_tables=None, post_norm: bool = False, biases=None):
         """The same step for projections laid out by a ``ProjectionLayout`` (key and value sizes that differ, rows
         padded to the cache's row size), with an optional RMS norm per head over the query and key dims before
         the encoding (``q_norm`` / ``k_norm``: fp32 weights [qk_dim] or None).  Stores keys and values in
@@ -223,13 +226,15 @@ class PositionEncoding(Part):
         rotation of leading dims only has to give ``rotation``.  ``value_tables``: (cos, sin) [T, v_dim / 2] of a
         rotation that the mixer wants on the VALUES before they are cached (given only by a mixer that has one).
         ``post_norm``: after the rotation queries and keys are divided by their root mean square per head (``norm_eps``,
-        no weight; given only by a mixer that wants it)."""
+        no weight; given only by a mixer that wants it).  ``biases``: (q, k, v) fp32 vectors (each may be None) added to the
+        projections first (given only by a mixer that has some)."""
         from ..kernels import ops
         cos, sin, rotary_dim = self.rotation(ctx, layout.qk_dim)
         return ops.qk_norm_rope_write(proj, layout.q_col, layout.k_col, layout.v_col, q_norm, k_norm, norm_eps, cos, sin,
                                       cache_layer, kv.slot_mapping, layout.n_heads, layout.n_kv_heads, layout.qk_dim,
                                       layout.v_dim, layout.row_dim, rotary_dim, kv.page_size,
-                                      *(value_tables or ()), **self._layout_options(post_norm))
+                                      *(value_tables or ()), **self._layout_options(post_norm),
+                                      **({"biases": biases} if biases is not None else {}))
 
     def _layout_options(self, post_norm: bool) -> dict:
         """Options of the fused rotation + write kernel beyond its defaults (a rotation of neighbouring pairs, a norm
@@ -290,6 +295,8 @@ def load_part(part: Part, tensors: Mapping[str, torch.Tensor], prefix: str = "")
     part.load(own)
     for sub_prefix, child in part.children().items():
         load_part(child, tensors, prefix + sub_prefix)
+    if hasattr(part, "loaded"):
+        part.loaded()
 
 
 def all_graph_safe(part: Part) -> bool:

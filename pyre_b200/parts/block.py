@@ -199,7 +199,8 @@ class SandwichBlock(Part):
     The stream ``x`` is fp32.  A sublayer's gated, normed result is formed in fp32 by one kernel (``gated_output`` of
     the norm part) and travels unadded, as ``pending``, to the next norm before a sublayer, whose kernel adds it to
     the stream while it normalises.  ``after``: a ``stream`` part that runs once the sublayers are done (a per-layer
-    input from the step's token ids); it gets the stream and what is pending.  ``names``: the prefixes of the
+    input from the step's token ids); it gets the stream and what is pending.  ``spare_norms``: the layer has no
+    feed-forward, but its checkpoint may hold the second sublayer's norms all the same.  ``names``: the prefixes of the
     sub-parts' tensors and the names of the gates' weights and biases."""
 
     graph_safe = True
@@ -210,13 +211,14 @@ class SandwichBlock(Part):
 
     def __init__(self, dtype, device, width: int, norm1: PartSpec, mixer: PartSpec, norm1b: PartSpec,
                  norm2: "PartSpec | None" = None, ffn: "PartSpec | None" = None, norm2b: "PartSpec | None" = None,
-                 gated: bool = True, names: "dict[str, str] | None" = None, after: "PartSpec | None" = None):
+                 gated: bool = True, names: "dict[str, str] | None" = None, after: "PartSpec | None" = None, spare_norms: bool = False):
         super().__init__(dtype, device)
         self.after = make_part("stream", after, dtype, device) if after is not None else None
         if len({norm2 is None, ffn is None, norm2b is None}) != 1:
             raise ValueError("a second sublayer needs its feed-forward and both of its norms")
         self.names = dict(self.DEFAULT_NAMES, **(names or {}))
         self.width, self.gated = int(width), bool(gated)
+        self.spare_norms = bool(spare_norms) and ffn is None
         self.norm1 = make_part("norm", norm1, dtype, device)
         self.mixer = make_part("mixer", mixer, dtype, device)
         self.norm1b = make_part("norm", norm1b, dtype, device)
@@ -239,10 +241,14 @@ class SandwichBlock(Part):
 
     def tensors(self):
         from ..weights.specs import TensorSpec
+        if self.spare_norms:
+            spare = {self.names[k]: TensorSpec((self.width,), role="vector", optional=True) for k in ("norm2", "norm2b")}
+        else:
+            spare = {}
         if not self.gated:
-            return {}
+            return spare
         n, W = self.names, self.width
-        t = {n["gate1"]: TensorSpec((W, W)), n["gate1_bias"]: TensorSpec((W,), role="vector")}
+        t = {**spare, n["gate1"]: TensorSpec((W, W)), n["gate1_bias"]: TensorSpec((W,), role="vector")}
         if self.ffn is not None:
             t.update({n["gate2"]: TensorSpec((W, W)), n["gate2_bias"]: TensorSpec((W,), role="vector")})
         return t

@@ -9,6 +9,20 @@ from ..weights.specs import TensorSpec
 from .base import Part, PartSpec, make_part, register_part
 
 
+def _limit(activation: str, limit: "float | None") -> float:
+    """The bound of a clamped gate; no other activation has one."""
+    if (activation == "clamped") != (limit is not None) or (limit is not None and not float(limit) > 0):
+        raise ValueError(f"activation {activation!r} with limit {limit}: 'clamped' needs a positive one, the others have none")
+    return float(limit or 0.0)
+
+
+def _kind(activation: str, limit: float) -> dict:
+    """The keyword arguments of a gated product beyond its default, silu."""
+    if activation == "clamped":
+        return {"kind": activation, "limit": limit}
+    return {} if activation == "silu" else {"kind": activation}
+
+
 class GatedMLP(Part):
     """down(act(gate(h)) * up(h)) without biases.  The gate and up weights are stacked
     into one [2 I, width] matrix at load, so one product feeds the activation; in bfloat16,
@@ -16,7 +30,9 @@ class GatedMLP(Part):
     output tile of the product holds both halves and the activation runs in its epilogue.
     ``names``: the checkpoint's names of the three projections (default gate_proj, up_proj, down_proj);
     ``weight_suffix``: what follows a projection's name (".weight").  ``activation``: ``silu`` or ``relu``
-    (both in the product's epilogue), or ``gelu_tanh`` (product, then the activation kernel on the stacked [gates | ups])."""
+    (both in the product's epilogue), or ``gelu_tanh`` (product, then the activation kernel on the stacked [gates | ups]);
+    ``clamped`` with ``limit`` (in the epilogue): g sigmoid(1.702 g) (u + 1) for g = min(gate(h), limit) and
+    u = clamp(up(h), -limit, limit)."""
 
     DEFAULT_NAMES = {"gate": "gate_proj", "up": "up_proj", "down": "down_proj"}
 
@@ -24,8 +40,9 @@ class GatedMLP(Part):
     takes_scaled_rows = True      # ``h`` may be ``ops.ScaledRows``: the gate/up product applies the norm's 1/rms itself
 
     def __init__(self, dtype, device, width: int, intermediate: int, activation: str = "silu",
-                 names: "dict[str, str] | None" = None, weight_suffix: str = ".weight"):
+                 names: "dict[str, str] | None" = None, weight_suffix: str = ".weight", limit: "float | None" = None):
         super().__init__(dtype, device)
+        self.limit = _limit(activation, limit)
         self.names = dict(self.DEFAULT_NAMES, **(names or {}))
         self.suffix = str(weight_suffix)
         self.width, self.intermediate = int(width), int(intermediate)
@@ -63,9 +80,9 @@ class GatedMLP(Part):
     def forward(self, ctx, h):
         with lib.section("gate_up"):
             if self.in_product:
-                act = ops.gated_linear(h, self.w_gate_up, self.interleaved, **({} if self.activation == "silu" else {"kind": self.activation}))
+                act = ops.gated_linear(h, self.w_gate_up, self.interleaved, **_kind(self.activation, self.limit))
             else:
-                act = ops.act_mul(ops.materialize(ops.linear(h, self.w_gate_up)), self.activation)
+                act = ops.act_mul(ops.materialize(ops.linear(h, self.w_gate_up)), self.activation, **({"limit": self.limit} if self.limit else {}))
         with lib.section("down"):
             return ops.linear(act, self.w_down, partials_ok=True, deferred_ok="residual")
 
@@ -137,7 +154,10 @@ class RoutedMLP(Part):
     is added (names under ``shared``), or None.
     ``gated=False``: an expert is down(act(up(h))) with ``activation`` silu, gelu_tanh or relu2 (no gate projection).
     ``router_bias``: a bias per router output added to the logits (name ``router_bias``).  ``renormalise``: the chosen
-    weights are divided by their sum (with softmax scores: the softmax over the chosen logits alone).
+    weights are divided by their sum plus ``renorm_eps`` (with softmax scores: the softmax over the chosen logits alone).
+    ``groups``: (count, keep): the router outputs form so many equal groups of neighbours, a group's score is the sum of its
+    two largest choice scores, and only outputs of the ``keep`` best groups can be chosen.
+    ``activation="clamped"`` (gated experts): with ``limit`` for the experts and ``shared_limit`` for the shared one.
     ``shared_gate``: the shared expert's result is multiplied by sigmoid(w_sg . h), one number per token (name
     ``shared_gate``, a tensor [1, width]).
 
@@ -154,8 +174,15 @@ class RoutedMLP(Part):
     def __init__(self, dtype, device, width: int, intermediate: int, n_experts: int, top: int, scale: float = 1.0,
                  n_identity: int = 0, activation: str = "silu", correction: bool = True, names: "dict[str, str] | None" = None,
                  scores: str = "softmax", weight_on: str = "output", shared: "int | None" = None, gated: bool = True,
-                 router_bias: bool = False, renormalise: bool = False, shared_gate: bool = False):
+                 router_bias: bool = False, renormalise: bool = False, shared_gate: bool = False, renorm_eps: float = 0.0,
+                 groups: "tuple | None" = None, limit: "float | None" = None, shared_limit: "float | None" = None):
         super().__init__(dtype, device)
+        self.limit = _limit(activation, limit)
+        self.renorm_eps = float(renorm_eps)
+        self.groups, self.keep = (int(groups[0]), int(groups[1])) if groups is not None else (1, 1)
+        outs = int(n_experts) + int(n_identity)
+        if self.groups > 1 and (outs % self.groups or not 0 < self.keep <= self.groups or int(top) > self.keep * (outs // self.groups)):
+            raise ValueError(f"{self.keep} of {self.groups} groups of {outs} router outputs cannot give {top}")
         self.gated, self.router_bias, self.renormalise = bool(gated), bool(router_bias), bool(renormalise)
         self.shared_gate = bool(shared_gate) and bool(shared)
         if self.router_bias and int(n_identity):
@@ -168,7 +195,7 @@ class RoutedMLP(Part):
         self.names = dict(self.DEFAULT_NAMES, **(names or {}))
         self.width, self.intermediate = int(width), int(intermediate)
         self.n_experts, self.n_identity, self.top, self.scale = int(n_experts), int(n_identity), int(top), float(scale)
-        known = ops.ACTIVATIONS if self.gated else {k: v for k, v in ops.BIAS_ACTIVATIONS.items() if k not in (None, "tanh")}
+        known = ops.MUL_ACTIVATIONS if self.gated else {k: v for k, v in ops.BIAS_ACTIVATIONS.items() if k not in (None, "tanh")}
         if activation not in known:
             raise ops.UnsupportedSize(f"activation {activation!r}: implemented are {sorted(known)}")
         if self.n_experts <= 0 or self.n_identity < 0 or not 0 < self.top <= self.n_experts + self.n_identity:
@@ -180,7 +207,7 @@ class RoutedMLP(Part):
             self.shared = None
         elif self.gated:
             self.shared = make_part("ffn", PartSpec("gated_mlp", {
-                "width": self.width, "intermediate": int(shared), "activation": activation, "weight_suffix": "",
+                "width": self.width, "intermediate": int(shared), "activation": activation, "weight_suffix": "", "limit": shared_limit,
                 "names": {"gate": n["gate"], "up": n["up"], "down": n["down"]}}), dtype, device)
         else:
             self.shared = make_part("ffn", PartSpec("dense_mlp", {
@@ -228,7 +255,9 @@ class RoutedMLP(Part):
         h = ops.materialize(h)
         T = h.shape[0]
         idx, weight = ops.route(h, self.w_router, self.correction, self.top, self.scale, sigmoid=self.sigmoid,
-                                bias=self.b_router, renormalise=self.renormalise)
+                                bias=self.b_router, renormalise=self.renormalise,
+                                **({"renorm_eps": self.renorm_eps} if self.renorm_eps else {}),
+                                **({"groups": self.groups, "keep": self.keep} if self.groups > 1 else {}))
         offsets, place_of, src = ops.group_pairs(idx, self.n_experts)
         places = T * self.top
         x = h
@@ -238,7 +267,7 @@ class RoutedMLP(Part):
             weight = torch.ones_like(weight)
         with lib.section("experts_gate_up"):
             gu = ops.expert_linear(x, self.w_gate_up, offsets, src, places)
-        act = ops.act_mul(gu, self.activation) if self.gated else ops.bias_act(gu, None, self.activation)
+        act = ops.act_mul(gu, self.activation, **({"limit": self.limit} if self.limit else {})) if self.gated else ops.bias_act(gu, None, self.activation)
         with lib.section("experts_down"):
             y = ops.expert_linear(act, self.w_down, offsets, None, places, out_dtype=torch.float32)
         out = ops.combine_pairs(y, h, place_of, weight)

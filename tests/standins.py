@@ -114,12 +114,14 @@ def linear_act(x, w, kind):
 
 
 def qk_norm_rope_write(proj, q_col, k_col, v_col, q_weight, k_weight, eps, cos, sin, cache_layer, slot_mapping, n_heads,
-                       n_kv_heads, qk_dim, v_dim, row_dim, rotary_dim, page_size, v_cos=None, v_sin=None, neighbours=False, post_norm=False):
+                       n_kv_heads, qk_dim, v_dim, row_dim, rotary_dim, page_size, v_cos=None, v_sin=None, neighbours=False, post_norm=False, biases=None):
     T = proj.shape[0]
     x = proj.float()
+    q_bias, k_bias, v_bias = biases or (None, None, None)
 
-    def heads(col, n, d, w):
-        t = x[:, col:col + n * d].reshape(T, n, d)
+    def heads(col, n, d, w, bias=None):
+        t = x[:, col:col + n * d]
+        t = (t if bias is None else t + bias).reshape(T, n, d)
         if w is not None:
             t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w
         if rotary_dim:
@@ -128,10 +130,11 @@ def qk_norm_rope_write(proj, q_col, k_col, v_col, q_weight, k_weight, eps, cos, 
             t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
         return torch.nn.functional.pad(t, (0, row_dim - d))
 
-    q = heads(q_col, n_heads, qk_dim, q_weight)
+    q = heads(q_col, n_heads, qk_dim, q_weight, q_bias)
     if cache_layer is not None:
-        k = heads(k_col, n_kv_heads, qk_dim, k_weight)
-        v = x[:, v_col:v_col + n_kv_heads * v_dim].reshape(T, n_kv_heads, v_dim)
+        k = heads(k_col, n_kv_heads, qk_dim, k_weight, k_bias)
+        v = x[:, v_col:v_col + n_kv_heads * v_dim]
+        v = (v if v_bias is None else v + v_bias).reshape(T, n_kv_heads, v_dim)
         if v_cos is not None:      # the values turn over all their dims, by tables of their own
             a, b = v[..., :v_dim // 2], v[..., v_dim // 2:]
             c, sn = v_cos[:, None, :], v_sin[:, None, :]
@@ -144,12 +147,20 @@ def qk_norm_rope_write(proj, q_col, k_col, v_col, q_weight, k_weight, eps, cos, 
     return q.reshape(T, n_heads * row_dim).to(proj.dtype)
 
 
-def sigmoid_gate(a, a_dim, proj, g_col, n_heads, v_dim):
+def _into(rows, out, out_col):
+    if out is None:
+        return rows
+    out[:, out_col:out_col + rows.shape[1]] = rows
+    return out
+
+
+def sigmoid_gate(a, a_dim, proj, g_col, n_heads, v_dim, out=None, out_col=0, scale=1.0):
+    target = out
     T = a.shape[0]
     out = a.float().reshape(T, n_heads, a_dim)[..., :v_dim].reshape(T, n_heads * v_dim)
     if proj is not None:
         out = out * torch.sigmoid(proj[:, g_col:g_col + n_heads * v_dim].float())
-    return out.to(a.dtype)
+    return _into((out * scale).to(a.dtype), target, out_col)
 
 
 def head_gate(a, a_dim, proj, g_col, n_heads, v_dim, cos=None, sin=None):
@@ -177,6 +188,9 @@ def add_row_vector(x, v):
 
 
 def gated_norm(y, y_bias, gate, gate_bias, weight, eps, act_dtype, center=True, out_bias=None):
+    from pyre_b200.kernels import ops
+    if isinstance(y, ops.BiasedRows):
+        y, y_bias = y.y, y.bias
     v = _partial_sums_or_tensor(y)
     if y_bias is not None:
         v = v + y_bias
@@ -258,13 +272,20 @@ def sgemm_nt(a, w, bias=None, out=None):
     return y if bias is None else y + bias
 
 
-_GATES = {"silu": torch.nn.functional.silu, "relu": torch.relu}
+def _gated(g, u, kind, limit=0.0):
+    if kind == "clamped":
+        assert limit > 0
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        return g * torch.sigmoid(1.702 * g) * (u + 1.0)
+    act = {"silu": torch.nn.functional.silu, "relu": torch.relu,
+           "gelu_tanh": lambda t: torch.nn.functional.gelu(t, approximate="tanh")}[kind]
+    return act(g) * u
 
 
-def silu_mul(gate_up, out=None, block=0, kind="silu"):
+def silu_mul(gate_up, out=None, block=0, kind="silu", limit=0.0):
     assert block == 0, "the float32 path stacks all gates before all ups"
     inter = gate_up.shape[1] // 2
-    return _GATES[kind](gate_up[:, :inter]) * gate_up[:, inter:]
+    return _gated(gate_up[:, :inter], gate_up[:, inter:], kind, limit)
 
 
 def sample(logits, temperature=None, seeds=None, token_index=None, out=None):
@@ -317,10 +338,9 @@ def stream_set(x, base, product):
     x.copy_(base + _branch(product))
 
 
-def act_mul(gate_up, kind):
+def act_mul(gate_up, kind, limit=0.0):
     g, u = gate_up.float().chunk(2, dim=1)
-    a = torch.nn.functional.gelu(g, approximate="tanh") if kind == "gelu_tanh" else _GATES[kind](g)
-    return (a * u).to(gate_up.dtype)
+    return _gated(g, u, kind, limit).to(gate_up.dtype)
 
 
 def _turn_pairs(v, cos, sin, rot, halves=False):
@@ -396,16 +416,21 @@ def headwise_linear(x, w, out=None):
     return out
 
 
-def route(h, w, correction, top, scale, sigmoid=False, bias=None, renormalise=False):
+def route(h, w, correction, top, scale, sigmoid=False, bias=None, renormalise=False, renorm_eps=0.0, groups=1, keep=1):
     z = h.float() @ w.t()
     if bias is not None:
         z = z + bias
     s = torch.sigmoid(z) if sigmoid else torch.softmax(z, dim=-1)
     choice = s if correction is None else s + correction
+    if groups > 1:
+        by_group = choice.reshape(choice.shape[0], groups, -1)
+        best_two = by_group.topk(min(2, by_group.shape[-1]), dim=-1).values.sum(-1)
+        kept = torch.zeros_like(best_two, dtype=torch.bool).scatter(1, best_two.topk(keep, dim=-1).indices, True)
+        choice = torch.where(kept[:, :, None], by_group, torch.full_like(by_group, float("-inf"))).reshape(choice.shape)
     idx = choice.topk(top, dim=-1).indices
     weight = s.gather(-1, idx) * scale
     if renormalise:
-        weight = weight / weight.sum(-1, keepdim=True)
+        weight = weight / (weight.sum(-1, keepdim=True) + renorm_eps)
     return idx.to(torch.int32), weight
 
 
@@ -456,6 +481,70 @@ def ssm_scan(xbc, proj, dt_col, dt_bias, a_log, d_skip, state_layer, slots, cu_s
             S.mul_(dec[t][:, None, None]).add_((dt[t][:, None] * x[t])[:, None, :] * B[t][:, :, None])
             y[t] = torch.einsum("hnp,hn->hp", S, C[t]) + d_skip[:, None] * x[t]
     return y.reshape(T, H * P)
+
+
+def channel_decay(proj, col, rank, weight, bias, tau):
+    return torch.nn.functional.logsigmoid(proj[:, col:col + rank].float() @ weight + bias) / tau
+
+
+def gated_linear_attention(proj, q_col, k_col, v_col, q_scale, logd, state_layer, slots, cu_seqlens, n_heads, qk_dim, v_dim, lens=None,
+                           chunked=None):
+    T, x = proj.shape[0], proj.float()
+    q = x[:, q_col:q_col + n_heads * qk_dim].reshape(T, n_heads, qk_dim) * q_scale
+    k = x[:, k_col:k_col + n_heads * qk_dim].reshape(T, n_heads, qk_dim)
+    v = x[:, v_col:v_col + n_heads * v_dim].reshape(T, n_heads, v_dim)
+    keep = logd.exp().reshape(T, n_heads, qk_dim, 1)
+    out = torch.empty((T, n_heads, v_dim))
+    cu = cu_seqlens.tolist()
+    assert lens is None or [b - a for a, b in zip(cu, cu[1:])] == list(lens)
+    for b in range(len(cu) - 1):
+        S = state_layer[int(slots[b])].view(-1)[:n_heads * qk_dim * v_dim].view(n_heads, qk_dim, v_dim)      # updated in place
+        for t in range(cu[b], cu[b + 1]):
+            S.mul_(keep[t]).add_(k[t][:, :, None] * v[t][:, None, :])
+            out[t] = (S * q[t][:, :, None]).sum(1)
+    return out.reshape(T, n_heads * v_dim)
+
+
+def matrix_memory(proj, q_col, k_col, v_col, q_scale, gates, gate_bias, cap, state_layer, slots, cu_seqlens, n_heads, qk_dim, v_dim,
+                  lens=None, chunked=None):
+    T, x, H = proj.shape[0], proj.float(), n_heads
+    q = x[:, q_col:q_col + H * qk_dim].reshape(T, H, qk_dim) * q_scale
+    k = x[:, k_col:k_col + H * qk_dim].reshape(T, H, qk_dim)
+    v = x[:, v_col:v_col + H * v_dim].reshape(T, H, v_dim)
+    z = cap * torch.tanh((_partial_sums_or_tensor(gates) + gate_bias) / cap)
+    gi, gf = z[:, :H], torch.nn.functional.logsigmoid(z[:, H:])
+    out, den = torch.empty((T, H, v_dim)), torch.empty((T, H))
+    cu = cu_seqlens.tolist()
+    for b in range(len(cu) - 1):
+        flat = state_layer[int(slots[b])].view(-1)
+        S = flat[:H * qk_dim * v_dim].view(H, qk_dim, v_dim)
+        n = flat[H * qk_dim * v_dim:H * qk_dim * (v_dim + 1)].view(H, qk_dim)
+        copies = flat[H * qk_dim * (v_dim + 1):H * (qk_dim * (v_dim + 1) + -(-v_dim // 16) + 1)].view(H, -1)
+        m = copies[:, 0].clone()
+        assert (copies == m[:, None]).all(), "the copies of the running maximum differ"
+        for t in range(cu[b], cu[b + 1]):
+            after = torch.maximum(gf[t] + m, gi[t])
+            keep, put = torch.exp(gf[t] + m - after), torch.exp(gi[t] - after)
+            S.mul_(keep[:, None, None]).add_(put[:, None, None] * k[t][:, :, None] * v[t][:, None, :])
+            n.mul_(keep[:, None]).add_(put[:, None] * k[t])
+            m = after
+            out[t] = (S * q[t][:, :, None]).sum(1)
+            den[t] = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+        copies.copy_(m[:, None].expand_as(copies))
+    return out.reshape(T, H * v_dim), den
+
+
+def heads_finish(o, den, weight, eps, proj, g_col, n_heads, v_dim, out_dtype, gate="silu", post=1.0, out=None, out_col=0):
+    T = o.shape[0]
+    u = o.reshape(T, n_heads, v_dim)
+    if den is not None:
+        u = u / den[:, :, None]
+    u = u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps)
+    u = (u * weight if weight.shape[0] == v_dim else u * weight.view(n_heads, v_dim)).reshape(T, n_heads * v_dim)
+    if proj is not None:
+        z = proj[:, g_col:g_col + n_heads * v_dim].float()
+        u = u * (torch.nn.functional.silu(z) if gate == "silu" else torch.sigmoid(z))
+    return _into((u * post).to(out_dtype), out, out_col)
 
 
 def group_norm_gate(y, groups, weight, eps, proj, g_col, out_dtype, gate="silu", gate_first=False, post=1.0):
@@ -556,7 +645,9 @@ def install(monkeypatch) -> None:
                          add_row_vector=add_row_vector, gated_norm=gated_norm, scale_to_places=scale_to_places,
                          token_shift_mix=token_shift_mix, wkv_scan=wkv_scan, scale_cap=scale_cap, short_conv=short_conv,
                          ssm_scan=ssm_scan, group_norm_gate=group_norm_gate, diff_combine=diff_combine, rotate_heads=rotate_heads,
-                         side_gate=side_gate, token_gate_add=token_gate_add, stream_rows=stream_rows, stream_set=stream_set).items():
+                         side_gate=side_gate, token_gate_add=token_gate_add, stream_rows=stream_rows, stream_set=stream_set,
+                         channel_decay=channel_decay, gated_linear_attention=gated_linear_attention, matrix_memory=matrix_memory,
+                         heads_finish=heads_finish).items():
         monkeypatch.setattr(ops, name, fn)
     monkeypatch.setattr(ops, "device_error_flag", lambda device: flag)
     monkeypatch.setattr(ops, "check_device_errors", lambda device="cpu": None)
@@ -591,12 +682,14 @@ def qkv_rope_write_any(qkv, bias, cos, sin, cache_layer, slot_mapping, n_heads, 
 
 def materialize(t):
     from pyre_b200.kernels import ops
+    if isinstance(t, ops.BiasedRows):
+        return bias_act(materialize(t.y), t.bias, None)
     if isinstance(t, ops.DeferredProduct):
         t = t.partials()
     return t.parts.sum(0).to(t.dtype) if isinstance(t, ops.PartialSums) else t
 
 
-def gemm_tc(x, w, out_dtype=torch.bfloat16, plan=None, reduce=True, gated=False, pair=None, checked=False):
+def gemm_tc(x, w, out_dtype=torch.bfloat16, plan=None, reduce=True, gated=False, pair=None, checked=False, limit=0.0):
     from pyre_b200.kernels import ops
     assert x.dtype == w.dtype == torch.bfloat16 and x.shape[1] == w.shape[1]
     M, K = x.shape
@@ -607,7 +700,7 @@ def gemm_tc(x, w, out_dtype=torch.bfloat16, plan=None, reduce=True, gated=False,
     if gated:
         assert N % (2 * ops.GATED_BLOCK) == 0
         y = (x.float() @ w.float().t()).view(M, N // (2 * ops.GATED_BLOCK), 2, ops.GATED_BLOCK)
-        return (_GATES["silu" if gated is True else gated](y[:, :, 0]) * y[:, :, 1]).reshape(M, N // 2).to(torch.bfloat16)
+        return _gated(y[:, :, 0], y[:, :, 1], "silu" if gated is True else gated, limit).reshape(M, N // 2).to(torch.bfloat16)
     per = -(-kb // splits) * 64
     parts = torch.stack([x[:, s * per:(s + 1) * per].float() @ w[:, s * per:(s + 1) * per].float().t() for s in range(splits)])
     if splits == 1 and reduce:
@@ -617,12 +710,12 @@ def gemm_tc(x, w, out_dtype=torch.bfloat16, plan=None, reduce=True, gated=False,
     return parts.sum(0).to(out_dtype)
 
 
-def silu_mul_any(gate_up, out=None, block=0, kind="silu"):
+def silu_mul_any(gate_up, out=None, block=0, kind="silu", limit=0.0):
     if block == 0:
-        return silu_mul(gate_up.float(), kind=kind).to(gate_up.dtype)
+        return silu_mul(gate_up.float(), kind=kind, limit=limit).to(gate_up.dtype)
     T, two_i = gate_up.shape
     y = gate_up.float().view(T, two_i // (2 * block), 2, block)
-    return (_GATES[kind](y[:, :, 0]) * y[:, :, 1]).reshape(T, two_i // 2).to(gate_up.dtype)
+    return _gated(y[:, :, 0], y[:, :, 1], kind, limit).reshape(T, two_i // 2).to(gate_up.dtype)
 
 
 def _attend_entries(q, cache_layer, block_table, cu_seqlens, positions, n_seqs, n_heads, n_kv_heads, head_dim, scale, window,
