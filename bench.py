@@ -1189,6 +1189,124 @@ def run_gadopel(args) -> dict:
     return out
 
 
+def run_gugidra(args) -> dict:
+    """``--workload gugidra``: the Gugidra design (random weights) at two sets of layer sizes, two layers that run twice
+    (gated linear attention with a clamped dense feed-forward; attention over its own keys beside a matrix memory, with
+    experts chosen in groups and a shared one), beside the package's closest layers at equal sizes: Tekarax's recurrent
+    layer with a dense feed-forward and its attention layer with routed experts, run as often, and two of Modovik's
+    constant-decay layers with dense feed-forwards, whose state is the matrix memory's.  A 2,048-token prompt step and
+    decode steps at batch 8 and 64 with 2,048 tokens of context, device-timed, and per kernel class the device time of one
+    such step with the fraction of the measured peak."""
+    import numpy as np
+
+    from pyre_b200.config import config_from_dict
+
+    peaks = load_peaks()
+    V = 32768
+    sizes = {
+        # width; attention heads of 128 over key/value heads (and as many memory heads of 128 x 128); recurrent head size and
+        # the decay map's inner size; dense feed-forward; experts in groups of which some are kept, chosen, their size, shared
+        "2k": dict(H=2048, nh=16, nkv=4, hd=128, wd=64, wr=64, I=8192, E=32, groups=8, keep=4, top=4, ff=1024, sh=2048),
+        "3.5k": dict(H=3584, nh=28, nkv=4, hd=128, wd=64, wr=96, I=18944, E=64, groups=8, keep=4, top=6, ff=1408, sh=2816),
+    }
+    T, ctx_len, times = PROMPT_LEN, 2048, 2
+    rng = np.random.default_rng(0)
+    out = {"workload": "gugidra", "peaks": peaks, "prompt": T, "decode_context": ctx_len, "sizes": {}}
+    for tag, z in sizes.items():
+        H, nh, nkv, hd, wd, wr, I, E, top, ff, sh = (z[k] for k in ("H", "nh", "nkv", "hd", "wd", "wr", "I", "E", "top", "ff", "sh"))
+        wh = H // wd
+        q, kv, whd = nh * hd, nkv * hd, wh * wd
+        dense = {"kind": "dense", "ff": I}
+        loop = {"start": 0, "stop": 2, "times": times}
+        raw_g = {"architecture": "Gugidra", "vocab": V, "width": H, "norm": {"eps": 1e-6}, "embedding": {"scale": H ** 0.5},
+                 "logit_softcap": 30.0, "loop": loop, "layers": [
+            {"type": "gla", "mixer": {"heads": wh, "dim": wd, "vdim": wd, "tau": 16.0, "decay_rank": wr}, "mlp": dict(dense, limit=7.0)},
+            {"type": "parallel", "mixer": {
+                "left": {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "rot": {"dims": hd, "base": 1e6}},
+                "right": {"heads": nh, "dim": hd, "vdim": hd, "gate_cap": 15.0}, "left_scale": 0.7, "right_scale": 0.8},
+             "mlp": {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": E, "top": top, "groups": {"count": z["groups"], "keep": z["keep"]}},
+                     "shared": {"ff": sh, "limit": 7.0}}}]}
+        raw_t = {"architecture": "Tekarax", "vocab": V, "width": H, "norm": {"eps": 1e-6}, "loop": loop, "layers": [
+            {"type": "wkv", "mixer": {"heads": wh, "dim": wd, "decay_rank": wr}, "mlp": dense},
+            {"type": "attention", "mixer": {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "rot": {"dims": hd, "base": 1e6}},
+             "mlp": {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": E, "top": top}, "shared": {"ff": sh}}}]}
+        raw_m = {"architecture": "Modovik", "vocab": V, "width": H, "norm": {"eps": 1e-6}, "layers": [
+            {"type": "lightning", "mixer": {"heads": nh, "dim": hd, "vdim": hd, "decay": [1.0 - 2.0 ** (-5 - 3 * i / nh) for i in range(nh)]},
+             "mlp": dense}] * times}
+
+        def pairs(Tn, B, before):
+            return B * float((np.arange(before, before + Tn // B) + 1).sum())
+
+        def product(rows, cols, Tn, n):
+            return {"bytes": n * (rows * cols * 2 + Tn * (rows + cols) * 2), "flops": 2.0 * n * Tn * rows * cols}
+
+        def state(Tn, B, heads, dim, n, extra=0):
+            """a recurrence over [dim, dim] states: q, k, v in, fp32 values out (and ``extra`` bytes per token), the state in and out"""
+            w = heads * dim
+            return {"bytes": n * (Tn * (w * (3 * 2 + 4) + extra) + B * 2 * heads * dim * dim * 4), "flops": 4.0 * n * Tn * heads * dim * dim}
+
+        def attention(Tn, B, before, n):
+            return {"bytes": n * (B * (before + Tn // B) * 2 * kv * 2 + 2 * Tn * q * 2), "flops": 4.0 * n * nh * hd * pairs(Tn, B, before)}
+
+        def routed(Tn, n):
+            chosen = Tn * top
+            used = min(E, chosen)
+            return {"experts_gate_up": {"bytes": n * (used * 2 * ff * H * 2 + chosen * (H + 2 * ff) * 2), "flops": 4.0 * n * chosen * H * ff},
+                    "experts_down": {"bytes": n * (used * H * ff * 2 + chosen * (ff * 2 + H * 4)), "flops": 2.0 * n * chosen * H * ff},
+                    "router": {"bytes": n * (E * H * 4 + Tn * H * 2 + chosen * H * 4 + Tn * H * 4), "flops": 2.0 * n * Tn * H * E}}
+
+        def tail(Tn, B):
+            return {"head": {"bytes": V * H * 2 + B * (H * 2 + V * 4), "flops": 2.0 * B * H * V}, "embed": {"bytes": Tn * H * (2 + 4), "flops": 0}}
+
+        def work_gugidra(Tn, B, before):
+            cols = 4 * whd + wr + q + kv + 4 * q
+            return {
+                "qkv": {"bytes": times * (cols * H * 2 + Tn * (2 * H + cols) * 2), "flops": 2.0 * times * Tn * H * cols},
+                "gates": {"bytes": times * (2 * nh * H * 2 + Tn * (H * 2 + 2 * nh * 4)), "flops": 2.0 * times * Tn * H * 2 * nh},
+                "decay": {"bytes": times * (whd * wr * 4 + Tn * (wr * 2 + whd * 4)), "flops": 2.0 * times * Tn * wr * whd},
+                "recurrence": state(Tn, B, wh, wd, times, extra=whd * 4), "matrix_memory": state(Tn, B, nh, hd, times, extra=nh * 12),
+                "attention": attention(Tn, B, before, times),
+                "o": {"bytes": times * ((whd + 2 * q) * H * 2 + Tn * (whd + 2 * q + 2 * H) * 2), "flops": 2.0 * times * Tn * H * (whd + 2 * q)},
+                "gate_up": {"bytes": times * (2 * (I + sh) * H * 2 + Tn * (2 * H + I + sh) * 2), "flops": 4.0 * times * Tn * H * (I + sh)},
+                "down": {"bytes": times * ((I + sh) * H * 2 + Tn * (I + sh + 2 * H) * 2), "flops": 2.0 * times * Tn * H * (I + sh)},
+                "activation": {"bytes": times * Tn * top * 3 * ff * 2, "flops": 0},
+                "norm": {"bytes": Tn * H * (2 + 4 + 4 + 2), "flops": 0, "per_launch": True},
+                "gate": {"bytes": times * Tn * ((whd + q) * (4 + 2 + 2) + q * (2 + 2)), "flops": 0},
+                "rotary+write": {"bytes": times * Tn * (q + 2 * kv) * 2 * 2, "flops": 0},
+                **routed(Tn, times), **tail(Tn, B)}
+
+        def work_tekarax(Tn, B, before):
+            cols = 4 * whd + q + 2 * kv + nh
+            return {
+                "qkv": {"bytes": times * (cols * H * 2 + Tn * (5 * H + cols) * 2), "flops": 2.0 * times * Tn * H * cols},
+                "decay": {"bytes": times * ((wr * H + whd * wr) * 2 + Tn * (H + 2 * wr) * 2 + Tn * whd * 4), "flops": 2.0 * times * Tn * wr * (H + whd)},
+                "recurrence": {"bytes": times * (Tn * (H * 2 * 6 + whd * (2 * 5 + 4)) + B * (2 * wh * wd * wd + 2 * H) * 4), "flops": 6.0 * times * Tn * wh * wd * wd},
+                "attention": attention(Tn, B, before, times),
+                "o": {"bytes": times * ((whd + q) * H * 2 + Tn * (whd + q + 2 * H) * 2), "flops": 2.0 * times * Tn * H * (whd + q)},
+                "up": product(I, H, Tn, times), "gate_up": product(2 * sh, H, Tn, times),
+                "down": {"bytes": times * ((I + sh) * H * 2 + Tn * (I + sh + 2 * H) * 2), "flops": 2.0 * times * Tn * H * (I + sh)},
+                "residual_gate": product(H, H, Tn, 4 * times),
+                "activation": {"bytes": times * (Tn * I * 4 + Tn * top * 3 * ff * 2), "flops": 0},
+                "norm": {"bytes": Tn * H * (2 + 2 + 4 + 4), "flops": 0, "per_launch": True},
+                "gate": {"bytes": Tn * q * (2 + 2), "flops": 0, "per_launch": True},
+                "rotary+write": {"bytes": times * Tn * (q + 2 * kv) * 2 * 2, "flops": 0},
+                **routed(Tn, times), **tail(Tn, B)}
+
+        def work_modovik(Tn, B, before):
+            return {
+                "qkv": product(4 * q, H, Tn, times), "linear_attention": state(Tn, B, nh, hd, times), "o": product(q, H, Tn, times),
+                "up": product(I, H, Tn, times), "down": product(I, H, Tn, times), "activation": {"bytes": times * Tn * I * 4, "flops": 0},
+                "norm": {"bytes": Tn * H * (2 + 4 + 4 + 2), "flops": 0, "per_launch": True},
+                "gate": {"bytes": Tn * q * (4 + 2 + 2), "flops": 0, "per_launch": True}, **tail(Tn, B)}
+
+        block = {"sizes": dict(z, recurrent_heads=wh), "models": {}}
+        for name, raw, work in (("gugidra", raw_g, work_gugidra), ("tekarax", raw_t, work_tekarax), ("modovik", raw_m, work_modovik)):
+            block["models"][name] = dict(layers=len(raw["layers"]), times=1 if name == "modovik" else times,
+                                         **_measure_design(config_from_dict(raw), work, args, peaks, V, T, ctx_len, rng))
+        out["sizes"][tag] = block
+    return out
+
+
 def run_sweep(args) -> dict:
     """Decode throughput over a grid of batch sizes and context lengths and prefill throughput over
     several portion lengths on the 7B shape, each with its fraction of the roofline (device-timed,
@@ -1312,11 +1430,11 @@ def main() -> int:
                     help="leave out the points at longer contexts and at the 14B and 32B shapes")
     ap.add_argument("--no-per-kernel", action="store_true",
                     help="leave out the `kernels` block (device time, bytes or flops and fraction of the peak per kernel class)")
-    ap.add_argument("--workload", choices=["serve14b", "mixed32b", "sweep", "modovik", "pivinex", "tekarax", "nipudra", "gadopel"], default=None,
+    ap.add_argument("--workload", choices=["serve14b", "mixed32b", "sweep", "modovik", "pivinex", "tekarax", "nipudra", "gadopel", "gugidra"], default=None,
                     help="run one of the two other baseline workloads, a sweep over batch sizes, context lengths and "
                          "portion lengths on the 7B shape, the Modovik or the Pivinex design beside the Qwen2.5 decoder at "
-                         "equal layer sizes, the Tekarax design beside the closest layers of those two, or the Nipudra design beside the closest "
-                         "layers of Tekarax and Modovik, or the Gadopel design beside the closest layers of Pivinex and Tekarax, instead (prints its own JSON line)")
+                         "equal layer sizes, the Tekarax design beside the closest layers of those two, the Nipudra design beside the closest "
+                         "layers of Tekarax and Modovik, the Gadopel design beside the closest layers of Pivinex and Tekarax, or the Gugidra design beside the closest layers of Tekarax and Modovik, instead (prints its own JSON line)")
     ap.add_argument("--cache-fraction", type=float, default=1.0,
                     help="serve14b: cache capacity as a fraction of what all requests need at once (< 1 forces preemption)")
     args = ap.parse_args()
@@ -1326,7 +1444,7 @@ def main() -> int:
     if args.workload:
         result = run_sweep(args) if args.workload == "sweep" else run_modovik(args) if args.workload == "modovik" else \
             run_pivinex(args) if args.workload == "pivinex" else run_tekarax(args) if args.workload == "tekarax" else run_nipudra(args) if args.workload == "nipudra" else \
-            run_gadopel(args) if args.workload == "gadopel" else run_workload(args)
+            run_gadopel(args) if args.workload == "gadopel" else run_gugidra(args) if args.workload == "gugidra" else run_workload(args)
         result["env"] = environment()
         print(json.dumps(result))
         return 0

@@ -666,6 +666,99 @@ PYRE_API int pyre_gated_norm(const void* y, const float* partials, int n_partial
 }
 
 // ---------------------------------------------------------------------------
+// The norm of a sublayer's result, the stream's update and the next sublayer's norm in one pass over the row:
+//   v      = y[src] + y_bias          src = rows[r] or r; y: activation dtype, or the sum of n_partials fp32 partial sums
+//   s      = x[src] + v / sqrt(mean(v^2) + eps_b) * w_b;      x[src] = s (update_x, without rows)
+//   out[r] = T( s / sqrt(mean(s^2) + eps) * w )
+// The arithmetic of gated_norm (without gate and centre) and add_rmsnorm behind one another.  One block per row; a thread
+// keeps its KEEP vectors of the row in registers; the block size depends on H only.
+// ---------------------------------------------------------------------------
+template <typename T, int VEC, int KEEP>
+__global__ void normed_add_norm_kernel(float* x, const T* y, const float* partials, int n_partials, long long partial_stride, const float* y_bias,
+                                       const float* w_b, float eps_b, const float* w, float eps, T* out, const int* rows, int H, int update_x) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const int r = blockIdx.x, src = rows ? rows[r] : r;
+    const T* yr = y ? y + (size_t)src * H : nullptr;
+    const float* pr = partials ? partials + (size_t)src * H : nullptr;
+    float* xr = x + (size_t)src * H;
+    Vec<float, VEC> v[KEEP], xs[KEEP];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * VEC;
+        if (i >= H) continue;
+        xs[j] = load_vec<float, VEC>(xr + i);
+        if (pr) {
+            v[j] = load_vec<float, VEC>(pr + i);
+            for (int p = 1; p < n_partials; ++p) {
+                const Vec<float, VEC> q = load_vec<float, VEC>(pr + (size_t)p * partial_stride + i);
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) v[j].v[k] += q.v[k];
+            }
+        } else {
+            const Vec<T, VEC> a = load_vec<T, VEC>(yr + i);
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) v[j].v[k] = to_f32<T>(a.v[k]);
+        }
+        if (y_bias) {
+            const Vec<float, VEC> b = load_vec<float, VEC>(y_bias + i);
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) v[j].v[k] += b.v[k];
+        }
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) ss = fmaf(v[j].v[k], v[j].v[k], ss);
+    }
+    const float rstd_b = 1.0f / sqrtf(block_sum(ss, scratch) / (float)H + eps_b);
+    ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * VEC;
+        if (i >= H) continue;
+        const Vec<float, VEC> g = load_vec<float, VEC>(w_b + i);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+            xs[j].v[k] = xs[j].v[k] + __fmul_rn(__fmul_rn(v[j].v[k], rstd_b), g.v[k]);
+            ss = fmaf(xs[j].v[k], xs[j].v[k], ss);
+        }
+        if (update_x) store_vec<float, VEC>(xr + i, xs[j]);
+    }
+    const float rstd = 1.0f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * VEC;
+        if (i >= H) continue;
+        const Vec<float, VEC> g = load_vec<float, VEC>(w + i);
+        Vec<T, VEC> o;
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) o.v[k] = from_f32<T>(__fmul_rn(__fmul_rn(xs[j].v[k], rstd), g.v[k]));
+        store_vec<T, VEC>(out + (size_t)r * H + i, o);
+    }
+}
+
+PYRE_API int pyre_normed_add_norm(float* x, const void* y, const float* partials, int n_partials, long long partial_stride, const float* y_bias,
+                                  const float* w_b, float eps_b, const float* w, float eps, void* out, const int* rows, int n_rows, int H,
+                                  int update_x, int dtype, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if ((y == nullptr) == (partials == nullptr) || (partials && n_partials < 1) || H <= 0 || !x || !w_b || !w || !out || (rows && update_x)) return PYRE_ERR_BAD_ARG;
+    const bool vec = H % 4 == 0 && partial_stride % 4 == 0 &&
+                     (((uintptr_t)x | (uintptr_t)y | (uintptr_t)partials | (uintptr_t)y_bias | (uintptr_t)w_b | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
+    const int per = vec ? H / 4 : H, rounds = ceil_div(per, 512);
+    if (rounds > 8) return PYRE_ERR_UNSUPPORTED;
+    const int threads = ceil_div(ceil_div(per, rounds), 32) * 32;
+#define GO(TT, V, KP) pyre_launch(normed_add_norm_kernel<TT, V, KP>, dim3(n_rows), dim3(threads), 0, stream, x, (const TT*)y, partials, n_partials, partial_stride, y_bias, w_b, eps_b, w, eps, (TT*)out, rows, H, update_x)
+#define PICK(TT, V) do { if (rounds <= 1) GO(TT, V, 1); else if (rounds <= 2) GO(TT, V, 2); else if (rounds <= 4) GO(TT, V, 4); else GO(TT, V, 8); } while (0)
+    if (dtype == PYRE_BF16) { if (vec) PICK(__nv_bfloat16, 4); else PICK(__nv_bfloat16, 1); }
+    else if (dtype == PYRE_F32) { if (vec) PICK(float, 4); else PICK(float, 1); }
+    else return PYRE_ERR_BAD_ARG;
+#undef PICK
+#undef GO
+    PYRE_LAUNCH_CHECK();
+    return 0;
+}
+
+// ---------------------------------------------------------------------------
 // One gate per HEAD on a mixer's output, after turning each head's sum of rotated values back:
 //   u = a[t, h, :dv]                     a head of `a` has a_dim >= dv columns (the rest is dropped)
 //   pairs (m, m + dv / 2) of u turn by MINUS the token's angle (cos, sin [T, dv / 2]; null: no turn)

@@ -1,7 +1,7 @@
 // Recurrences over a matrix state per head whose decays depend on the token, with the state in a slot of the cache
 // manager (fp32, zero when a request begins).  Two kinds:
 //
-//   kind 0, a decay per key channel (gated linear attention), a_t = exp(logd_t) per channel of the head:
+//   kind 0, a decay per key channel (gated linear attention), a_t = sigmoid(z_t + bias)^(1 / tau) per channel of the head:
 //       S_t = diag(a_t) S_(t-1) + k_t v_t^T                       o_t = S_t^T q_t
 //   kind 1, a matrix memory with exponential gates: log input gate i, log forget gate f per head and token, and a running
 //   maximum m (0 when a request begins) that keeps every exponential at most 1:
@@ -26,7 +26,9 @@ struct StateArgs {
     long long row_stride;
     int q_col, k_col, v_col;
     float qscale;
-    const float* logd;           // kind 0: [tokens, H * dk] log decays
+    const float* z;              // kind 0: [tokens, H * dk] raw decays, their bias [H * dk] and 1 / tau
+    const float* z_bias;
+    float inv_tau;
     const float* gates;          // kind 1: raw gates [n_parts][tokens][2 H] (input gates, then forget gates), parts to be added
     int n_parts;
     long long part_stride;
@@ -42,6 +44,8 @@ struct StateArgs {
 };
 
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+// log decay of a head's channel
+__device__ __forceinline__ float log_decay(const StateArgs& a, float z, int channel) { return log_sigmoid(__fadd_rn(z, a.z_bias[channel])) * a.inv_tau; }
 __device__ __forceinline__ int m_copies(int dv) { return (dv + 15) / 16 + 1; }
 
 // a token's raw gate logits of one head: column h the input gate's, column H + h the forget gate's
@@ -57,22 +61,24 @@ __device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tan
 // Token by token.  Grid (tiles of 32 value columns, heads, entries); a CTA of four warps (two for dk <= 16) holds a
 // [dk, 32] tile of the state in registers.  A warp owns eight columns, its lanes split the rows four ways in groups of
 // four (row = 16 g + 4 r + e), so q, k and the decays come from shared memory as conflict-free 16-byte loads and the four
-// row groups of a column meet in two shuffles.  Tokens are staged CH at a time, the next ones on their way into registers
-// meanwhile.  n and den belong to the first warp of tile 0.
+// row groups of a column meet in two shuffles.  Tokens are staged CH at a time (FEW: a step of single tokens, where
+// staging more would only cost registers and instructions), the next ones on their way into registers meanwhile.  n and
+// den belong to the first warp of tile 0.
 // ---------------------------------------------------------------------------
-template <int G> struct ScanShape {
+template <int G, bool FEW> struct ScanShape {
     static constexpr int DP = 16 * G;
     static constexpr int WARPS = G >= 2 ? 4 : 2;
     static constexpr int THREADS = WARPS * 32;
     static constexpr int CT = WARPS * 8;                // columns of a tile
-    static constexpr int CH = G <= 8 ? 16 : 8;          // tokens staged at a time
+    static constexpr int CH = FEW ? (G == 3 ? 8 : 4) : G <= 8 ? 16 : 8;   // tokens staged at a time
     static constexpr int PER = CH * DP / THREADS;       // staged (token, row) pairs per thread
     static constexpr int PERV = CH * CT / THREADS;      // staged (token, column) pairs per thread
+    static_assert(CH * DP % THREADS == 0 && CH * CT % THREADS == 0, "the threads stage whole chunks");
 };
 
 template <int G, int KIND, int U>
 __device__ __forceinline__ void scan_tokens(float (&S)[4 * G], const float (*sq)[16 * G], const float (*sk)[16 * G],
-                                            const float (*sd)[16 * G], const float (*sv)[ScanShape<G>::CT], const float* keep,
+                                            const float (*sd)[16 * G], const float (*sv)[ScanShape<G, false>::CT], const float* keep,
                                             const float* put, int tt, int r, int cw, bool store, float* o_at, size_t o_stride) {
     float acc[U];
 #pragma unroll
@@ -106,9 +112,9 @@ __device__ __forceinline__ void scan_tokens(float (&S)[4 * G], const float (*sq)
     }
 }
 
-template <typename T, int G, int KIND>
-__global__ void __launch_bounds__(ScanShape<G>::THREADS) state_scan_kernel(StateArgs a, int max_len) {
-    using Sh = ScanShape<G>;
+template <typename T, int G, int KIND, bool FEW>
+__global__ void __launch_bounds__(ScanShape<G, FEW>::THREADS) state_scan_kernel(StateArgs a, int max_len) {
+    using Sh = ScanShape<G, FEW>;
     constexpr int DP = Sh::DP, THREADS = Sh::THREADS, CT = Sh::CT, CH = Sh::CH, PER = Sh::PER, PERV = Sh::PERV;
     __shared__ __align__(16) float sq[CH][DP];
     __shared__ __align__(16) float sk[CH][DP];
@@ -164,7 +170,7 @@ __global__ void __launch_bounds__(ScanShape<G>::THREADS) state_scan_kernel(State
             const size_t row = (size_t)(c0 + tt) * a.row_stride + i;
             pq[p] = real ? qs[row] : from_f32<T>(0.f);
             pk[p] = real ? ks[row] : from_f32<T>(0.f);
-            if (KIND == 0) pd[p] = real ? a.logd[((size_t)(c0 + tt) * H + head) * dk + i] : 0.f;
+            if (KIND == 0) pd[p] = real ? a.z[((size_t)(c0 + tt) * H + head) * dk + i] : 0.f;
         }
 #pragma unroll
         for (int p = 0; p < PERV; ++p) {
@@ -186,7 +192,7 @@ __global__ void __launch_bounds__(ScanShape<G>::THREADS) state_scan_kernel(State
             const int e = p * THREADS + tid, tt = e / DP, i = e - tt * DP;
             sq[tt][i] = to_f32<T>(pq[p]) * a.qscale;
             sk[tt][i] = to_f32<T>(pk[p]);
-            if (KIND == 0) sd[tt][i] = expf(pd[p]);
+            if (KIND == 0) sd[tt][i] = i < dk ? expf(log_decay(a, pd[p], head * dk + i)) : 0.f;
         }
 #pragma unroll
         for (int p = 0; p < PERV; ++p) {
@@ -214,7 +220,8 @@ __global__ void __launch_bounds__(ScanShape<G>::THREADS) state_scan_kernel(State
         const bool store = col_ok && r == 0;
         const float (*dd)[DP] = KIND == 0 ? sd : sk;
         int tt = 0;
-        for (; tt + 4 <= n; tt += 4) scan_tokens<G, KIND, 4>(S, sq, sk, dd, sv, keep, put, tt, r, cw, store, o_at, (size_t)H * dv);
+        if (!FEW)
+            for (; tt + 4 <= n; tt += 4) scan_tokens<G, KIND, 4>(S, sq, sk, dd, sv, keep, put, tt, r, cw, store, o_at, (size_t)H * dv);
         for (; tt < n; ++tt) scan_tokens<G, KIND, 1>(S, sq, sk, dd, sv, keep, put, tt, r, cw, store, o_at, (size_t)H * dv);
         if (owns_n) {
             for (tt = 0; tt < n; ++tt) {
@@ -270,7 +277,7 @@ __global__ void __launch_bounds__(ScanShape<G>::THREADS) state_scan_kernel(State
 constexpr int SB = 16;      // tokens of a block
 
 __device__ __forceinline__ void sb_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ uint32_t sb_pack(float lo, float hi) {
@@ -306,6 +313,7 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
     __nv_bfloat16* sK = sQ + SB * QP;                                                           // [16][QP]
     __nv_bfloat16* sV = sK + SB * QP;                                                           // [16][VP]
     __shared__ int where[2];
+    __shared__ float4 half[64];      // the other warp's share of the scores
     pdl_trigger();
     pdl_wait();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
@@ -358,10 +366,13 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
         for (int d = tid; d < KD; d += 128) {
             float x[SB];
 #pragma unroll
-            for (int j = 0; j < SB; ++j) x[j] = (j < n && d < dk) ? a.logd[((size_t)(t0 + j) * H + head) * dk + d] : 0.f;
+            for (int j = 0; j < SB; ++j) x[j] = (j < n && d < dk) ? a.z[((size_t)(t0 + j) * H + head) * dk + d] : 0.f;
             float sum = 0.f;
 #pragma unroll
-            for (int j = 0; j < SB; ++j) { sum += x[j]; sB[j * QP + d] = sum; }
+            for (int j = 0; j < SB; ++j) {
+                if (j < n && d < dk) sum += log_decay(a, x[j], head * dk + d);
+                sB[j * QP + d] = sum;
+            }
         }
     } else if (warp == 0) {
         float f = 0.f, in = 0.f;
@@ -403,7 +414,7 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
                         const int c = d + (e & 1) + (e >> 1) * 8;
-                        x[e] = q_at(i, c) * a.qscale * expf(sB[i * QP + c]);
+                        x[e] = q_at(i, c) * a.qscale * __expf(sB[i * QP + c]);
                     }
                     sb_split(x[0], x[1], w.x, w.z);
                     sb_split(x[2], x[3], w.y, w.w);
@@ -418,7 +429,7 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int j = 2 * t + (e & 1) + (e >> 1) * 8;
-                const float w = KIND == 0 ? expf(sB[(SB - 1) * QP + d] - sB[j * QP + d]) : expf(gb[16 + j] - gb[32 + SB - 1]);
+                const float w = KIND == 0 ? __expf(sB[(SB - 1) * QP + d] - sB[j * QP + d]) : __expf(gb[16 + j] - gb[32 + SB - 1]);
                 x[e] = k_at(j, d) * w;
             }
             uint4 w;
@@ -429,7 +440,7 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
     } else if (warp == 3) {   // scalars; values: column 16 vt + g (+ 8), tokens 2 t (+ 1) (+ 8)
         float* sc = reinterpret_cast<float*>(out + rec_scalars(KS) * 32);
         if (KIND == 0) {
-            for (int d = lane; d < KD; d += 32) sc[d] = expf(sB[(SB - 1) * QP + d]);
+            for (int d = lane; d < KD; d += 32) sc[d] = __expf(sB[(SB - 1) * QP + d]);
         } else if (lane < SB) {
             sc[lane] = gb[lane];
             sc[16 + lane] = gb[32 + lane];
@@ -446,8 +457,10 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
             }
             out[(rec_values(KS) + vt) * 32 + lane] = make_uint4(w[0], w[1], w[2], w[3]);
         }
-    } else {                  // scores A_ij, i the rows
-        float acc[2][4];
+    }
+    // scores A_ij, i the rows: the first and the last warp, each every other 16 channels
+    float acc[2][4];
+    if (warp == 0 || warp == 3) {
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
@@ -461,7 +474,7 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
         }
         if (!far) {
 #pragma unroll 1
-            for (int ks = 0; ks < KS; ++ks) {
+            for (int ks = warp == 0 ? 0 : 1; ks < KS; ks += 2) {
                 const int d = 16 * ks + 2 * t;
                 uint32_t ah[4], al[4];
                 float mid[4];
@@ -477,7 +490,7 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
                         al[q] = 0;
                     } else {
                         const float m0 = mid[(q >> 1) * 2], m1 = mid[(q >> 1) * 2 + 1];
-                        sb_split(q_at(i, c) * a.qscale * expf(sB[i * QP + c] - m0), q_at(i, c + 1) * a.qscale * expf(sB[i * QP + c + 1] - m1), ah[q], al[q]);
+                        sb_split(q_at(i, c) * a.qscale * __expf(sB[i * QP + c] - m0), q_at(i, c + 1) * a.qscale * __expf(sB[i * QP + c + 1] - m1), ah[q], al[q]);
                     }
                 }
 #pragma unroll
@@ -491,7 +504,7 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
                             bh[q] = *reinterpret_cast<const uint32_t*>(sK + j * QP + c);
                             bl[q] = 0;
                         } else {
-                            sb_split(k_at(j, c) * expf(mid[2 * q] - sB[j * QP + c]), k_at(j, c + 1) * expf(mid[2 * q + 1] - sB[j * QP + c + 1]), bh[q], bl[q]);
+                            sb_split(k_at(j, c) * __expf(mid[2 * q] - sB[j * QP + c]), k_at(j, c + 1) * __expf(mid[2 * q + 1] - sB[j * QP + c + 1]), bh[q], bl[q]);
                         }
                     }
                     sb_mma(acc[nt], ah[0], ah[1], ah[2], ah[3], bh[0], bh[1]);
@@ -501,7 +514,7 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
                     }
                 }
             }
-        } else {
+        } else if (warp == 0) {
 #pragma unroll 1
             for (int nt = 0; nt < 2; ++nt)
 #pragma unroll 1
@@ -509,10 +522,22 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
                     const int i = g + (e >> 1) * 8, j = 8 * nt + 2 * t + (e & 1);
                     float sum = 0.f;
                     if (j <= i)
-                        for (int d = 0; d < dk; ++d) sum = fmaf(q_at(i, d) * a.qscale * k_at(j, d), expf(sB[i * QP + d] - sB[j * QP + d]), sum);
+                        for (int d = 0; d < dk; ++d) sum = fmaf(q_at(i, d) * a.qscale * k_at(j, d), __expf(sB[i * QP + d] - sB[j * QP + d]), sum);
                     if (nt == 0) { if (e == 0) acc[0][0] = sum; else if (e == 1) acc[0][1] = sum; else if (e == 2) acc[0][2] = sum; else acc[0][3] = sum; }
                     else { if (e == 0) acc[1][0] = sum; else if (e == 1) acc[1][1] = sum; else if (e == 2) acc[1][2] = sum; else acc[1][3] = sum; }
                 }
+        }
+        if (warp == 3) {
+            half[lane] = make_float4(acc[0][0], acc[0][1], acc[0][2], acc[0][3]);
+            half[32 + lane] = make_float4(acc[1][0], acc[1][1], acc[1][2], acc[1][3]);
+        }
+    }
+    __syncthreads();
+    if (warp == 0) {
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+            const float4 h = half[32 * nt + lane];
+            acc[nt][0] += h.x; acc[nt][1] += h.y; acc[nt][2] += h.z; acc[nt][3] += h.w;
         }
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)
@@ -520,7 +545,7 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
             for (int e = 0; e < 4; ++e) {
                 const int i = g + (e >> 1) * 8, j = 8 * nt + 2 * t + (e & 1);
                 float x = j <= i ? acc[nt][e] : 0.f;
-                if (KIND == 1) x = j <= i ? x * a.qscale * expf(gb[16 + j] - gb[32 + i]) : 0.f;
+                if (KIND == 1) x = j <= i ? x * a.qscale * __expf(gb[16 + j] - gb[32 + i]) : 0.f;
                 acc[nt][e] = x;
             }
         // as the right operand of (values^T A^T): tokens j in pairs, column i = 8 nt + g
@@ -600,11 +625,13 @@ __global__ void state_blocks_kernel(StateArgs a, const uint4* rec, int min_len) 
         uint4 v;
         if (is_n) { v.x = v.z = g == 0 ? 0x3f803f80u : 0u; v.y = v.w = 0u; }
         else v = st[COMMON + 32 * warp + lane];
-        float oi[2][4], oa[2][4];
+        // an MMA's result takes tens of cycles and a warp is alone on its scheduler: the rounded values' products and the
+        // remainders' have accumulators of their own, so that no chain is longer than KS
+        float oi[3][2][4], oa[2][4];
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) oi[nt][e] = oa[nt][e] = 0.f;
+            for (int e = 0; e < 4; ++e) oi[0][nt][e] = oi[1][nt][e] = oi[2][nt][e] = oa[nt][e] = 0.f;
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
             const uint4 w = st[(rec_scores(KS) + nt) * 32 + lane];
@@ -621,9 +648,9 @@ __global__ void state_blocks_kernel(StateArgs a, const uint4* rec, int min_len) 
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt) {
                 const uint4 w = st[(ks * 2 + nt) * 32 + lane];
-                sb_mma(oi[nt], h[0], h[1], h[2], h[3], w.x, w.y);
-                sb_mma(oi[nt], l[0], l[1], l[2], l[3], w.x, w.y);
-                if (KIND == 0) sb_mma(oi[nt], h[0], h[1], h[2], h[3], w.z, w.w);
+                sb_mma(oi[0][nt], h[0], h[1], h[2], h[3], w.x, w.y);
+                sb_mma(oi[1][nt], l[0], l[1], l[2], l[3], w.x, w.y);
+                if (KIND == 0) sb_mma(oi[2][nt], h[0], h[1], h[2], h[3], w.z, w.w);
             }
         }
         // the block's outputs: row (value column) 16 tile + g (+ 8), tokens 8 nt + 2 t (+ 1)
@@ -640,7 +667,8 @@ __global__ void state_blocks_kernel(StateArgs a, const uint4* rec, int min_len) 
                     fa = expf(G - M);
                     mi = sc[i] + M;
                 }
-                const float lo = fmaf(fi, oi[nt][x], fa * oa[nt][x]), hi = fmaf(fi, oi[nt][2 + x], fa * oa[nt][2 + x]);
+                const float lo = fmaf(fi, oi[0][nt][x] + (oi[1][nt][x] + oi[2][nt][x]), fa * oa[nt][x]);
+                const float hi = fmaf(fi, oi[0][nt][2 + x] + (oi[1][nt][2 + x] + oi[2][nt][2 + x]), fa * oa[nt][2 + x]);
                 if (tok < t1) {
                     if (is_n) {
                         if (g == 0) a.den[(size_t)tok * H + head] = fmaxf(fabsf(lo), expf(-mi)) + 1e-6f;
@@ -685,39 +713,6 @@ __global__ void state_blocks_kernel(StateArgs a, const uint4* rec, int min_len) 
             if (p) *p = S[nt][e];
         }
     if (KIND == 1 && lane == 0) mg[is_n ? MB - 1 : tile] = m;
-}
-
-// ---------------------------------------------------------------------------
-// Log decays of gated linear attention: out[t, c] = logsigmoid(sum_r inner[t, r] w[r, c] + bias[c]) / tau, inner the R columns
-// of the token's projection row from `col` on, w fp32 [R, C].  A thread owns a channel for 8 tokens.
-// ---------------------------------------------------------------------------
-constexpr int CD_TOKENS = 8;
-
-template <typename T>
-__global__ void __launch_bounds__(128) channel_decay_kernel(const T* proj, long long row_stride, int col, int R, const float* w, const float* bias,
-                                                            float inv_tau, float* out, int n_tokens, int C) {
-    extern __shared__ float cd_smem[];      // [R][CD_TOKENS]
-    pdl_trigger();
-    pdl_wait();
-    const int t0 = blockIdx.y * CD_TOKENS, c = blockIdx.x * 128 + threadIdx.x, n = min(CD_TOKENS, n_tokens - t0);
-    for (int e = threadIdx.x; e < R * CD_TOKENS; e += 128) {
-        const int x = e / R, r = e - x * R;
-        cd_smem[r * CD_TOKENS + x] = x < n ? to_f32<T>(proj[(size_t)(t0 + x) * row_stride + col + r]) : 0.f;
-    }
-    __syncthreads();
-    if (c >= C) return;
-    float acc[CD_TOKENS];
-#pragma unroll
-    for (int x = 0; x < CD_TOKENS; ++x) acc[x] = 0.f;
-    for (int r = 0; r < R; ++r) {
-        const float wr = w[(size_t)r * C + c];
-#pragma unroll
-        for (int x = 0; x < CD_TOKENS; ++x) acc[x] = fmaf(cd_smem[r * CD_TOKENS + x], wr, acc[x]);
-    }
-    const float b = bias[c];
-#pragma unroll
-    for (int x = 0; x < CD_TOKENS; ++x)
-        if (x < n) out[(size_t)(t0 + x) * C + c] = log_sigmoid(acc[x] + b) * inv_tau;
 }
 
 // ---------------------------------------------------------------------------
@@ -771,11 +766,11 @@ __global__ void __launch_bounds__(128) heads_finish_kernel(const float* o, const
     }
 }
 
-StateArgs state_args(const void* proj, long long row_stride, int q_col, int k_col, int v_col, float qscale, const float* logd,
-                     const float* gates, int n_parts, long long part_stride, const float* gate_bias, float cap, float* state,
+StateArgs state_args(const void* proj, long long row_stride, int q_col, int k_col, int v_col, float qscale, const float* z,
+                     const float* z_bias, float tau, const float* gates, int n_parts, long long part_stride, const float* gate_bias, float cap, float* state,
                      long long slot_stride, const int* slots, const int* cu, float* o, float* den, int n_seqs, int H, int dk, int dv) {
     StateArgs a;
-    a.proj = proj; a.row_stride = row_stride; a.q_col = q_col; a.k_col = k_col; a.v_col = v_col; a.qscale = qscale; a.logd = logd;
+    a.proj = proj; a.row_stride = row_stride; a.q_col = q_col; a.k_col = k_col; a.v_col = v_col; a.qscale = qscale; a.z = z; a.z_bias = z_bias; a.inv_tau = 1.0f / tau;
     a.gates = gates; a.n_parts = n_parts; a.part_stride = part_stride; a.gate_bias = gate_bias; a.cap = cap; a.state = state;
     a.slot_stride = slot_stride; a.slots = slots; a.cu = cu; a.o = o; a.den = den; a.n_seqs = n_seqs; a.H = H; a.dk = dk; a.dv = dv;
     return a;
@@ -783,7 +778,7 @@ StateArgs state_args(const void* proj, long long row_stride, int q_col, int k_co
 
 int check_state(const StateArgs& a, int kind) {
     if (a.H <= 0 || a.dk <= 0 || a.dv <= 0 || !a.proj || !a.state || !a.slots || !a.cu || !a.o || a.q_col < 0 || a.k_col < 0 || a.v_col < 0) return PYRE_ERR_BAD_ARG;
-    if (kind == 0 && !a.logd) return PYRE_ERR_BAD_ARG;
+    if (kind == 0 && (!a.z || !a.z_bias || !(a.inv_tau > 0.f))) return PYRE_ERR_BAD_ARG;
     if (kind == 1 && (!a.gates || a.n_parts < 1 || !a.gate_bias || !(a.cap > 0.f) || !a.den)) return PYRE_ERR_BAD_ARG;
     if (kind != 0 && kind != 1) return PYRE_ERR_BAD_ARG;
     const long long need = (long long)a.H * a.dk * a.dv + (kind == 1 ? (long long)a.H * (a.dk + (a.dv + 15) / 16 + 1) : 0);
@@ -793,10 +788,12 @@ int check_state(const StateArgs& a, int kind) {
 }
 
 template <typename T, int G>
-void launch_scan(const StateArgs& a, int kind, int max_len, cudaStream_t stream) {
-    const dim3 grid(ceil_div(a.dv, ScanShape<G>::CT), a.H, a.n_seqs);
-    if (kind == 0) pyre_launch(state_scan_kernel<T, G, 0>, grid, dim3(ScanShape<G>::THREADS), 0, stream, a, max_len);
-    else pyre_launch(state_scan_kernel<T, G, 1>, grid, dim3(ScanShape<G>::THREADS), 0, stream, a, max_len);
+void launch_scan(const StateArgs& a, int kind, int max_len, bool few, cudaStream_t stream) {
+    const dim3 grid(ceil_div(a.dv, ScanShape<G, false>::CT), a.H, a.n_seqs), block(ScanShape<G, false>::THREADS);
+    if (kind == 0 && few) pyre_launch(state_scan_kernel<T, G, 0, true>, grid, block, 0, stream, a, max_len);
+    else if (kind == 0) pyre_launch(state_scan_kernel<T, G, 0, false>, grid, block, 0, stream, a, max_len);
+    else if (few) pyre_launch(state_scan_kernel<T, G, 1, true>, grid, block, 0, stream, a, max_len);
+    else pyre_launch(state_scan_kernel<T, G, 1, false>, grid, block, 0, stream, a, max_len);
 }
 
 template <int KS, int KIND>
@@ -829,20 +826,21 @@ int launch_chunked(const StateArgs& a, uint4* rec, int min_len, int n_blocks, in
 }  // namespace
 
 // The entries of at most max_len tokens (0: all of them), token by token.
-PYRE_API int pyre_state_scan(const void* proj, long long row_stride, int q_col, int k_col, int v_col, float qscale, const float* logd,
-                             const float* gates, int n_parts, long long part_stride, const float* gate_bias, float cap, float* state,
+PYRE_API int pyre_state_scan(const void* proj, long long row_stride, int q_col, int k_col, int v_col, float qscale, const float* z,
+                             const float* z_bias, float tau, const float* gates, int n_parts, long long part_stride, const float* gate_bias, float cap, float* state,
                              long long slot_stride, const int* slots, const int* cu_seqlens, float* o, float* den, int n_tokens,
                              int n_seqs, int H, int dk, int dv, int max_len, int kind, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
-    const StateArgs a = state_args(proj, row_stride, q_col, k_col, v_col, qscale, logd, gates, n_parts, part_stride, gate_bias, cap,
+    const StateArgs a = state_args(proj, row_stride, q_col, k_col, v_col, qscale, z, z_bias, tau, gates, n_parts, part_stride, gate_bias, cap,
                                    state, slot_stride, slots, cu_seqlens, o, den, n_seqs, H, dk, dv);
     const int rc = check_state(a, kind);
     if (rc) return rc;
     if (dk > 256) return PYRE_ERR_UNSUPPORTED;
-#define PICK(TT) do { if (dk <= 16) launch_scan<TT, 1>(a, kind, max_len, stream); else if (dk <= 32) launch_scan<TT, 2>(a, kind, max_len, stream); \
-                      else if (dk <= 48) launch_scan<TT, 3>(a, kind, max_len, stream); else if (dk <= 64) launch_scan<TT, 4>(a, kind, max_len, stream); \
-                      else if (dk <= 96) launch_scan<TT, 6>(a, kind, max_len, stream); else if (dk <= 128) launch_scan<TT, 8>(a, kind, max_len, stream); \
-                      else launch_scan<TT, 16>(a, kind, max_len, stream); } while (0)
+    const bool few = n_tokens <= 2 * n_seqs;      // (nearly) all entries bring one token
+#define PICK(TT) do { if (dk <= 16) launch_scan<TT, 1>(a, kind, max_len, few, stream); else if (dk <= 32) launch_scan<TT, 2>(a, kind, max_len, few, stream); \
+                      else if (dk <= 48) launch_scan<TT, 3>(a, kind, max_len, few, stream); else if (dk <= 64) launch_scan<TT, 4>(a, kind, max_len, few, stream); \
+                      else if (dk <= 96) launch_scan<TT, 6>(a, kind, max_len, few, stream); else if (dk <= 128) launch_scan<TT, 8>(a, kind, max_len, few, stream); \
+                      else launch_scan<TT, 16>(a, kind, max_len, few, stream); } while (0)
     if (dtype == PYRE_BF16) PICK(__nv_bfloat16);
     else if (dtype == PYRE_F32) PICK(float);
     else return PYRE_ERR_BAD_ARG;
@@ -862,13 +860,13 @@ PYRE_API int pyre_state_record_floats(int dk, int dv, int kind) {
 // The entries of at least min_len tokens, in blocks of 16 on the tensor cores (bfloat16 activations).  n_blocks: the sum of
 // ceil(tokens / 16) over those entries; scratch: n_blocks * H * pyre_state_record_floats floats, 16-byte aligned; warps: 16-column
 // tiles of a head's state per CTA.
-PYRE_API int pyre_state_chunked(const void* proj, long long row_stride, int q_col, int k_col, int v_col, float qscale, const float* logd,
-                                const float* gates, int n_parts, long long part_stride, const float* gate_bias, float cap, float* state,
+PYRE_API int pyre_state_chunked(const void* proj, long long row_stride, int q_col, int k_col, int v_col, float qscale, const float* z,
+                                const float* z_bias, float tau, const float* gates, int n_parts, long long part_stride, const float* gate_bias, float cap, float* state,
                                 long long slot_stride, const int* slots, const int* cu_seqlens, float* o, float* den, void* scratch,
                                 int n_tokens, int n_seqs, int H, int dk, int dv, int min_len, int n_blocks, int kind, int warps,
                                 cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0 || n_blocks <= 0) return 0;
-    const StateArgs a = state_args(proj, row_stride, q_col, k_col, v_col, qscale, logd, gates, n_parts, part_stride, gate_bias, cap,
+    const StateArgs a = state_args(proj, row_stride, q_col, k_col, v_col, qscale, z, z_bias, tau, gates, n_parts, part_stride, gate_bias, cap,
                                    state, slot_stride, slots, cu_seqlens, o, den, n_seqs, H, dk, dv);
     const int rc = check_state(a, kind);
     if (rc) return rc;
@@ -885,22 +883,6 @@ PYRE_API int pyre_state_chunked(const void* proj, long long row_stride, int q_co
     if (dk <= 96) return GO(6);
     return GO(8);
 #undef GO
-}
-
-PYRE_API int pyre_channel_decay(const void* proj, long long row_stride, int col, int R, const float* w, const float* bias, float tau,
-                                float* out, int n_tokens, int C, int dtype, cudaStream_t stream) {
-    if (n_tokens <= 0 || C <= 0) return 0;
-    if (R <= 0 || col < 0 || !(tau > 0.f) || !w || !bias || !out) return PYRE_ERR_BAD_ARG;
-    const size_t smem = (size_t)R * CD_TOKENS * sizeof(float);
-    if (smem > 48 * 1024 || ceil_div(n_tokens, CD_TOKENS) > 65535) return PYRE_ERR_UNSUPPORTED;
-    const dim3 grid(ceil_div(C, 128), ceil_div(n_tokens, CD_TOKENS));
-    if (dtype == PYRE_BF16)
-        pyre_launch(channel_decay_kernel<__nv_bfloat16>, grid, dim3(128), smem, stream, (const __nv_bfloat16*)proj, row_stride, col, R, w, bias, 1.0f / tau, out, n_tokens, C);
-    else if (dtype == PYRE_F32)
-        pyre_launch(channel_decay_kernel<float>, grid, dim3(128), smem, stream, (const float*)proj, row_stride, col, R, w, bias, 1.0f / tau, out, n_tokens, C);
-    else return PYRE_ERR_BAD_ARG;
-    PYRE_LAUNCH_CHECK();
-    return 0;
 }
 
 PYRE_API int pyre_heads_finish(const float* o, const float* den, const float* w, int w_period, const void* proj, long long row_stride,

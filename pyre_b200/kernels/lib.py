@@ -53,12 +53,12 @@ SIGNATURES: dict[str, tuple[str, list]] = {
     "pyre_bias_act": ("blockops", [P, P, P, LL, I, I, I, P]),
     "pyre_add_row_vector": ("blockops", [P, P, LL, I, P]),
     "pyre_gated_norm": ("blockops", [P, P, I, LL, P, P, P, P, P, P, I, I, F, I, I, P]),
+    "pyre_normed_add_norm": ("blockops", [P, P, P, I, LL, P, P, F, P, F, P, P, I, I, I, I, P]),
     "pyre_token_shift_mix": ("wkv", [P, P, LL, LL, P, P, P, P, P, I, I, I, I, P]),
     "pyre_wkv_scan": ("wkv", [P, P, P, P, P, P, P, P, P, LL, LL, P, P, P, P, P, I, I, I, I, I, F, I, P]),
-    "pyre_channel_decay": ("matrix_state", [P, LL, I, I, P, P, F, P, I, I, I, P]),
-    "pyre_state_scan": ("matrix_state", [P, LL, I, I, I, F, P, P, I, LL, P, F, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, P]),
+    "pyre_state_scan": ("matrix_state", [P, LL, I, I, I, F, P, P, F, P, I, LL, P, F, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, P]),
     "pyre_state_record_floats": ("matrix_state", [I, I, I]),
-    "pyre_state_chunked": ("matrix_state", [P, LL, I, I, I, F, P, P, I, LL, P, F, P, LL, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P]),
+    "pyre_state_chunked": ("matrix_state", [P, LL, I, I, I, F, P, P, F, P, I, LL, P, F, P, LL, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P]),
     "pyre_heads_finish": ("matrix_state", [P, P, P, I, P, LL, I, I, F, P, LL, I, I, I, F, I, P]),
     "pyre_linear_attention_scan": ("linear_attention", [P, LL, I, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, P]),
     "pyre_linear_attention_chunked": ("linear_attention", [P, LL, I, I, I, P, P, P, P, P, I, I, I, I, I, I, I, P]),
@@ -109,8 +109,8 @@ DEFAULT_CLASS = {
     "pyre_add_layernorm": "norm", "pyre_scaled_sum": "norm", "pyre_stream_rows": "norm", "pyre_stream_set": "norm", "pyre_act_mul": "activation", "pyre_latent_prepare": "rotary+write",
     "pyre_latent_rotate_q": "rotary+write", "pyre_latent_attention_exact": "latent_attention", "pyre_latent_attention_mma": "latent_attention", "pyre_grouped_linear": "grouped_product",
     "pyre_route": "router", "pyre_group_pairs": "router", "pyre_combine_pairs": "router", "pyre_scale_to_places": "router",
-    "pyre_head_gate": "gate", "pyre_bias_act": "activation", "pyre_add_row_vector": "norm", "pyre_gated_norm": "norm",
-    "pyre_channel_decay": "decay", "pyre_state_scan": "recurrence", "pyre_state_chunked": "recurrence", "pyre_heads_finish": "gate",
+    "pyre_head_gate": "gate", "pyre_bias_act": "activation", "pyre_add_row_vector": "norm", "pyre_gated_norm": "norm", "pyre_normed_add_norm": "norm",
+    "pyre_state_scan": "recurrence", "pyre_state_chunked": "recurrence", "pyre_heads_finish": "gate",
     "pyre_token_shift_mix": "recurrence", "pyre_wkv_scan": "recurrence",
     "pyre_scale_cap": "scale", "pyre_short_conv": "short_conv", "pyre_ssm_scan": "recurrence", "pyre_group_norm_gate": "gate",
     "pyre_diff_combine": "gate", "pyre_rotate_heads": "rotary+write", "pyre_side_gate": "activation", "pyre_token_gate_add": "router",

@@ -104,9 +104,34 @@ class BiasedRows:
         return self.y.shape
 
 
-def materialize(t: "torch.Tensor | PartialSums | DeferredProduct | ScaledRows | ScaledSum | BiasedRows") -> torch.Tensor:
+class NormedBranch:
+    """An RMS norm of a branch output that is not formed yet: rmsnorm(y) * weight with ``y`` a tensor or any lazy form and
+    ``weight`` fp32 [N].  ``add_rmsnorm`` forms it, adds it to the stream and norms the sum in one pass over the row; any other
+    consumer of a pending branch output calls ``formed``."""
+
+    def __init__(self, y, weight: torch.Tensor, eps: float, dtype: torch.dtype):
+        self.y, self.weight, self.eps, self.dtype = y, weight, float(eps), dtype
+
+    @property
+    def shape(self):
+        return self.y.shape
+
+    def formed(self):
+        """The branch output in fp32: a tensor (float32), or one unrounded part (bfloat16)."""
+        out = gated_norm(self.y, None, None, None, self.weight, self.eps, self.dtype, center=False)
+        return out if self.dtype == torch.float32 else PartialSums(out.unsqueeze(0), self.dtype)
+
+
+def formed(t):
+    """A pending branch output without the forms that only some consumers know."""
+    return t.formed() if isinstance(t, NormedBranch) else materialize(t) if isinstance(t, BiasedRows) else t
+
+
+def materialize(t: "torch.Tensor | PartialSums | DeferredProduct | ScaledRows | ScaledSum | BiasedRows | NormedBranch") -> torch.Tensor:
     """A plain tensor in the activation dtype from a tensor or any of the lazy forms a branch output or a
     norm's output may take."""
+    if isinstance(t, NormedBranch):
+        t = t.formed()
     if isinstance(t, BiasedRows):
         return bias_act(materialize(t.y), t.bias, None)
     if isinstance(t, ScaledSum):
@@ -194,6 +219,39 @@ def embedding(table: torch.Tensor, ids: torch.Tensor, out: "torch.Tensor | None"
     return out
 
 
+NORMED_ADD_MAX_WIDTH = 4096      # rows of any width up to here, and of multiples of 4 up to four times as many
+
+
+def _normed_add_norm(x: torch.Tensor, branch: NormedBranch, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
+                     rows: "torch.Tensor | None", update_x: bool) -> torch.Tensor:
+    """``add_rmsnorm`` of a ``NormedBranch``: x += rmsnorm(y + bias) * its weight and out = rmsnorm(x) * weight in one kernel."""
+    _check(x, "x", torch.float32, 2)
+    T, H = x.shape
+    y, bias = (branch.y.y, branch.y.bias) if isinstance(branch.y, BiasedRows) else (branch.y, None)
+    if isinstance(y, DeferredProduct):
+        y = y.partials()
+    parts, n_parts = None, 0
+    if isinstance(y, PartialSums):
+        parts, n_parts, y = y.parts, y.n, None
+    else:
+        _check(y, "y", out_dtype, 2)
+    if tuple((parts[0] if y is None else y).shape) != (T, H):
+        raise ValueError(f"branch output {tuple((parts[0] if y is None else y).shape)} != stream {(T, H)}")
+    for w, name in ((weight, "weight"), (branch.weight, "branch weight"), (bias, "bias")):
+        if w is not None:
+            _check(w, name, torch.float32, 1)
+            if w.shape[0] != H:
+                raise ValueError(f"{name} has {w.shape[0]} entries, rows have {H}")
+    if rows is not None:
+        _check(rows, "rows", torch.int32, 1)
+        update_x = False
+    n_rows = T if rows is None else rows.shape[0]
+    out = torch.empty((n_rows, H), dtype=out_dtype, device=x.device)
+    lib.call("pyre_normed_add_norm", x.data_ptr(), _ptr(y), _ptr(parts), n_parts, T * H, _ptr(bias), branch.weight.data_ptr(), branch.eps,
+             weight.data_ptr(), float(eps), out.data_ptr(), _ptr(rows), n_rows, H, int(bool(update_x)), _dt(out_dtype), _stream())
+    return out
+
+
 def add_rmsnorm(x: torch.Tensor, delta: "torch.Tensor | None", weight: torch.Tensor, eps: float,
                 out_dtype: torch.dtype, rows: "torch.Tensor | None" = None, update_x: bool = True,
                 out: "torch.Tensor | None" = None, scaled_ok: bool = False) -> "torch.Tensor | ScaledRows":
@@ -201,12 +259,13 @@ def add_rmsnorm(x: torch.Tensor, delta: "torch.Tensor | None", weight: torch.Ten
 
     ``x`` is the fp32 residual stream [T, H]; with ``update_x`` (and no ``rows``) the sum is
     written back to it.  ``delta`` has the activation dtype, or is a ``PartialSums`` whose
-    parts the kernel adds, or a ``DeferredProduct``.  ``weight`` is fp32 [H].
+    parts the kernel adds, or a ``DeferredProduct``, or a ``NormedBranch``.  ``weight`` is fp32 [H].
 
     ``scaled_ok``: the caller's consumer takes ``ScaledRows``.  Then a deferred product is launched with the
     residual add and the norm's preparation as its fix-up, and no norm kernel runs at all."""
-    if isinstance(delta, BiasedRows):
-        delta = materialize(delta)
+    if isinstance(delta, NormedBranch) and out is None and x.shape[1] <= NORMED_ADD_MAX_WIDTH * (4 if x.shape[1] % 4 == 0 else 1):
+        return _normed_add_norm(x, delta, weight, eps, out_dtype, rows, update_x)
+    delta = formed(delta)
     _check(x, "x", torch.float32, 2)
     _check(weight, "weight", torch.float32, 1)
     T, H = x.shape
@@ -1115,8 +1174,7 @@ def norm_add(x: torch.Tensor, y: "torch.Tensor | PartialSums | DeferredProduct",
     """x[t] += rmsnorm(y[t]) * weight in place on the fp32 stream ``x`` [T, H]: the norm sits on a branch's OUTPUT
     ``y`` (activation dtype, or fp32 partial sums that the kernel adds).  ``want_next``: also return the new stream
     as activations (what the next branch reads), written in the same pass."""
-    if isinstance(y, BiasedRows):
-        y = materialize(y)
+    y = formed(y)
     _check(x, "x", torch.float32, 2)
     _check(weight, "weight", torch.float32, 1)
     T, H = x.shape
@@ -1534,8 +1592,7 @@ def add_layernorm(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSum
     plain branch output or partial sums (gain one), or None.  ``out_dtype`` float32 with bfloat16 activations
     (``act_dtype``) gives the normalised rows in fp32: a norm applied to the stream itself.  ``weight2``: a second norm
     of the SAME rows (no bias) written in the same pass; the result is then the pair."""
-    if isinstance(delta, BiasedRows):
-        delta = materialize(delta)
+    delta = formed(delta)
     _check(x, "x", torch.float32, 2)
     _check(weight, "weight", torch.float32, 1)
     T, H = x.shape
@@ -1575,8 +1632,7 @@ def add_layernorm(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSum
 def stream_rows(x: torch.Tensor, delta: "ScaledSum | torch.Tensor | PartialSums | None", dtype: torch.dtype) -> torch.Tensor:
     """The fp32 stream ``x`` [T, H] with ``delta`` (as in ``add_layernorm``) added, as activations for a product that
     reads the stream itself: a new tensor in ``dtype``; ``x`` stays as it is."""
-    if isinstance(delta, BiasedRows):
-        delta = materialize(delta)
+    delta = formed(delta)
     _check(x, "x", torch.float32, 2)
     T, H = x.shape
     if delta is not None and not isinstance(delta, ScaledSum):
@@ -2146,7 +2202,7 @@ def group_norm_gate(y: torch.Tensor, groups: int, weight: "torch.Tensor | None",
 # ---------------------------------------------------------------------------------- matrix states with decays that depend on the token
 STATE_MAX_DIM = 256            # query/key entries per head
 STATE_CHUNK_MIN_LEN = 32       # bfloat16 entries with at least this many tokens run in blocks on the tensor cores
-STATE_CHUNK_WARPS = 2          # tiles of 16 value columns per CTA of that kernel
+STATE_CHUNK_WARPS = {0: 2, 1: 4}      # tiles of 16 value columns per CTA of that kernel: gated linear attention, matrix memory
 USE_STATE_CHUNKS = True
 
 
@@ -2156,22 +2212,7 @@ def memory_state_floats(n_heads: int, qk_dim: int, v_dim: int) -> int:
     return n_heads * (qk_dim * v_dim + qk_dim + -(-v_dim // 16) + 1)
 
 
-def channel_decay(proj: torch.Tensor, col: int, rank: int, weight: torch.Tensor, bias: torch.Tensor, tau: float) -> torch.Tensor:
-    """Log decays of gated linear attention, fp32 [T, C]: logsigmoid(inner w + bias) / tau with ``inner`` the ``rank``
-    columns of ``proj`` from ``col`` on and ``weight`` fp32 [rank, C] (the map's transpose)."""
-    _check(proj, "proj", dim=2)
-    _check(weight, "weight", torch.float32, 2)
-    _check(bias, "bias", torch.float32, 1)
-    T, C = proj.shape[0], weight.shape[1]
-    if weight.shape[0] != rank or bias.shape[0] != C or col < 0 or col + rank > proj.shape[1]:
-        raise ValueError("the decay's map does not match the projection row")
-    out = torch.empty((T, C), dtype=torch.float32, device=proj.device)
-    lib.call("pyre_channel_decay", proj.data_ptr(), proj.shape[1], int(col), int(rank), weight.data_ptr(), bias.data_ptr(), float(tau),
-             out.data_ptr(), T, C, _dt(proj.dtype), _stream())
-    return out
-
-
-def _matrix_state(kind: int, proj, q_col, k_col, v_col, q_scale, logd, gates, gate_bias, cap, state_layer, slots, cu_seqlens, n_heads,
+def _matrix_state(kind: int, proj, q_col, k_col, v_col, q_scale, z, z_bias, tau, gates, gate_bias, cap, state_layer, slots, cu_seqlens, n_heads,
                   qk_dim, v_dim, lens, chunked):
     _check(proj, "proj", dim=2)
     _check(state_layer, "state_layer", torch.float32)
@@ -2195,34 +2236,35 @@ def _matrix_state(kind: int, proj, q_col, k_col, v_col, q_scale, logd, gates, ga
     blocks = sum(-(-int(n) // 16) for n in lens if n >= STATE_CHUNK_MIN_LEN) if record else 0
     if blocks:
         scratch = torch.empty(blocks * n_heads * record, dtype=torch.float32, device=proj.device)
-        lib.call("pyre_state_chunked", proj.data_ptr(), W, int(q_col), int(k_col), int(v_col), float(q_scale), _ptr(logd), _ptr(parts), n_parts,
-                 T * 2 * n_heads, _ptr(gate_bias), float(cap), state_layer.data_ptr(), slot_floats, slots.data_ptr(), cu_seqlens.data_ptr(),
+        lib.call("pyre_state_chunked", proj.data_ptr(), W, int(q_col), int(k_col), int(v_col), float(q_scale), _ptr(z), _ptr(z_bias), float(tau),
+                 _ptr(parts), n_parts, T * 2 * n_heads, _ptr(gate_bias), float(cap), state_layer.data_ptr(), slot_floats, slots.data_ptr(), cu_seqlens.data_ptr(),
                  o.data_ptr(), _ptr(den), scratch.data_ptr(), T, n_seqs, n_heads, qk_dim, v_dim, STATE_CHUNK_MIN_LEN, blocks, kind,
-                 STATE_CHUNK_WARPS, _stream())
+                 STATE_CHUNK_WARPS[kind], _stream())
     if not blocks or any(n < STATE_CHUNK_MIN_LEN for n in lens):
-        lib.call("pyre_state_scan", proj.data_ptr(), W, int(q_col), int(k_col), int(v_col), float(q_scale), _ptr(logd), _ptr(parts), n_parts,
-                 T * 2 * n_heads, _ptr(gate_bias), float(cap), state_layer.data_ptr(), slot_floats, slots.data_ptr(), cu_seqlens.data_ptr(),
+        lib.call("pyre_state_scan", proj.data_ptr(), W, int(q_col), int(k_col), int(v_col), float(q_scale), _ptr(z), _ptr(z_bias), float(tau),
+                 _ptr(parts), n_parts, T * 2 * n_heads, _ptr(gate_bias), float(cap), state_layer.data_ptr(), slot_floats, slots.data_ptr(), cu_seqlens.data_ptr(),
                  o.data_ptr(), _ptr(den), T, n_seqs, n_heads, qk_dim, v_dim, STATE_CHUNK_MIN_LEN - 1 if blocks else 0, kind,
                  _dt(proj.dtype), _stream())
     return o, den
 
 
-def gated_linear_attention(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_scale: float, logd: torch.Tensor,
-                           state_layer: torch.Tensor, slots: torch.Tensor, cu_seqlens: torch.Tensor, n_heads: int, qk_dim: int,
+def gated_linear_attention(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_scale: float, z: torch.Tensor,
+                           z_bias: torch.Tensor, tau: float, state_layer: torch.Tensor, slots: torch.Tensor, cu_seqlens: torch.Tensor, n_heads: int, qk_dim: int,
                            v_dim: int, lens=None, chunked: "bool | None" = None) -> torch.Tensor:
     """Linear attention with a decay per key channel over the step's entries, continuing each request's state: per head
-    S_t = diag(exp(logd_t)) S_(t-1) + k_t v_t^T, o_t = S_t^T (q_scale q_t), with q, k, v columns of ``proj`` and ``logd``
-    fp32 [T, heads * qk_dim].  ``state_layer`` [slots, ...] fp32 holds S [heads, qk_dim, v_dim] at slot ``slots[b]`` of
+    S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T (q_scale q_t), with q, k, v columns of ``proj`` and the decays
+    a = sigmoid(z + z_bias)^(1 / tau), ``z`` fp32 [T, heads * qk_dim].  ``state_layer`` [slots, ...] fp32 holds S [heads, qk_dim, v_dim] at slot ``slots[b]`` of
     entry b and is left updated.  ``lens``: the entries' token counts on the host; with them bfloat16 entries of
     ``STATE_CHUNK_MIN_LEN`` tokens or more run in blocks of 16 tokens on the tensor cores (query/key sizes up to 128,
     ``chunked=False``: not); everything else walks token by token, bit-identical under any cutting.
     Returns fp32 [T, heads * v_dim]."""
-    _check(logd, "logd", torch.float32, 2)
-    if tuple(logd.shape) != (proj.shape[0], n_heads * qk_dim):
-        raise ValueError("one log decay per token, head and key channel")
+    _check(z, "z", torch.float32, 2)
+    _check(z_bias, "z_bias", torch.float32, 1)
+    if tuple(z.shape) != (proj.shape[0], n_heads * qk_dim) or z_bias.shape[0] != n_heads * qk_dim or not tau > 0:
+        raise ValueError("one decay per token, head and key channel, one bias per head and channel, a positive tau")
     if state_layer[0].numel() < n_heads * qk_dim * v_dim:
         raise ValueError("the state does not lie inside the slot")
-    return _matrix_state(0, proj, q_col, k_col, v_col, q_scale, logd, None, None, 0.0, state_layer, slots, cu_seqlens, n_heads, qk_dim,
+    return _matrix_state(0, proj, q_col, k_col, v_col, q_scale, z, z_bias, tau, None, None, 0.0, state_layer, slots, cu_seqlens, n_heads, qk_dim,
                          v_dim, lens, chunked)[0]
 
 
@@ -2245,7 +2287,7 @@ def matrix_memory(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, q_scal
         raise ValueError("one bias per gate, and a positive cap")
     if state_layer[0].numel() < memory_state_floats(n_heads, qk_dim, v_dim):
         raise ValueError("the state does not lie inside the slot")
-    return _matrix_state(1, proj, q_col, k_col, v_col, q_scale, None, gates, gate_bias, cap, state_layer, slots, cu_seqlens, n_heads,
+    return _matrix_state(1, proj, q_col, k_col, v_col, q_scale, None, None, 1.0, gates, gate_bias, cap, state_layer, slots, cu_seqlens, n_heads,
                          qk_dim, v_dim, lens, chunked)
 
 

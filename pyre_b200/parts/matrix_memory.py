@@ -72,9 +72,10 @@ class MatrixMemory(StackedMixer):
         st = ctx.state_group(call.state_group)
         with lib.section("gates"):
             gates = ops.linear(h, self.w_gates, out_dtype=torch.float32, partials_ok=True)
-        o, den = ops.matrix_memory(proj, col, col + self.k_col, col + self.v_col, self.head_dim ** -0.5, gates, self.b_gates, self.gate_cap,
-                                   st.buffer[call.state_layer], st.slots, ctx.cu_seqlens, self.n_heads, self.head_dim, self.v_head_dim,
-                                   lens=ctx.entry_lengths)
+        with lib.section("matrix_memory"):
+            o, den = ops.matrix_memory(proj, col, col + self.k_col, col + self.v_col, self.head_dim ** -0.5, gates, self.b_gates,
+                                       self.gate_cap, st.buffer[call.state_layer], st.slots, ctx.cu_seqlens, self.n_heads, self.head_dim,
+                                       self.v_head_dim, lens=ctx.entry_lengths)
         return ops.heads_finish(o, den, self.norm_w, self.eps, proj, col + self.g_col, self.n_heads, self.v_head_dim, self.dtype,
                                 gate="sigmoid", post=scale, out=out, out_col=out_col)
 

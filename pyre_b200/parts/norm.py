@@ -47,7 +47,10 @@ class RMSNorm(Part):
 
     def gated_output(self, ctx, y, gate=None, gate_bias=None):
         """norm(y * sigmoid(gate + gate_bias)) * gain for a sublayer's result ``y`` that is not added to the stream
-        here: it comes back as an fp32 branch output (one unrounded part in bfloat16) for the next norm to add."""
+        here: it comes back as an fp32 branch output (one unrounded part in bfloat16) for the next norm to add; without a
+        gate as an ``ops.NormedBranch``, which the next norm's kernel forms on the way."""
+        if gate is None:
+            return ops.NormedBranch(y, self.weight, self.eps, self.dtype)
         out = ops.gated_norm(y, None, gate, gate_bias, self.weight, self.eps, self.dtype, center=False)
         return out if self.dtype == torch.float32 else ops.PartialSums(out.unsqueeze(0), self.dtype)
 

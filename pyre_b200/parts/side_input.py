@@ -50,6 +50,7 @@ class TokenSideInput(Part):
 
     def forward(self, ctx, x, pending):
         if pending is not None:
+            pending = ops.formed(pending)
             if isinstance(pending, ops.PartialSums):
                 for i in range(pending.n):
                     ops.add_residual(x, pending.parts[i])          # fp32 parts enter the stream unrounded

@@ -16,7 +16,7 @@ def embedding(table, ids, out=None, err_flag=None):
 
 
 def add_rmsnorm(x, delta, weight, eps, out_dtype, rows=None, update_x=True, out=None, scaled_ok=False):
-    v = x if delta is None else x + delta.float()
+    v = x if delta is None else x + _partial_sums_or_tensor(delta)
     if rows is None and update_x and delta is not None:
         x.copy_(v)
     if rows is not None:
@@ -483,17 +483,13 @@ def ssm_scan(xbc, proj, dt_col, dt_bias, a_log, d_skip, state_layer, slots, cu_s
     return y.reshape(T, H * P)
 
 
-def channel_decay(proj, col, rank, weight, bias, tau):
-    return torch.nn.functional.logsigmoid(proj[:, col:col + rank].float() @ weight + bias) / tau
-
-
-def gated_linear_attention(proj, q_col, k_col, v_col, q_scale, logd, state_layer, slots, cu_seqlens, n_heads, qk_dim, v_dim, lens=None,
-                           chunked=None):
+def gated_linear_attention(proj, q_col, k_col, v_col, q_scale, z, z_bias, tau, state_layer, slots, cu_seqlens, n_heads, qk_dim, v_dim,
+                           lens=None, chunked=None):
     T, x = proj.shape[0], proj.float()
     q = x[:, q_col:q_col + n_heads * qk_dim].reshape(T, n_heads, qk_dim) * q_scale
     k = x[:, k_col:k_col + n_heads * qk_dim].reshape(T, n_heads, qk_dim)
     v = x[:, v_col:v_col + n_heads * v_dim].reshape(T, n_heads, v_dim)
-    keep = logd.exp().reshape(T, n_heads, qk_dim, 1)
+    keep = torch.exp(torch.nn.functional.logsigmoid(z + z_bias) / tau).reshape(T, n_heads, qk_dim, 1)
     out = torch.empty((T, n_heads, v_dim))
     cu = cu_seqlens.tolist()
     assert lens is None or [b - a for a, b in zip(cu, cu[1:])] == list(lens)
@@ -646,7 +642,7 @@ def install(monkeypatch) -> None:
                          token_shift_mix=token_shift_mix, wkv_scan=wkv_scan, scale_cap=scale_cap, short_conv=short_conv,
                          ssm_scan=ssm_scan, group_norm_gate=group_norm_gate, diff_combine=diff_combine, rotate_heads=rotate_heads,
                          side_gate=side_gate, token_gate_add=token_gate_add, stream_rows=stream_rows, stream_set=stream_set,
-                         channel_decay=channel_decay, gated_linear_attention=gated_linear_attention, matrix_memory=matrix_memory,
+                         gated_linear_attention=gated_linear_attention, matrix_memory=matrix_memory,
                          heads_finish=heads_finish).items():
         monkeypatch.setattr(ops, name, fn)
     monkeypatch.setattr(ops, "device_error_flag", lambda device: flag)
@@ -663,6 +659,8 @@ def install(monkeypatch) -> None:
 
 def _partial_sums_or_tensor(t):
     from pyre_b200.kernels import ops
+    if isinstance(t, ops.NormedBranch):
+        t = t.formed()
     if isinstance(t, ops.DeferredProduct):      # a product not launched yet: the stand-ins never fold, they run it plainly
         t = t.partials()
     return t.parts.sum(0) if isinstance(t, ops.PartialSums) else t.float()
