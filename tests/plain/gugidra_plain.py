@@ -197,9 +197,10 @@ def routed_mlp(h, w, prefix, mlp, lowp=False, margins=None):
     weight = s.gather(-1, idx)
     weight = weight / (weight.sum(-1, keepdim=True) + 1e-20)
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for e, wt in zip(idx[t].tolist(), weight[t]):
-            out[t] += wt * clamped_mlp(h[t:t + 1], w, f"{prefix}e{e}.", mlp["expert"]["limit"], lowp)[0]
+    for e in range(router["experts"]):
+        tokens, place = torch.where(idx == e)
+        if len(tokens):
+            out[tokens] += weight[tokens, place, None] * clamped_mlp(h[tokens], w, f"{prefix}e{e}.", mlp["expert"]["limit"], lowp)
     if mlp.get("shared"):
         out = out + clamped_mlp(h, w, prefix + "shared.", mlp["shared"]["limit"], lowp)
     return out
