@@ -272,7 +272,9 @@ __global__ void __launch_bounds__(ScanShape<G, FEW>::THREADS) state_scan_kernel(
 // take them (one 16-byte vector per lane, "fragment"); operands that are not bf16 numbers enter as a rounded value and a
 // rounded remainder (16 bits of mantissa).  state_blocks_kernel walks an entry's blocks: a warp holds S^T for 16 value
 // columns as accumulators, which are in the layout of the next product's left operand, so the state never leaves its
-// registers.  For kind 1 one more warp carries n as the row of a value column of ones.
+// registers.  Several warps share a tile, each with some of the channels; they hand their shares of a block's outputs over
+// through shared memory, and the first one writes the sum while the next block runs.  For kind 1 one more tile carries n
+// as the row of a value column of ones.
 // ---------------------------------------------------------------------------
 constexpr int SB = 16;      // tokens of a block
 
@@ -560,86 +562,132 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateArgs a, uint4* 
 }
 
 constexpr int SB_STAGES = 4;      // blocks on their way from memory
+// warps that share a tile of 16 value columns, each with 32 of its channels
+__host__ __device__ constexpr int tile_warps(int KS) { return KS / 2; }
+__host__ __device__ constexpr int stage_vecs(int KS) { return (rec_values(KS) + 1) * 32; }
 
+// grid (tiles of 16 value columns and, for kind 1, one for n; heads; entries)
 template <int KS, int KIND>
-__global__ void state_blocks_kernel(StateArgs a, const uint4* rec, int min_len) {
-    constexpr int COMMON = rec_values(KS) * 32;      // vectors that every warp of a head reads
-    extern __shared__ __align__(16) uint4 sb_smem[];               // [stages][COMMON + 32 warps]
+__global__ void __launch_bounds__(32 * tile_warps(KS)) state_blocks_kernel(StateArgs a, const uint4* rec, int min_len) {
+    constexpr int NW = tile_warps(KS), KH = KS / NW, THREADS = 32 * NW, COMMON = rec_values(KS) * 32, STAGE = stage_vecs(KS);
+    static_assert(KS % 2 == 0 && KS % NW == 0, "a tile's warps share its channels evenly");
+    extern __shared__ __align__(16) uint4 sb_smem[];               // [stages][STAGE], then [2][NW - 1][2][32] float4
     pdl_trigger();
     pdl_wait();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-    const int head = blockIdx.y, b = blockIdx.z, H = a.H, dk = a.dk, dv = a.dv;
-    const int DT = (dv + 15) / 16, n_warps = blockDim.x >> 5, tile = blockIdx.x * n_warps + warp;
+    const int tile = blockIdx.x, head = blockIdx.y, b = blockIdx.z, H = a.H, dk = a.dk, dv = a.dv, DT = (dv + 15) / 16;
     const int nb = entry_blocks(a.cu, b, a.n_seqs, min_len);
     if (nb == 0) return;
     int base = 0;             // the entry's first block among all
     for (int s = lane; s < b; s += 32) base += entry_blocks(a.cu, s, a.n_seqs, min_len);
     base = __reduce_add_sync(0xffffffffu, base);
     const int t0 = a.cu[b], t1 = a.cu[b + 1];
-    const bool is_n = KIND == 1 && tile == DT, live = tile < DT || is_n;
-    const int rec_vecs = (rec_values(KS) + DT) * 32, stage_vecs = COMMON + 32 * n_warps;
+    const bool is_n = KIND == 1 && tile == DT;
+    float4* other = reinterpret_cast<float4*>(sb_smem + SB_STAGES * STAGE);      // the other warps' shares of a block's outputs
 
-    auto load = [&](int blk) {
-        if (blk < nb) {
-            const uint4* src = rec + ((size_t)(base + blk) * H + head) * rec_vecs;
-            uint4* dst = sb_smem + (blk % SB_STAGES) * stage_vecs;
-            for (int e = tid; e < COMMON; e += blockDim.x)
-                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst + e)), "l"(src + e) : "memory");
-            if (tile < DT)
-                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst + COMMON + 32 * warp + lane)),
-                             "l"(src + COMMON + 32 * tile + lane) : "memory");
+    // a thread copies the vectors tid, tid + THREADS, ... of a record; the next block's record lies rec_step further on
+    const size_t rec_step = (size_t)(rec_values(KS) + DT) * 32 * H;
+    const uint4* src = rec + (size_t)base * rec_step + (size_t)head * ((rec_values(KS) + DT) * 32) + tid;
+    const uint32_t dst0 = (uint32_t)__cvta_generic_to_shared(sb_smem + tid);
+    int to_load = 0;
+    auto load = [&]() {
+        if (to_load < nb) {
+            const uint32_t dst = dst0 + (uint32_t)(to_load % SB_STAGES) * (STAGE * 16);
+#pragma unroll
+            for (int x = 0; x < (COMMON + THREADS - 1) / THREADS; ++x)
+                if ((x + 1) * THREADS <= COMMON || tid < COMMON - x * THREADS)
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst + x * THREADS * 16), "l"(src + x * THREADS) : "memory");
+            if (warp == NW - 1 && !is_n)
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst + (COMMON - 32 * (NW - 1)) * 16), "l"(src + COMMON - 32 * (NW - 1) + 32 * tile) : "memory");
+            src += rec_step;
+            ++to_load;
         }
         asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
 #pragma unroll
-    for (int s = 0; s < SB_STAGES - 1; ++s) load(s);
+    for (int s = 0; s < SB_STAGES - 1; ++s) load();
 
     float* slot = a.state + (size_t)a.slots[b] * a.slot_stride;
     float* Sg = slot + (size_t)head * dk * dv;
     float* ng = slot + (size_t)H * dk * dv + (size_t)head * dk;
     const int MB = m_copies(dv);
-    float* mg = slot + (size_t)H * dk * dv + (size_t)H * dk + (size_t)head * MB;
-    float S[2 * KS][4];       // S^T: row 16 tile + g (+ 8), channel 8 nt + 2 t (+ 1)
+    float* mg = slot + (size_t)H * dk * dv + (size_t)H * dk + (size_t)head * MB + (is_n ? MB - 1 : tile);
+    float S[2 * KH][4];       // S^T: row 16 tile + g (+ 8), channel 16 KH warp + 8 nt + 2 t (+ 1)
     auto state_at = [&](int nt, int e) -> float* {
-        const int d = 8 * nt + 2 * t + (e & 1), c = 16 * tile + g + (e >> 1) * 8;
+        const int d = 16 * KH * warp + 8 * nt + 2 * t + (e & 1), c = 16 * tile + g + (e >> 1) * 8;
         if (d >= dk) return nullptr;
         if (is_n) return (g == 0 && e < 2) ? ng + d : nullptr;
         return c < dv ? Sg + (size_t)d * dv + c : nullptr;
     };
 #pragma unroll
-    for (int nt = 0; nt < 2 * KS; ++nt)
+    for (int nt = 0; nt < 2 * KH; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const float* p = live ? state_at(nt, e) : nullptr;
+            const float* p = state_at(nt, e);
             S[nt][e] = p ? *p : 0.f;
         }
-    float m = (KIND == 1 && live) ? mg[is_n ? MB - 1 : tile] : 0.f;
+    float m = KIND == 1 ? *mg : 0.f;
+    uint4 v = make_uint4(g == 0 ? 0x3f803f80u : 0u, 0u, g == 0 ? 0x3f803f80u : 0u, 0u);      // a value column of ones (n)
 
-    for (int blk = 0; blk < nb; ++blk) {
+    float mine[2][4], m_at[2][2];      // the first warp's share of the block before and that block's maxima
+    const bool col0 = 16 * tile + g < dv, col1 = 16 * tile + g + 8 < dv;
+    const size_t row = (size_t)H * dv;
+    float* o_at = a.o + ((size_t)(t0 + 2 * t) * H + head) * dv + 16 * tile + g;      // this lane's first token of the next block to write
+    auto put_out = [&](int blk) {      // row (value column) 16 tile + g (+ 8), tokens 8 nt + 2 t (+ 1)
+        const float4* from = other + (blk & 1) * (NW - 1) * 64 + lane;
+        const int left = t1 - (t0 + blk * SB + 2 * t);      // the lane's tokens that are there: 8 nt + e < left
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+            float o[4] = {mine[nt][0], mine[nt][1], mine[nt][2], mine[nt][3]};
+#pragma unroll
+            for (int p = 0; p < NW - 1; ++p) {
+                const float4 x = from[64 * p + 32 * nt];
+                o[0] += x.x; o[1] += x.y; o[2] += x.z; o[3] += x.w;
+            }
+            if (KIND == 1 && is_n) {
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    if (g == 0 && 8 * nt + e < left)
+                        a.den[(size_t)(t0 + blk * SB + 2 * t + 8 * nt + e) * H + head] = fmaxf(fabsf(o[e]), expf(-m_at[nt][e])) + 1e-6f;
+            } else {
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    float* at = o_at + (8 * nt + e) * row;
+                    if (col0 && 8 * nt + e < left) at[0] = o[e];
+                    if (col1 && 8 * nt + e < left) at[8] = o[2 + e];
+                }
+            }
+        }
+        o_at += SB * row;
+    };
+
+    for (int blk = 0; blk <= nb; ++blk) {
         asm volatile("cp.async.wait_group %0;\n" ::"n"(SB_STAGES - 2) : "memory");
-        __syncthreads();      // this block's record is here; the buffer that the next load fills has been read
-        load(blk + SB_STAGES - 1);
-        if (!live) continue;
-        const uint4* st = sb_smem + (blk % SB_STAGES) * stage_vecs;
-        const float* sc = reinterpret_cast<const float*>(st + rec_scalars(KS) * 32);
-        uint4 v;
-        if (is_n) { v.x = v.z = g == 0 ? 0x3f803f80u : 0u; v.y = v.w = 0u; }
-        else v = st[COMMON + 32 * warp + lane];
-        // an MMA's result takes tens of cycles and a warp is alone on its scheduler: the rounded values' products and the
-        // remainders' have accumulators of their own, so that no chain is longer than KS
+        __syncthreads();      // this block's record and the other warps' shares of the one before are here
+        load();
+        if (warp == 0 && blk > 0) put_out(blk - 1);
+        if (blk == nb) break;
+        const uint4* st = sb_smem + (blk % SB_STAGES) * STAGE + lane;
+        const float* sc = reinterpret_cast<const float*>(sb_smem + (blk % SB_STAGES) * STAGE + rec_scalars(KS) * 32);
+        if (!is_n) v = st[COMMON];
+        // an MMA's result takes tens of cycles and few warps share a scheduler: the rounded values' products and the remainders'
+        // have accumulators of their own
         float oi[3][2][4], oa[2][4];
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
             for (int e = 0; e < 4; ++e) oi[0][nt][e] = oi[1][nt][e] = oi[2][nt][e] = oa[nt][e] = 0.f;
+        if (warp == NW - 1) {      // the last warp has the block's own tokens
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-            const uint4 w = st[(rec_scores(KS) + nt) * 32 + lane];
-            sb_mma(oa[nt], v.x, v.y, v.z, v.w, w.x, w.y);
-            sb_mma(oa[nt], v.x, v.y, v.z, v.w, w.z, w.w);
+            for (int nt = 0; nt < 2; ++nt) {
+                const uint4 w = st[(rec_scores(KS) + nt) * 32];
+                sb_mma(oa[nt], v.x, v.y, v.z, v.w, w.x, w.y);
+                sb_mma(oa[nt], v.x, v.y, v.z, v.w, w.z, w.w);
+            }
         }
+        const uint4* qs = st + warp * (KH * 2 * 32);
 #pragma unroll
-        for (int ks = 0; ks < KS; ++ks) {
+        for (int ks = 0; ks < KH; ++ks) {
             uint32_t h[4], l[4];
             sb_split(S[2 * ks][0], S[2 * ks][1], h[0], l[0]);
             sb_split(S[2 * ks][2], S[2 * ks][3], h[1], l[1]);
@@ -647,72 +695,72 @@ __global__ void state_blocks_kernel(StateArgs a, const uint4* rec, int min_len) 
             sb_split(S[2 * ks + 1][2], S[2 * ks + 1][3], h[3], l[3]);
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt) {
-                const uint4 w = st[(ks * 2 + nt) * 32 + lane];
+                const uint4 w = qs[(ks * 2 + nt) * 32];
                 sb_mma(oi[0][nt], h[0], h[1], h[2], h[3], w.x, w.y);
                 sb_mma(oi[1][nt], l[0], l[1], l[2], l[3], w.x, w.y);
                 if (KIND == 0) sb_mma(oi[2][nt], h[0], h[1], h[2], h[3], w.z, w.w);
             }
         }
-        // the block's outputs: row (value column) 16 tile + g (+ 8), tokens 8 nt + 2 t (+ 1)
-        const int tok0 = t0 + blk * SB;
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-            for (int x = 0; x < 2; ++x) {
-                const int i = 8 * nt + 2 * t + x, tok = tok0 + i;
-                float fi = 1.f, fa = 1.f, mi = 0.f;
-                if (KIND == 1) {
-                    const float G = sc[16 + i], M = fmaxf(m, G);
-                    fi = expf(m - M) * a.qscale;
-                    fa = expf(G - M);
-                    mi = sc[i] + M;
-                }
-                const float lo = fmaf(fi, oi[0][nt][x] + (oi[1][nt][x] + oi[2][nt][x]), fa * oa[nt][x]);
-                const float hi = fmaf(fi, oi[0][nt][2 + x] + (oi[1][nt][2 + x] + oi[2][nt][2 + x]), fa * oa[nt][2 + x]);
-                if (tok < t1) {
-                    if (is_n) {
-                        if (g == 0) a.den[(size_t)tok * H + head] = fmaxf(fabsf(lo), expf(-mi)) + 1e-6f;
-                    } else {
-                        float* o = a.o + ((size_t)tok * H + head) * dv + 16 * tile + g;
-                        if (16 * tile + g < dv) o[0] = lo;
-                        if (16 * tile + g + 8 < dv) o[8] = hi;
-                    }
-                }
-            }
-        // the state after it
+        // the state after the block
         float c1 = 1.f, c2 = 1.f;
+        const float m_before = m;
         if (KIND == 1) {
             const float G = sc[16 + SB - 1], M = fmaxf(m, G);
-            c1 = expf(m - M);
-            c2 = expf(G - M);
+            c1 = __expf(m - M);
+            c2 = __expf(G - M);
             m = sc[SB - 1] + M;
         }
+        const uint4* kts = st + (rec_keys(KS) + warp * 2 * KH) * 32;
+        const float* dec = sc + 16 * KH * warp + 2 * t;
 #pragma unroll
-        for (int nt = 0; nt < 2 * KS; ++nt) {
-            const uint4 w = st[(rec_keys(KS) + nt) * 32 + lane];
+        for (int nt = 0; nt < 2 * KH; ++nt) {
+            const uint4 w = kts[nt * 32];
             float u[4] = {0.f, 0.f, 0.f, 0.f};
             sb_mma(u, v.x, v.y, v.z, v.w, w.x, w.y);
             sb_mma(u, v.x, v.y, v.z, v.w, w.z, w.w);
             float d0 = c1, d1 = c1;
             if (KIND == 0) {
-                const float2 d = *reinterpret_cast<const float2*>(sc + 8 * nt + 2 * t);
+                const float2 d = *reinterpret_cast<const float2*>(dec + 8 * nt);
                 d0 = d.x;
                 d1 = d.y;
             }
 #pragma unroll
             for (int e = 0; e < 4; ++e) S[nt][e] = fmaf(e & 1 ? d1 : d0, S[nt][e], KIND == 1 ? c2 * u[e] : u[e]);
         }
+        // this warp's share of the block's outputs
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+            float fi[2] = {1.f, 1.f}, fa[2] = {1.f, 1.f};
+            if (KIND == 1) {
+                const float2 G = *reinterpret_cast<const float2*>(sc + 16 + 8 * nt + 2 * t), B = *reinterpret_cast<const float2*>(sc + 8 * nt + 2 * t);
+                const float M0 = fmaxf(m_before, G.x), M1 = fmaxf(m_before, G.y);
+                fi[0] = __expf(m_before - M0) * a.qscale;
+                fi[1] = __expf(m_before - M1) * a.qscale;
+                fa[0] = __expf(G.x - M0);
+                fa[1] = __expf(G.y - M1);
+                m_at[nt][0] = B.x + M0;
+                m_at[nt][1] = B.y + M1;
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                float x = oi[0][nt][e] + oi[1][nt][e];
+                if (KIND == 0) x += oi[2][nt][e];
+                if (KIND == 1) x *= fi[e & 1];
+                if (warp == NW - 1) x = KIND == 1 ? fmaf(fa[e & 1], oa[nt][e], x) : x + oa[nt][e];
+                mine[nt][e] = x;
+            }
+            if (NW > 1 && warp > 0) other[((blk & 1) * (NW - 1) + warp - 1) * 64 + 32 * nt + lane] = make_float4(mine[nt][0], mine[nt][1], mine[nt][2], mine[nt][3]);
+        }
     }
     asm volatile("cp.async.wait_group 0;\n" ::: "memory");
-    if (!live) return;
 #pragma unroll
-    for (int nt = 0; nt < 2 * KS; ++nt)
+    for (int nt = 0; nt < 2 * KH; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             float* p = state_at(nt, e);
             if (p) *p = S[nt][e];
         }
-    if (KIND == 1 && lane == 0) mg[is_n ? MB - 1 : tile] = m;
+    if (KIND == 1 && tid == 0) *mg = m;
 }
 
 // ---------------------------------------------------------------------------
@@ -797,12 +845,11 @@ void launch_scan(const StateArgs& a, int kind, int max_len, bool few, cudaStream
 }
 
 template <int KS, int KIND>
-int launch_chunked(const StateArgs& a, uint4* rec, int min_len, int n_blocks, int warps, int vec, cudaStream_t stream) {
+int launch_chunked(const StateArgs& a, uint4* rec, int min_len, int n_blocks, int vec, cudaStream_t stream) {
     constexpr int KD = 16 * KS, QP = KD + 8;
     const int DT = ceil_div(a.dv, 16), tiles = DT + (KIND == 1 ? 1 : 0);
     const size_t smem_p = (size_t)(KIND == 0 ? SB * QP : 64) * 4 + (size_t)SB * (2 * QP + DT * 16 + 8) * 2;
-    warps = min(warps, tiles);
-    const size_t smem_b = (size_t)SB_STAGES * (rec_values(KS) * 32 + 32 * warps) * 16;
+    const size_t smem_b = ((size_t)SB_STAGES * stage_vecs(KS) + (size_t)2 * (tile_warps(KS) - 1) * 64) * 16;
     if (smem_p > 227 * 1024 || smem_b > 227 * 1024) return PYRE_ERR_UNSUPPORTED;
     static size_t have_p[PYRE_MAX_DEVICES] = {}, have_b[PYRE_MAX_DEVICES] = {};
     const int dev = pyre_current_device();
@@ -818,7 +865,7 @@ int launch_chunked(const StateArgs& a, uint4* rec, int min_len, int n_blocks, in
     }
     pyre_launch(state_prepare_kernel<KS, KIND>, dim3(n_blocks, a.H), dim3(128), smem_p, stream, a, rec, min_len, vec);
     PYRE_LAUNCH_CHECK();
-    pyre_launch(state_blocks_kernel<KS, KIND>, dim3(ceil_div(tiles, warps), a.H, a.n_seqs), dim3(32 * warps), smem_b, stream, a, (const uint4*)rec, min_len);
+    pyre_launch(state_blocks_kernel<KS, KIND>, dim3(tiles, a.H, a.n_seqs), dim3(32 * tile_warps(KS)), smem_b, stream, a, (const uint4*)rec, min_len);
     PYRE_LAUNCH_CHECK();
     return 0;
 }
@@ -853,32 +900,28 @@ PYRE_API int pyre_state_scan(const void* proj, long long row_stride, int q_col, 
 PYRE_API int pyre_state_record_floats(int dk, int dv, int kind) {
     (void)kind;
     if (dk <= 0 || dk > 128 || dv <= 0 || dv > 512) return 0;
-    const int KS = dk <= 16 ? 1 : dk <= 32 ? 2 : dk <= 48 ? 3 : dk <= 64 ? 4 : dk <= 96 ? 6 : 8;
+    const int KS = dk <= 32 ? 2 : dk <= 64 ? 4 : dk <= 96 ? 6 : 8;
     return (rec_values(KS) + ceil_div(dv, 16)) * 128;
 }
 
 // The entries of at least min_len tokens, in blocks of 16 on the tensor cores (bfloat16 activations).  n_blocks: the sum of
-// ceil(tokens / 16) over those entries; scratch: n_blocks * H * pyre_state_record_floats floats, 16-byte aligned; warps: 16-column
-// tiles of a head's state per CTA.
+// ceil(tokens / 16) over those entries; scratch: n_blocks * H * pyre_state_record_floats floats, 16-byte aligned.
 PYRE_API int pyre_state_chunked(const void* proj, long long row_stride, int q_col, int k_col, int v_col, float qscale, const float* z,
                                 const float* z_bias, float tau, const float* gates, int n_parts, long long part_stride, const float* gate_bias, float cap, float* state,
                                 long long slot_stride, const int* slots, const int* cu_seqlens, float* o, float* den, void* scratch,
-                                int n_tokens, int n_seqs, int H, int dk, int dv, int min_len, int n_blocks, int kind, int warps,
-                                cudaStream_t stream) {
+                                int n_tokens, int n_seqs, int H, int dk, int dv, int min_len, int n_blocks, int kind, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0 || n_blocks <= 0) return 0;
     const StateArgs a = state_args(proj, row_stride, q_col, k_col, v_col, qscale, z, z_bias, tau, gates, n_parts, part_stride, gate_bias, cap,
                                    state, slot_stride, slots, cu_seqlens, o, den, n_seqs, H, dk, dv);
     const int rc = check_state(a, kind);
     if (rc) return rc;
-    if (min_len < 1 || warps < 1 || warps > 8 || !scratch || ((uintptr_t)scratch & 15)) return PYRE_ERR_BAD_ARG;
+    if (min_len < 1 || !scratch || ((uintptr_t)scratch & 15)) return PYRE_ERR_BAD_ARG;
     if (pyre_state_record_floats(dk, dv, kind) == 0) return PYRE_ERR_UNSUPPORTED;
     // rows of 8 elements at a time where everything starts on 16-byte boundaries
     const int vec = row_stride % 8 == 0 && q_col % 8 == 0 && k_col % 8 == 0 && v_col % 8 == 0 && dk % 8 == 0 && dv % 8 == 0 && ((uintptr_t)proj & 15) == 0;
     uint4* rec = (uint4*)scratch;
-#define GO(KSV) (kind == 0 ? launch_chunked<KSV, 0>(a, rec, min_len, n_blocks, warps, vec, stream) : launch_chunked<KSV, 1>(a, rec, min_len, n_blocks, warps, vec, stream))
-    if (dk <= 16) return GO(1);
+#define GO(KSV) (kind == 0 ? launch_chunked<KSV, 0>(a, rec, min_len, n_blocks, vec, stream) : launch_chunked<KSV, 1>(a, rec, min_len, n_blocks, vec, stream))
     if (dk <= 32) return GO(2);
-    if (dk <= 48) return GO(3);
     if (dk <= 64) return GO(4);
     if (dk <= 96) return GO(6);
     return GO(8);

@@ -31,6 +31,7 @@ from .step import StepEntry, Stepper
 
 DEFAULT_PAGE_SIZE = 16
 MAX_LIVE_REQUESTS = 64
+REPLAY_REQUESTS = 4     # the program's own default: state slots for so many live requests, so that a longer trace uses them again
 TOKEN_QUANTUM = 64      # --max-tokens counts each live request rounded up to a multiple of this (or of the page size)
 
 
@@ -130,13 +131,16 @@ def main(argv=None) -> int:
     ap.add_argument("--max-tokens", type=int, required=True,
                     help="most tokens live requests hold at any time (each rounded up to a multiple of 64)")
     ap.add_argument("--page-size", type=int, default=DEFAULT_PAGE_SIZE, help="tokens per cache page (any size the engine takes)")
+    ap.add_argument("--max-requests", type=int, default=REPLAY_REQUESTS, help="requests that are live at a time (state slots)")
     ap.add_argument("--device", default="cuda:0")
     ap.add_argument("--poison-freed-pages", action="store_true",
                     help="debug: fill pages with NaN when they go back to the pool")
     args = ap.parse_args(argv)
     if args.page_size <= 0:
         ap.error("--page-size must be positive")
-    _, _, stepper = build_runtime(args.model, args.dtype, args.max_tokens, args.page_size, args.device,
+    if args.max_requests <= 0:
+        ap.error("--max-requests must be positive")
+    _, _, stepper = build_runtime(args.model, args.dtype, args.max_tokens, args.page_size, args.device, args.max_requests,
                                   poison=args.poison_freed_pages)
 
     def done(msg):

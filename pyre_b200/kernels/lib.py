@@ -58,7 +58,7 @@ SIGNATURES: dict[str, tuple[str, list]] = {
     "pyre_wkv_scan": ("wkv", [P, P, P, P, P, P, P, P, P, LL, LL, P, P, P, P, P, I, I, I, I, I, F, I, P]),
     "pyre_state_scan": ("matrix_state", [P, LL, I, I, I, F, P, P, F, P, I, LL, P, F, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, P]),
     "pyre_state_record_floats": ("matrix_state", [I, I, I]),
-    "pyre_state_chunked": ("matrix_state", [P, LL, I, I, I, F, P, P, F, P, I, LL, P, F, P, LL, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P]),
+    "pyre_state_chunked": ("matrix_state", [P, LL, I, I, I, F, P, P, F, P, I, LL, P, F, P, LL, P, P, P, P, P, I, I, I, I, I, I, I, I, P]),
     "pyre_heads_finish": ("matrix_state", [P, P, P, I, P, LL, I, I, F, P, LL, I, I, I, F, I, P]),
     "pyre_linear_attention_scan": ("linear_attention", [P, LL, I, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, P]),
     "pyre_linear_attention_chunked": ("linear_attention", [P, LL, I, I, I, P, P, P, P, P, I, I, I, I, I, I, I, P]),

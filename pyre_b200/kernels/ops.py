@@ -2202,7 +2202,6 @@ def group_norm_gate(y: torch.Tensor, groups: int, weight: "torch.Tensor | None",
 # ---------------------------------------------------------------------------------- matrix states with decays that depend on the token
 STATE_MAX_DIM = 256            # query/key entries per head
 STATE_CHUNK_MIN_LEN = 32       # bfloat16 entries with at least this many tokens run in blocks on the tensor cores
-STATE_CHUNK_WARPS = {0: 2, 1: 4}      # tiles of 16 value columns per CTA of that kernel: gated linear attention, matrix memory
 USE_STATE_CHUNKS = True
 
 
@@ -2239,7 +2238,7 @@ def _matrix_state(kind: int, proj, q_col, k_col, v_col, q_scale, z, z_bias, tau,
         lib.call("pyre_state_chunked", proj.data_ptr(), W, int(q_col), int(k_col), int(v_col), float(q_scale), _ptr(z), _ptr(z_bias), float(tau),
                  _ptr(parts), n_parts, T * 2 * n_heads, _ptr(gate_bias), float(cap), state_layer.data_ptr(), slot_floats, slots.data_ptr(), cu_seqlens.data_ptr(),
                  o.data_ptr(), _ptr(den), scratch.data_ptr(), T, n_seqs, n_heads, qk_dim, v_dim, STATE_CHUNK_MIN_LEN, blocks, kind,
-                 STATE_CHUNK_WARPS[kind], _stream())
+                 _stream())
     if not blocks or any(n < STATE_CHUNK_MIN_LEN for n in lens):
         lib.call("pyre_state_scan", proj.data_ptr(), W, int(q_col), int(k_col), int(v_col), float(q_scale), _ptr(z), _ptr(z_bias), float(tau),
                  _ptr(parts), n_parts, T * 2 * n_heads, _ptr(gate_bias), float(cap), state_layer.data_ptr(), slot_floats, slots.data_ptr(), cu_seqlens.data_ptr(),
