@@ -388,10 +388,10 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_mma_kernel(const _
         } else {
             const uint32_t parity = (it / STAGES) & 1;
             if (!mbar_try_wait(bar0 + 8 * stage, parity)) {
-                const unsigned long long t0 = pyre_now_ns();
+                const long long t0 = clock64();
                 uint32_t spins = 0;
                 while (!mbar_try_wait(bar0 + 8 * stage, parity)) {
-                    if ((++spins & 255) == 0 && pyre_now_ns() - t0 > PYRE_WAIT_NS) { timed_out = true; break; }
+                    if ((++spins & 255) == 0 && clock64() - t0 > PYRE_WAIT_CYCLES) { timed_out = true; break; }
                 }
             }
             timed_out = __any_sync(0xffffffffu, timed_out);   // the whole warp gives up together

@@ -79,12 +79,12 @@ __device__ __forceinline__ bool mbar_try_wait(uint32_t bar, uint32_t parity) {
 }
 __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatile int* abort_flag, int* err_flag) {
     if (mbar_try_wait(bar, parity)) return true;
-    const unsigned long long t0 = pyre_now_ns();
+    const long long t0 = clock64();
     for (uint32_t it = 1;; ++it) {
         if (mbar_try_wait(bar, parity)) return true;
         if ((it & 63) == 0) {
             if (*abort_flag) return false;
-            if (pyre_now_ns() - t0 > PYRE_WAIT_NS) break;
+            if (clock64() - t0 > PYRE_WAIT_CYCLES) break;
         }
     }
     *abort_flag = 1;
@@ -229,7 +229,6 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     volatile int* abort_flag = reinterpret_cast<volatile int*>(gen + L::OFF_BAR + L::N_BARS * 8 + 8);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    pdl_trigger();
 
     // ---- which 128-token tile of which entry?  tiles are numbered from the end of each portion
     // (the last tile sees the most keys and starts first)
@@ -294,6 +293,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem_base = *tmem_slot;
+    pdl_trigger();      // only now: a later kernel's CTA must not find tensor memory that this one has yet to take
 
     if (warp == 0 || warp == 6) {
         // ---------------- producers: warp 0 copies Q and the K tiles, warp 6 the V tiles.  The whole

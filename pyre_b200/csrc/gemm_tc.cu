@@ -64,12 +64,12 @@ __device__ __forceinline__ bool mbar_try_wait(uint32_t bar, uint32_t parity) {
 // Bounded wait.  Returns false if the limit ran out or another thread already gave up.
 __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatile int* abort_flag, int* err_flag) {
     if (mbar_try_wait(bar, parity)) return true;
-    const unsigned long long t0 = pyre_now_ns();
+    const long long t0 = clock64();
     for (uint32_t it = 1;; ++it) {
         if (mbar_try_wait(bar, parity)) return true;
         if ((it & 63) == 0) {
             if (*abort_flag) return false;
-            if (pyre_now_ns() - t0 > PYRE_WAIT_NS) break;
+            if (clock64() - t0 > PYRE_WAIT_CYCLES) break;
         }
     }
     *abort_flag = 1;
@@ -94,6 +94,11 @@ __device__ __forceinline__ uint32_t mapa_u32(uint32_t addr, uint32_t rank) {
     uint32_t r;
     asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
     return r;
+}
+__device__ __forceinline__ uint32_t ld_cluster_u32(uint32_t addr) {
+    uint32_t v;
+    asm volatile("ld.volatile.shared::cluster.u32 %0, [%1];" : "=r"(v) : "r"(addr) : "memory");
+    return v;
 }
 __device__ __forceinline__ void cluster_sync_all() {
     asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
@@ -296,7 +301,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
     constexpr uint32_t ACC_COLS = BN <= 32 ? 32 : BN <= 64 ? 64 : BN <= 128 ? 128 : 256;   // columns of one accumulator (a power of two)
     constexpr uint32_t TMEM_COLS = 2 * ACC_COLS;        // power of two >= 32, at most 512
 
-    pdl_trigger();
     if (threadIdx.x == 0) {
         *abort_flag = 0;
         for (int s = 0; s < STAGES; ++s) {
@@ -309,7 +313,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
         }
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
+    // A pair takes and frees its tensor memory as one operation of both CTAs, and a CTA may start some time after its
+    // peer: both run before either allocates.  Without this a pair now and then never got its columns (one in about
+    // 10,000 launches that followed one another closely), and everything behind it in the stream waited for good.
+    if constexpr (CTAS == 2) { __syncwarp(); cluster_sync_all(); }
     if (warp == 1) {
+        __syncwarp();
         if constexpr (CTAS == 2) {      // the same warp of both CTAs allocates the same columns in both
             asm volatile("tcgen05.alloc.cta_group::2.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32((const void*)tmem_slot)), "r"(TMEM_COLS) : "memory");
             asm volatile("tcgen05.relinquish_alloc_permit.cta_group::2.sync.aligned;" ::: "memory");
@@ -323,6 +332,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
     else __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem_base = *tmem_slot;
+    // only now: a later kernel's CTA must not find tensor memory that this one has yet to take
+    pdl_trigger();
 
     if (warp == 0) {
         if (lane == 0) {
@@ -426,6 +437,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
         if (n_kb == 0) pdl_wait();   // nothing orders the zero stores after the earlier kernels otherwise
         // the accumulator goes back to the MMA thread, which for a pair sits in the first CTA
         const uint32_t acc_empty_to = CTAS == 2 ? mapa_u32(bar_acc_empty, 0) : bar_acc_empty;
+        [[maybe_unused]] const uint32_t abort_of_issuer = CTAS == 2 ? mapa_u32(base + L::TILES + L::N_BARS * 8 + 8, 0) : 0u;
         auto hand_back = [&](int buf) {
             if constexpr (CTAS == 2) asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(acc_empty_to + 8 * buf) : "memory");
             else asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(acc_empty_to + 8 * buf) : "memory");
@@ -473,7 +485,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
             bool ok = true;
             if (n_kb > 0) ok = mbar_wait(bar_acc_full + 8 * buf, (j >> 1) & 1, abort_flag, p.err_flag);
             ok = ok && !*abort_flag;   // the issuer signals the accumulator even when it gave up
-            if constexpr (CTAS == 2) ok = ok && (p.err_flag == nullptr || *(volatile int*)p.err_flag == 0);   // ... and it may sit in the peer CTA
+            if constexpr (CTAS == 2) ok = ok && ld_cluster_u32(abort_of_issuer) == 0;   // ... and it may sit in the peer CTA
             alive = __all_sync(0xffffffffu, ok);
             if constexpr (X_CONTIGUOUS_OUT) {
                 if (in_step) alive = epilogue_warps_all(alive);     // the warps meet at barriers below: all of them or none
@@ -1064,6 +1076,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
         if constexpr (CTAS == 2) asm volatile("tcgen05.dealloc.cta_group::2.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(TMEM_COLS) : "memory");
         else asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(TMEM_COLS) : "memory");
     }
+    if constexpr (CTAS == 2) { __syncwarp(); cluster_sync_all(); }     // ... nor before both have freed their columns
 }
 
 // ---------------------------------------------------------------- host side
